@@ -88,15 +88,17 @@ class PageLedger:
     gives pages back as soon as every position in them has fallen out of every future query's
     sight; the page-table entry then goes stale and is never read again.  ``chunk`` (tokens, or None): the
     group's layers only read keys of the query's own block of ``chunk`` positions, so every page wholly before
-    the block of the next position goes back the same way.
+    the block of the next position goes back the same way.  ``keep_first`` (tokens): pages that hold any of the sequence's first
+    ``keep_first`` positions stay whatever the window.
     """
 
     def __init__(self, n_pages: int, page_size: int, max_pages_per_slot: int, window: Optional[int] = None,
-                 chunk: Optional[int] = None):
+                 chunk: Optional[int] = None, keep_first: int = 0):
         self.page_size = page_size
         self.max_pages_per_slot = max_pages_per_slot
         self.window = window
         self.chunk = chunk
+        self.keep_pages = pages_for(keep_first, page_size)
         self.pool = FreeList(n_pages, "page")
         self._pages: Dict[int, Dict[int, int]] = {}  # slot -> {logical page index -> physical page}
 
@@ -145,7 +147,7 @@ class PageLedger:
         if held is None:
             raise CacheError(f"slot {slot} is not open")
         first = self.first_live_page(next_pos)
-        dead = [lp for lp in held if lp < first]
+        dead = [lp for lp in held if self.keep_pages <= lp < first]
         phys = [held.pop(lp) for lp in dead]
         self.pool.give_back(phys)
         return phys

@@ -39,7 +39,8 @@ class KVNeed:
     mixer keeps ONE key row and one value row per block of ``pool`` positions (what it puts there -- the block's mean, say --
     is its own business); those rows live in pages of their own that are never given back early, and reach the mixer as
     ``CacheEntry.pooled``.  With a ``pool``, ``window`` is how many of the last tokens' rows must stay (the mixer's own
-    window or the block it is still to summarise, whichever is longer)."""
+    window or the block it is still to summarise, whichever is longer).  ``keep_first``: with a ``window``, the sequence's first
+    ``keep_first`` tokens stay visible to every query, and the pages that hold them are never given back early."""
 
     kv_heads: int
     head_dim: int
@@ -48,6 +49,7 @@ class KVNeed:
     chunk: Optional[int] = None
     values: bool = True
     pool: Optional[int] = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -86,7 +88,7 @@ class _KVGroup:
         # what the owners could give back, the borrower may still read
         self.trims = trim and (need.window is not None or need.chunk is not None)
         self.ledger = PageLedger(n_pages, page_size, max_pages_per_slot, need.window if trim else None,
-                                 need.chunk if trim else None)
+                                 need.chunk if trim else None, need.keep_first if trim else 0)
         shape = (len(run_steps), n_pages, need.kv_heads, page_size, need.head_dim)
         self.k = torch.zeros(shape, dtype=dtype, device=device)
         self.v = torch.zeros(shape[:-1] + (need.v_head_dim or need.head_dim,), dtype=dtype, device=device) if need.values else None
@@ -161,8 +163,8 @@ class SequenceCache:
                     raise CacheError(f"run step {i}: state_need() must give a StateNeed or a mapping of names to StateNeed, "
                                      f"got {st!r}")
         for need, steps in by_need.items():
-            # a borrower's own view of the keys (window, chunk) must be the owner's for pages to be given back early
-            same_view = all(needs[i][0] is None or (needs[i][0].window, needs[i][0].chunk) == (need.window, need.chunk)
+            # a borrower's own view of the keys (window, chunk, kept first tokens) must be the owner's for pages to be given back early
+            same_view = all(needs[i][0] is None or (needs[i][0].window, needs[i][0].chunk, needs[i][0].keep_first) == (need.window, need.chunk, need.keep_first)
                             for i, src in enumerate(borrow) if src is not None and src in steps)
             g = _KVGroup(need, steps, n_pages, page_size, max_slots, max_pages_per_slot, dtype, device, trim=same_view)
             for j, s in enumerate(steps):

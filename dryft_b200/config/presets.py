@@ -201,6 +201,33 @@ PRESETS.update({
 EQUAL_SIZE.update({"kerirax-1k": "mogelix-1k", "kerirax-2k": "mogelix-2k"})
 
 
+def _dusupel(width: int, heads: int, kv_heads: int, dim: int, ff: int, window: int, keep: int, vocab: int, stretch: int, times: int,
+             tail: int) -> dict:
+    """A Dusupel ``config.json``: a stretch of ``stretch`` layers run ``times`` times, then ``tail`` more layers; every third
+    layer is a gated delta rule with a decay per channel, the others windowed attention beside a gated delta rule with a
+    decay per head."""
+    delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": 4}
+    pair = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": 4, "scale": dim ** -0.5,
+                     "rot": {"dims": dim, "base": 500000.0}, "mask": {"size": window, "keep_first": keep}}, "left_scale": 1.0,
+            "right": {"heads": heads, "kv_heads": heads // 2, "dim": dim, "vdim": dim, "conv": 4}, "right_scale": 1.0}
+    mlp = {"kind": "dense", "ff": ff}
+    layers = [{"type": "channel_delta", "mixer": delta, "mlp": mlp} if i % 3 == 1 else {"type": "parallel", "mixer": pair, "mlp": mlp}
+              for i in range(stretch + tail)]
+    return {"architecture": "Dusupel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "loop": {"start": 0, "stop": stretch, "times": times}, "layers": layers}
+
+
+# Dusupel shapes with layers the size of a real model's, and beside each the closest design at equal size: the Kerirax shape of
+# the same width, number of layer runs, head counts and size and vocabulary, its feed-forwards' size equal to the experts a
+# token uses there (its scan keeps a vector per channel where the delta rule keeps a matrix per head).
+PRESETS.update({
+    "dusupel-tiny": _dusupel(width=64, heads=4, kv_heads=2, dim=16, ff=96, window=40, keep=3, vocab=256, stretch=2, times=2, tail=1),
+    "dusupel-1k": _dusupel(width=1024, heads=8, kv_heads=2, dim=128, ff=2048, window=1024, keep=4, vocab=32768, stretch=2, times=3, tail=2),
+    "dusupel-2k": _dusupel(width=2048, heads=16, kv_heads=4, dim=128, ff=6144, window=2048, keep=4, vocab=65536, stretch=3, times=3, tail=3),
+})
+EQUAL_SIZE.update({"dusupel-1k": "kerirax-1k", "dusupel-2k": "kerirax-2k"})
+
+
 def preset(name: str) -> dict:
     if name not in PRESETS:
         raise KeyError(f"unknown preset {name!r}; known: " + ", ".join(sorted(PRESETS)))

@@ -1,0 +1,634 @@
+// A gated delta rule: per head a d x dv matrix state S that decays, is corrected along the current key and read along the
+// current query.  Everything behind the mixer's products is 32-bit; T is the activation type of the products' results.
+//
+// The mixer's input product leaves, per token, [q (G*d) | k (G*d) | v (H*dv)] from column x_off on (row stride ld) and one
+// logit per head for beta (column b_off); the decay's pre-activation is one value per head, or one per (head, key channel),
+// in rows of its own (`dec`, stride dec_ld).  Head h reads q and k of group h / (H/G).  Then
+//
+//     q, k, v   a short causal convolution per channel (shortconv.cuh), then silu
+//     q, k      divided by sqrt(sum of squares + 1e-6) per head; q also times d^(-1/2)
+//     beta      sigmoid(logit) ;   log g = -exp(A_log_h) * softplus(dec + dt_bias)      (per head or per key channel)
+//     S <- g S ;  u = beta (v - S^T k) ;  S <- S + k u^T ;  o = S^T q
+//     out       o / sqrt(mean over the head's dv of o^2 + eps) * norm_w * act(gate)     (act: silu or sigmoid; gate [H*dv])
+//
+// The state lives transposed, [slots, H, dv, dp] with dp = d rounded up to a multiple of four (the rows beyond d stay zero),
+// so that a value column's key vector is one piece of memory: the lanes of a warp hold RPL neighbouring rows each of a few
+// columns, and the sums over the key channels are warp sums.  Decays are applied as S + S * (g - 1) with g - 1 = expm1(log g):
+// a decay close to one keeps its distance from one.
+//
+// A step of many tokens goes by quads of four tokens.  With G_i the sum of the log decays of a quad's tokens 0..i,
+//
+//     u_i = beta_i (v_i - (k_i e^{G_i})^T S0) - sum_{j<i} beta_i A_ij u_j ,    A_ij = sum_c k_i k_j e^{G_i - G_j}
+//     o_i = (q_i e^{G_i})^T S0 + sum_{j<=i} P_ij u_j ,                         P_ij = sum_c q_i k_j e^{G_i - G_j}
+//     S4  = e^{G_3} S0 + sum_j (k_j e^{G_3 - G_j}) u_j^T
+//
+// so the eight products with S0 of a quad do not wait for one another and their warp sums are formed together; every exponent
+// is a sum of log decays, hence never positive.
+//
+//   delta_prep    one block per (tile of a sequence's tokens, head): a warp a quad; leaves a record per (quad, head):
+//                 [beta_i k_i e^{G_i}: 4 dp | q_i e^{G_i}: 4 dp | k_j e^{G_3-G_j}: 4 dp | expm1(G_3): dp | beta 4 |
+//                 beta_i A_ij: 6 (+2) | P: 4 x 4].  Further blocks convolve v into [n, H, dvp] floats.
+//   delta_walk    one block per (16 value columns, head, sequence), a warp four columns: quads in order from the slot's state,
+//                 records and v brought to shared memory a few quads ahead by cp.async; the 32 sums of a warp and quad are
+//                 formed by one butterfly that leaves lane l with sum l.  Leaves o [n, H*dv] and the slot's state.
+//   delta_norm    one warp per (token, head): the norm over dv, the weight and the gate.
+//   delta_decode  one token per sequence: one block per (head, sequence) does all of it, the ring's new row included.
+// Sequences with slot -1 (padding) are skipped (their output rows are zeros).  No block waits on another block; the only waits
+// are cp.async.wait_group and __syncthreads.
+#include "shortconv.cuh"
+#include <math.h>
+
+namespace {
+constexpr float UNIT_EPS = 1e-6f;     // inside the root of the unit vectors' length: fixed by the rule
+constexpr int QUAD = 4;
+constexpr int PREP_THREADS = 256;
+constexpr int V_SPLIT = 4;            // blocks a tile's quads are dealt to while v is convolved
+constexpr int WALK_WARPS = 4;
+constexpr int CPW = 4;                // value columns a warp of the walk owns
+constexpr int WALK_COLS = WALK_WARPS * CPW;
+constexpr int SCAL = 28;              // numbers of a record behind its vectors
+constexpr int DEC_COLS = 8;           // value columns a warp of the decode kernel holds at once
+constexpr int DEC_THREADS = 512;
+constexpr unsigned FULL = 0xffffffffu;
+
+__device__ __forceinline__ float sigmoidf_(float v) { return 1.f / (1.f + expf(-v)); }
+__device__ __forceinline__ float siluf_(float v) { return v / (1.f + expf(-v)); }
+__device__ __forceinline__ float softplusf_(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+__device__ __forceinline__ int seq_of(const int* __restrict__ cu_q, int n_seqs, int t) {
+  int lo = 0, hi = n_seqs - 1;        // largest b with cu_q[b] <= t
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  return lo;
+}
+
+// the first quad's record of sequence b whose first packed token is t0: sequences take disjoint ranges in order
+__device__ __forceinline__ size_t quad_base(int t0, int b) { return (size_t)((t0 + 3 * b) / QUAD); }
+
+__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
+  unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem));
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N)); }
+
+// RPL neighbouring floats; rows behind dp read as zeros (dp is a multiple of four, RPL a divisor or a multiple of it)
+template <int RPL>
+__device__ __forceinline__ void load_rows(float (&v)[RPL], const float* p, int row0, int dp) {
+  if constexpr (RPL >= 4) {
+#pragma unroll
+    for (int e = 0; e < RPL; e += 4) {
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (row0 + e < dp) x = *reinterpret_cast<const float4*>(p + row0 + e);
+      v[e] = x.x; v[e + 1] = x.y; v[e + 2] = x.z; v[e + 3] = x.w;
+    }
+  } else if constexpr (RPL == 2) {
+    float2 x = make_float2(0.f, 0.f);
+    if (row0 < dp) x = *reinterpret_cast<const float2*>(p + row0);
+    v[0] = x.x; v[1] = x.y;
+  } else {
+    v[0] = row0 < dp ? p[row0] : 0.f;
+  }
+}
+template <int RPL>
+__device__ __forceinline__ void store_rows(const float (&v)[RPL], float* p, int row0, int dp) {
+  if constexpr (RPL >= 4) {
+#pragma unroll
+    for (int e = 0; e < RPL; e += 4)
+      if (row0 + e < dp) *reinterpret_cast<float4*>(p + row0 + e) = make_float4(v[e], v[e + 1], v[e + 2], v[e + 3]);
+  } else if constexpr (RPL == 2) {
+    if (row0 < dp) *reinterpret_cast<float2*>(p + row0) = make_float2(v[0], v[1]);
+  } else {
+    if (row0 < dp) p[row0] = v[0];
+  }
+}
+
+// x[i] summed over the warp, i < N (a power of two up to 32); lane l is left with the sum of index l / (32 / N)
+template <int N>
+__device__ __forceinline__ float butterfly(float (&x)[N], int lane) {
+  int off = 16;
+#pragma unroll
+  for (int n = N / 2; n > 0; n >>= 1, off >>= 1) {
+    const bool up = (lane & off) != 0;
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+      if (i < n) {
+        const float send = up ? x[i] : x[i + n], keep = up ? x[i + n] : x[i];
+        x[i] = keep + __shfl_xor_sync(FULL, send, off);
+      }
+    }
+  }
+  float r = x[0];
+  for (; off > 0; off >>= 1) r += __shfl_xor_sync(FULL, r, off);
+  return r;
+}
+
+template <typename T, int DR, bool CHAN>
+__global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
+    const T* __restrict__ proj, int ld, int x_off, int b_off, const T* __restrict__ dec, int dec_ld, const float* __restrict__ conv_w,
+    int taps, const T* __restrict__ ring, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+    const int* __restrict__ tile_tok0, const int* __restrict__ tile_rows, const int* __restrict__ cu_q, int n_seqs,
+    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, int H, int G, int d, int dv, int dp, int dvp,
+    float* __restrict__ rec, float* __restrict__ vbuf) {
+  const int tile = blockIdx.x;
+  const int tok0 = tile_tok0[tile], rows = tile_rows[tile];
+  const int slot = tok_slot[tok0];
+  if (slot < 0 || rows <= 0) return;
+  const int b = seq_of(cu_q, n_seqs, tok0);
+  const int t0 = cu_q[b], n = cu_q[b + 1] - t0, p0 = tok_pos[t0], i_tile = tok0 - t0;
+  const T* x = proj + x_off;
+  const int CH = 2 * G * d + H * dv;
+  const int nq = (rows + QUAD - 1) / QUAD;
+
+  if ((int)blockIdx.y >= H) {      // v: a thread a column of [H, dvp]
+    const int part = (int)blockIdx.y - H;
+    const int col = (part / V_SPLIT) * PREP_THREADS + threadIdx.x;
+    if (col >= H * dvp) return;
+    const int h = col / dvp, c = col % dvp;
+    for (int qd = part % V_SPLIT; qd < nq; qd += V_SPLIT) {
+      const int i0 = i_tile + qd * QUAD;
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      if (c < dv) conv4<T>(acc, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, 2 * G * d + h * dv + c);
+#pragma unroll
+      for (int k = 0; k < QUAD; ++k)
+        if (i0 + k < n) vbuf[(size_t)(t0 + i0 + k) * H * dvp + col] = c < dv ? siluf_(acc[k]) : 0.f;
+    }
+    return;
+  }
+
+  const int h = blockIdx.y, g = h / (H / G);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float rate = -expf(a_log[h]);
+  const size_t RS = (size_t)13 * dp + SCAL;
+  for (int qd = warp; qd < nq; qd += PREP_THREADS / 32) {
+    const int i0 = i_tile + qd * QUAD, m = min(QUAD, n - i0);
+    float q[QUAD][DR], k[QUAD][DR], lg[QUAD][DR];
+    float sq[QUAD] = {0.f, 0.f, 0.f, 0.f}, sk[QUAD] = {0.f, 0.f, 0.f, 0.f};
+    float head_lg[QUAD];
+    if (!CHAN) {
+#pragma unroll
+      for (int i = 0; i < QUAD; ++i)
+        head_lg[i] = i < m ? rate * softplusf_(to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h]) + dt_bias[h]) : 0.f;
+    }
+#pragma unroll
+    for (int r = 0; r < DR; ++r) {
+      const int c = lane + 32 * r;
+      float aq[4] = {0.f, 0.f, 0.f, 0.f}, ak[4] = {0.f, 0.f, 0.f, 0.f};
+      if (c < d) {
+        conv4<T>(aq, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, g * d + c);
+        conv4<T>(ak, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, (G + g) * d + c);
+      }
+#pragma unroll
+      for (int i = 0; i < QUAD; ++i) {
+        const bool on = c < d && i < m;
+        q[i][r] = on ? siluf_(aq[i]) : 0.f;
+        k[i][r] = on ? siluf_(ak[i]) : 0.f;
+        sq[i] = fmaf(q[i][r], q[i][r], sq[i]);
+        sk[i] = fmaf(k[i][r], k[i][r], sk[i]);
+        if (CHAN) lg[i][r] = on ? rate * softplusf_(to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h * d + c]) + dt_bias[h * d + c]) : 0.f;
+        else lg[i][r] = head_lg[i];
+      }
+    }
+    const float qscale = 1.f / sqrtf((float)d);
+    float beta[QUAD];
+#pragma unroll
+    for (int i = 0; i < QUAD; ++i) {
+      const float rq = qscale / sqrtf(warp_sum(sq[i]) + UNIT_EPS), rk = 1.f / sqrtf(warp_sum(sk[i]) + UNIT_EPS);
+      beta[i] = i < m ? sigmoidf_(to_f32<T>(proj[(size_t)(t0 + i0 + i) * ld + b_off + h])) : 0.f;
+#pragma unroll
+      for (int r = 0; r < DR; ++r) { q[i][r] *= rq; k[i][r] *= rk; }
+    }
+    float A[6] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f};      // (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
+    float P[10] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};   // (0,0) (1,0) (1,1) (2,0) ...
+    float* rc = rec + ((quad_base(t0, b) + (size_t)(i0 / QUAD)) * H + h) * RS;
+#pragma unroll
+    for (int r = 0; r < DR; ++r) {
+      const int c = lane + 32 * r;
+      const float l1 = lg[1][r], l2 = lg[2][r], l3 = lg[3][r];
+      const float g0 = lg[0][r], g1 = g0 + l1, g2 = g1 + l2, g3 = g2 + l3;
+      // decays from token j to token i of the quad: sums of the log decays in between, so e^0 = 1 where nothing decays
+      const float e10 = expf(l1), e21 = expf(l2), e20 = expf(l1 + l2), e32 = expf(l3), e31 = expf(l2 + l3), e30 = expf(l1 + l2 + l3);
+      A[0] = fmaf(k[1][r] * k[0][r], e10, A[0]);
+      A[1] = fmaf(k[2][r] * k[0][r], e20, A[1]); A[2] = fmaf(k[2][r] * k[1][r], e21, A[2]);
+      A[3] = fmaf(k[3][r] * k[0][r], e30, A[3]); A[4] = fmaf(k[3][r] * k[1][r], e31, A[4]); A[5] = fmaf(k[3][r] * k[2][r], e32, A[5]);
+      P[0] = fmaf(q[0][r], k[0][r], P[0]);
+      P[1] = fmaf(q[1][r] * k[0][r], e10, P[1]); P[2] = fmaf(q[1][r], k[1][r], P[2]);
+      P[3] = fmaf(q[2][r] * k[0][r], e20, P[3]); P[4] = fmaf(q[2][r] * k[1][r], e21, P[4]); P[5] = fmaf(q[2][r], k[2][r], P[5]);
+      P[6] = fmaf(q[3][r] * k[0][r], e30, P[6]); P[7] = fmaf(q[3][r] * k[1][r], e31, P[7]);
+      P[8] = fmaf(q[3][r] * k[2][r], e32, P[8]); P[9] = fmaf(q[3][r], k[3][r], P[9]);
+      if (c < dp) {
+        const float x0 = expf(g0), x1 = expf(g1), x2 = expf(g2), x3 = expf(g3);
+        rc[c] = beta[0] * k[0][r] * x0; rc[dp + c] = beta[1] * k[1][r] * x1;
+        rc[2 * dp + c] = beta[2] * k[2][r] * x2; rc[3 * dp + c] = beta[3] * k[3][r] * x3;
+        rc[4 * dp + c] = q[0][r] * x0; rc[5 * dp + c] = q[1][r] * x1; rc[6 * dp + c] = q[2][r] * x2; rc[7 * dp + c] = q[3][r] * x3;
+        rc[8 * dp + c] = k[0][r] * e30; rc[9 * dp + c] = k[1][r] * e31; rc[10 * dp + c] = k[2][r] * e32; rc[11 * dp + c] = k[3][r];
+        rc[12 * dp + c] = c < d ? expm1f(g3) : 0.f;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 6; ++i) A[i] = warp_sum(A[i]);
+#pragma unroll
+    for (int i = 0; i < 10; ++i) P[i] = warp_sum(P[i]);
+    if (lane == 0) {
+      float4* s = reinterpret_cast<float4*>(rc + 13 * dp);
+      s[0] = make_float4(beta[0], beta[1], beta[2], beta[3]);
+      s[1] = make_float4(beta[1] * A[0], beta[2] * A[1], beta[2] * A[2], beta[3] * A[3]);
+      s[2] = make_float4(beta[3] * A[4], beta[3] * A[5], 0.f, 0.f);
+      s[3] = make_float4(P[0], 0.f, 0.f, 0.f);
+      s[4] = make_float4(P[1], P[2], 0.f, 0.f);
+      s[5] = make_float4(P[3], P[4], P[5], 0.f);
+      s[6] = make_float4(P[6], P[7], P[8], P[9]);
+    }
+  }
+}
+
+template <int RPL> struct WalkStages { static constexpr int value = RPL >= 8 ? 3 : 4; };   // quads in shared memory at once
+
+template <int RPL>
+__global__ void __launch_bounds__(WALK_WARPS * 32) delta_walk_kernel(
+    const float* __restrict__ rec, const float* __restrict__ vbuf, const int* __restrict__ cu_q, const int* __restrict__ seq_slot,
+    int H, int dv, int dp, int dvp, float* __restrict__ state, float* __restrict__ o) {
+  constexpr int NST = WalkStages<RPL>::value;
+  extern __shared__ __align__(16) float stage_mem[];
+  __shared__ __align__(16) float sums[WALK_WARPS][16];
+  const int b = blockIdx.z, h = blockIdx.y;
+  const int slot = seq_slot[b];
+  const int t0 = cu_q[b], n = cu_q[b + 1] - t0;
+  if (slot < 0 || n <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int blk0 = blockIdx.x * WALK_COLS, col0 = blk0 + warp * CPW;
+  const int RS = 13 * dp + SCAL;
+  const int stage_floats = RS + QUAD * WALK_COLS;
+  const int nq = (n + QUAD - 1) / QUAD;
+  const float* rc0 = rec + (quad_base(t0, b) * H + h) * (size_t)RS;
+  const size_t rstep = (size_t)H * RS;
+
+  auto issue = [&](int j) {      // record and v rows of quad j -> its stage
+    if (j < nq) {
+      float* sm = stage_mem + (j % NST) * stage_floats;
+      const float* src = rc0 + (size_t)j * rstep;
+      for (int i = tid * 4; i < RS; i += WALK_WARPS * 32 * 4) cp_async16(sm + i, src + i);
+      for (int i = tid; i < QUAD * (WALK_COLS / 4); i += WALK_WARPS * 32) {
+        const int r = i / (WALK_COLS / 4), c = (i % (WALK_COLS / 4)) * 4;
+        const int t = min(j * QUAD + r, n - 1);      // a quad's missing tokens have beta = 0: any finite row will do
+        cp_async16(sm + RS + r * WALK_COLS + c, vbuf + (size_t)(t0 + t) * H * dvp + (size_t)h * dvp + blk0 + c);
+      }
+    }
+    cp_async_commit();
+  };
+#pragma unroll
+  for (int j = 0; j < NST - 1; ++j) issue(j);
+
+  float S[CPW][RPL];
+  float* sp = state + (((size_t)slot * H + h) * dv + col0) * dp;
+  const int row0 = lane * RPL;
+#pragma unroll
+  for (int c = 0; c < CPW; ++c) {
+    if (col0 + c < dv) load_rows<RPL>(S[c], sp + (size_t)c * dp, row0, dp);
+    else
+#pragma unroll
+      for (int r = 0; r < RPL; ++r) S[c][r] = 0.f;
+  }
+
+  for (int j = 0; j < nq; ++j) {
+    cp_async_wait<NST - 2>();
+    __syncthreads();               // quad j is in shared memory; everyone is done with quad j - 1
+    issue(j + NST - 1);
+    const float* sm = stage_mem + (j % NST) * stage_floats;
+    float x[32];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      float kt[RPL];
+      load_rows<RPL>(kt, sm + i * dp, row0, dp);
+#pragma unroll
+      for (int c = 0; c < CPW; ++c) {
+        float a = kt[0] * S[c][0];
+#pragma unroll
+        for (int r = 1; r < RPL; ++r) a = fmaf(kt[r], S[c][r], a);
+        x[i * CPW + c] = a;
+      }
+    }
+    const float mine = butterfly<32>(x, lane);     // lane l < 16: key sum of token l / 4, column l % 4; above: query sums
+    if (lane < 16) sums[warp][lane] = mine;
+    __syncwarp();
+    const float* sc = sm + 13 * dp;
+    const float4 be = *reinterpret_cast<const float4*>(sc), a0 = *reinterpret_cast<const float4*>(sc + 4),
+                 a1 = *reinterpret_cast<const float4*>(sc + 8);
+    float u[QUAD][CPW];
+    {
+      const float bi[4] = {be.x, be.y, be.z, be.w};
+      const float A[6] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y};
+#pragma unroll
+      for (int i = 0; i < QUAD; ++i) {
+        const float4 dk = *reinterpret_cast<const float4*>(&sums[warp][i * 4]);
+        const float4 vv = *reinterpret_cast<const float4*>(sm + RS + i * WALK_COLS + warp * CPW);
+        u[i][0] = fmaf(bi[i], vv.x, -dk.x); u[i][1] = fmaf(bi[i], vv.y, -dk.y);
+        u[i][2] = fmaf(bi[i], vv.z, -dk.z); u[i][3] = fmaf(bi[i], vv.w, -dk.w);
+#pragma unroll
+        for (int jj = 0; jj < i; ++jj)
+#pragma unroll
+          for (int c = 0; c < CPW; ++c) u[i][c] = fmaf(-A[i * (i - 1) / 2 + jj], u[jj][c], u[i][c]);
+      }
+    }
+    {
+      float gm[RPL];
+      load_rows<RPL>(gm, sm + 12 * dp, row0, dp);
+#pragma unroll
+      for (int c = 0; c < CPW; ++c)
+#pragma unroll
+        for (int r = 0; r < RPL; ++r) S[c][r] = fmaf(S[c][r], gm[r], S[c][r]);
+    }
+#pragma unroll
+    for (int i = 0; i < QUAD; ++i) {
+      float kb[RPL];
+      load_rows<RPL>(kb, sm + (8 + i) * dp, row0, dp);
+#pragma unroll
+      for (int c = 0; c < CPW; ++c)
+#pragma unroll
+        for (int r = 0; r < RPL; ++r) S[c][r] = fmaf(kb[r], u[i][c], S[c][r]);
+    }
+    if (lane >= 16) {
+      const int i = (lane >> 2) & 3, c = lane & 3;
+      const float4 Pr = *reinterpret_cast<const float4*>(sc + 12 + i * 4);
+      const float pr[4] = {Pr.x, Pr.y, Pr.z, Pr.w};
+      float val = mine;
+#pragma unroll
+      for (int jj = 0; jj < QUAD; ++jj) {
+        const float uc = c < 2 ? (c == 0 ? u[jj][0] : u[jj][1]) : (c == 2 ? u[jj][2] : u[jj][3]);
+        val = fmaf(pr[jj], uc, val);
+      }
+      const int t = j * QUAD + i;
+      if (t < n && col0 + c < dv) o[(size_t)(t0 + t) * H * dv + (size_t)h * dv + col0 + c] = val;
+    }
+  }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int c = 0; c < CPW; ++c)
+    if (col0 + c < dv) store_rows<RPL>(S[c], sp + (size_t)c * dp, row0, dp);
+}
+
+constexpr int NORM_WARPS = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(NORM_WARPS * 32) delta_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_ld,
+                                                                    const float* __restrict__ w, float eps, int sigmoid_gate,
+                                                                    const int* __restrict__ tok_slot, T* __restrict__ out, int n, int H,
+                                                                    int dv) {
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * NORM_WARPS + (threadIdx.x >> 5);
+  if (item >= (long long)n * H) return;
+  const int t = (int)(item / H), h = (int)(item % H);
+  T* dst = out + (size_t)t * H * dv + (size_t)h * dv;
+  if (tok_slot[t] < 0) {
+    for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(0.f);
+    return;
+  }
+  const float* src = o + (size_t)t * H * dv + (size_t)h * dv;
+  const T* gt = gate + (size_t)t * gate_ld + (size_t)h * dv;
+  float ss = 0.f;
+  for (int c = lane; c < dv; c += 32) { const float v = src[c]; ss = fmaf(v, v, ss); }
+  const float rinv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
+  for (int c = lane; c < dv; c += 32) {
+    const float z = to_f32<T>(gt[c]);
+    dst[c] = from_f32<T>(src[c] * rinv * w[c] * (sigmoid_gate ? sigmoidf_(z) : siluf_(z)));
+  }
+}
+
+template <typename T, int RPL, bool CHAN>
+__global__ void __launch_bounds__(DEC_THREADS) delta_decode_kernel(
+    const T* __restrict__ proj, int ld, int x_off, int b_off, const T* __restrict__ dec, int dec_ld, const T* __restrict__ gate,
+    int gate_ld, const float* __restrict__ conv_w, int taps, T* __restrict__ ring, const float* __restrict__ a_log,
+    const float* __restrict__ dt_bias, const float* __restrict__ norm_w, float eps, int sigmoid_gate, const int* __restrict__ tok_slot,
+    const int* __restrict__ tok_pos, int H, int G, int d, int dv, int dp, float* __restrict__ state, T* __restrict__ out) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float scratch[33];
+  const int h = blockIdx.x, t = blockIdx.y;
+  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, nwarp = nthr >> 5;
+  const int slot = tok_slot[t];
+  if (slot < 0) {
+    for (int c = tid; c < dv; c += nthr) out[(size_t)t * H * dv + (size_t)h * dv + c] = from_f32<T>(0.f);
+    return;
+  }
+  const int row0 = lane * RPL;
+  float* sp = state + ((size_t)slot * H + h) * dv * dp;
+  float S[DEC_COLS][RPL];
+  // the first columns' state is requested before anything else
+#pragma unroll
+  for (int c = 0; c < DEC_COLS; ++c) {
+    const int col = warp * DEC_COLS + c;
+    if (col < dv) load_rows<RPL>(S[c], sp + (size_t)col * dp, row0, dp);
+    else
+#pragma unroll
+      for (int r = 0; r < RPL; ++r) S[c][r] = 0.f;
+  }
+  float *qs = sm, *ks = qs + dp, *gm = ks + dp, *vs = gm + dp, *os = vs + dv;
+  const int pos = tok_pos[t], g = h / (H / G), CH = 2 * G * d + H * dv;
+  const bool first = h % (H / G) == 0;                       // one head of a group stores the group's q and k in the ring
+  const T* x = proj + x_off;
+  T* ring_row = ring + ((size_t)slot * taps + pos % taps) * CH;
+  float aq = 0.f, ak = 0.f, aqk = 0.f;
+  for (int c = tid; c < dp; c += nthr) {
+    float q = 0.f, k = 0.f, gmc = 0.f;
+    if (c < d) {
+      const int cq = g * d + c, ck = (G + g) * d + c;
+      q = siluf_(conv1<T>(conv_w, x, ld, ring, taps, CH, slot, t, pos, 0, cq));
+      k = siluf_(conv1<T>(conv_w, x, ld, ring, taps, CH, slot, t, pos, 0, ck));
+      if (first && taps > 1) { ring_row[cq] = x[(size_t)t * ld + cq]; ring_row[ck] = x[(size_t)t * ld + ck]; }
+      const int gi = CHAN ? h * d + c : h;
+      gmc = expm1f(-expf(a_log[h]) * softplusf_(to_f32<T>(dec[(size_t)t * dec_ld + gi]) + dt_bias[gi]));
+    }
+    qs[c] = q; ks[c] = k; gm[c] = gmc;
+    aq = fmaf(q, q, aq); ak = fmaf(k, k, ak); aqk = fmaf(q, k, aqk);
+  }
+  for (int c = tid; c < dv; c += nthr) {
+    const int cv = 2 * G * d + h * dv + c;
+    vs[c] = siluf_(conv1<T>(conv_w, x, ld, ring, taps, CH, slot, t, pos, 0, cv));
+    if (taps > 1) ring_row[cv] = x[(size_t)t * ld + cv];
+  }
+  const float rq = 1.f / (sqrtf((float)d) * sqrtf(block_sum(aq, scratch) + UNIT_EPS));
+  const float rk = 1.f / sqrtf(block_sum(ak, scratch) + UNIT_EPS);
+  const float qk = block_sum(aqk, scratch) * rq * rk;        // (the barriers inside also publish q, k, v and the decays)
+  const float beta = sigmoidf_(to_f32<T>(proj[(size_t)t * ld + b_off + h]));
+  float kr[RPL], qr[RPL], gr[RPL];
+  load_rows<RPL>(kr, ks, row0, dp);
+  load_rows<RPL>(qr, qs, row0, dp);
+  load_rows<RPL>(gr, gm, row0, dp);
+#pragma unroll
+  for (int r = 0; r < RPL; ++r) { kr[r] *= rk; qr[r] *= rq; }
+
+  for (int base = warp * DEC_COLS; base < dv; base += nwarp * DEC_COLS) {
+    if (base != warp * DEC_COLS) {
+#pragma unroll
+      for (int c = 0; c < DEC_COLS; ++c) {
+        if (base + c < dv) load_rows<RPL>(S[c], sp + (size_t)(base + c) * dp, row0, dp);
+        else
+#pragma unroll
+          for (int r = 0; r < RPL; ++r) S[c][r] = 0.f;
+      }
+    }
+    float xs[2 * DEC_COLS];
+#pragma unroll
+    for (int c = 0; c < DEC_COLS; ++c) {
+      float a = 0.f, q = 0.f;
+#pragma unroll
+      for (int r = 0; r < RPL; ++r) {
+        S[c][r] = fmaf(S[c][r], gr[r], S[c][r]);
+        a = fmaf(kr[r], S[c][r], a);
+        q = fmaf(qr[r], S[c][r], q);
+      }
+      xs[c] = a;
+      xs[DEC_COLS + c] = q;
+    }
+    const float mine = butterfly<2 * DEC_COLS>(xs, lane);    // lane l: sum l / 2 (key sums of the eight columns, then query sums)
+    const int id = lane >> 1, c_own = id & (DEC_COLS - 1), col = base + c_own;
+    const float uval = col < dv ? beta * (vs[col] - mine) : 0.f;
+    const float u_own = __shfl_sync(FULL, uval, 2 * c_own);
+    if (id >= DEC_COLS && !(lane & 1) && col < dv) os[col] = fmaf(qk, u_own, mine);
+#pragma unroll
+    for (int c = 0; c < DEC_COLS; ++c) {
+      const float u = __shfl_sync(FULL, uval, 2 * c);
+#pragma unroll
+      for (int r = 0; r < RPL; ++r) S[c][r] = fmaf(kr[r], u, S[c][r]);
+      if (base + c < dv) store_rows<RPL>(S[c], sp + (size_t)(base + c) * dp, row0, dp);
+    }
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < dv; c += nthr) ss = fmaf(os[c], os[c], ss);
+  const float rinv = 1.f / sqrtf(block_sum(ss, scratch) / (float)dv + eps);
+  for (int c = tid; c < dv; c += nthr) {
+    const float z = to_f32<T>(gate[(size_t)t * gate_ld + (size_t)h * dv + c]);
+    out[(size_t)t * H * dv + (size_t)h * dv + c] = from_f32<T>(os[c] * rinv * norm_w[c] * (sigmoid_gate ? sigmoidf_(z) : siluf_(z)));
+  }
+}
+
+template <typename T, int DR, bool CHAN>
+int prep_launch(const void* proj, int ld, int x_off, int b_off, const void* dec, int dec_ld, const float* conv_w, int taps,
+                const void* ring, const float* a_log, const float* dt_bias, const int* tile_tok0, const int* tile_rows, int n_tiles,
+                const int* cu_q, int n_seqs, const int* tok_slot, const int* tok_pos, int H, int G, int d, int dv, int dp, int dvp,
+                float* rec, float* vbuf, cudaStream_t st) {
+  const long long vb = ((long long)H * dvp + PREP_THREADS - 1) / PREP_THREADS * V_SPLIT;
+  if (H + vb > 65535) return DRYFT_ERR_UNSUPPORTED;
+  dim3 grid(n_tiles, (unsigned)(H + vb));
+  delta_prep_kernel<T, DR, CHAN><<<grid, PREP_THREADS, 0, st>>>(
+      (const T*)proj, ld, x_off, b_off, (const T*)dec, dec_ld, conv_w, taps, (const T*)ring, a_log, dt_bias, tile_tok0, tile_rows, cu_q,
+      n_seqs, tok_slot, tok_pos, H, G, d, dv, dp, dvp, rec, vbuf);
+  return launch_status();
+}
+
+template <int RPL>
+int walk_launch(const float* rec, const float* vbuf, const int* cu_q, const int* seq_slot, int n_seqs, int H, int dv, int dp, int dvp,
+                float* state, float* o, cudaStream_t st) {
+  const size_t smem = sizeof(float) * WalkStages<RPL>::value * ((size_t)13 * dp + SCAL + QUAD * WALK_COLS);
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(delta_walk_kernel<RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  dim3 grid((dv + WALK_COLS - 1) / WALK_COLS, H, n_seqs);
+  delta_walk_kernel<RPL><<<grid, WALK_WARPS * 32, smem, st>>>(rec, vbuf, cu_q, seq_slot, H, dv, dp, dvp, state, o);
+  return launch_status();
+}
+
+template <typename T, int RPL, bool CHAN>
+int decode_launch(const void* proj, int ld, int x_off, int b_off, const void* dec, int dec_ld, const void* gate, int gate_ld,
+                  const float* conv_w, int taps, void* ring, const float* a_log, const float* dt_bias, const float* norm_w, float eps,
+                  int sigmoid_gate, const int* tok_slot, const int* tok_pos, int n, int H, int G, int d, int dv, int dp, float* state,
+                  void* out, cudaStream_t st) {
+  const size_t smem = sizeof(float) * ((size_t)3 * dp + 2 * dv);
+  if (smem > 48 * 1024) return DRYFT_ERR_UNSUPPORTED;
+  int warps = (dv + DEC_COLS - 1) / DEC_COLS;
+  warps = warps < 4 ? 4 : (warps > DEC_THREADS / 32 ? DEC_THREADS / 32 : warps);
+  dim3 grid(H, n);
+  delta_decode_kernel<T, RPL, CHAN><<<grid, warps * 32, smem, st>>>(
+      (const T*)proj, ld, x_off, b_off, (const T*)dec, dec_ld, (const T*)gate, gate_ld, conv_w, taps, (T*)ring, a_log, dt_bias, norm_w, eps,
+      sigmoid_gate, tok_slot, tok_pos, H, G, d, dv, dp, state, (T*)out);
+  return launch_status();
+}
+
+bool sizes_ok(int H, int G, int d, int dv, int taps) {
+  return H >= 1 && G >= 1 && H % G == 0 && H <= 32768 && d >= 1 && d <= 256 && dv >= 1 && dv <= 4096 && taps >= 1 && taps <= DRYFT_CONV_MAX_TAPS;
+}
+int rows_per_lane(int d) { return d <= 32 ? 1 : d <= 64 ? 2 : d <= 128 ? 4 : 8; }
+}  // namespace
+
+DRYFT_API int dryft_delta_prep(int is_bf16, int per_channel, const void* proj, int ld, int x_off, int b_off, const void* dec, int dec_ld,
+                               const float* conv_w, int taps, const void* ring, const float* a_log, const float* dt_bias,
+                               const int* tile_tok0, const int* tile_rows, int n_tiles, int tile_size, const int* cu_q, int n_seqs,
+                               const int* tok_slot, const int* tok_pos, int H, int G, int d, int dv, float* rec, float* vbuf,
+                               cudaStream_t st) {
+  if (n_tiles <= 0) return 0;
+  if (!sizes_ok(H, G, d, dv, taps) || tile_size % QUAD || (taps > 1 && ring == nullptr)) return DRYFT_ERR_UNSUPPORTED;
+  const int dp = (d + 3) / 4 * 4, dvp = (dv + WALK_COLS - 1) / WALK_COLS * WALK_COLS;
+#define DRYFT_PREP(T, DR, CH)                                                                                                       \
+  return prep_launch<T, DR, CH>(proj, ld, x_off, b_off, dec, dec_ld, conv_w, taps, ring, a_log, dt_bias, tile_tok0, tile_rows, n_tiles, \
+                                cu_q, n_seqs, tok_slot, tok_pos, H, G, d, dv, dp, dvp, rec, vbuf, st)
+#define DRYFT_PREP_R(T, CH)                  \
+  switch (rows_per_lane(d)) {                \
+    case 1: DRYFT_PREP(T, 1, CH);            \
+    case 2: DRYFT_PREP(T, 2, CH);            \
+    case 4: DRYFT_PREP(T, 4, CH);            \
+    default: DRYFT_PREP(T, 8, CH);           \
+  }
+  if (is_bf16) {
+    if (per_channel) { DRYFT_PREP_R(__nv_bfloat16, true) } else { DRYFT_PREP_R(__nv_bfloat16, false) }
+  } else {
+    if (per_channel) { DRYFT_PREP_R(float, true) } else { DRYFT_PREP_R(float, false) }
+  }
+#undef DRYFT_PREP_R
+#undef DRYFT_PREP
+}
+
+DRYFT_API int dryft_delta_walk(const float* rec, const float* vbuf, const int* cu_q, const int* seq_slot, int n_seqs, int H, int d, int dv,
+                               float* state, float* o, cudaStream_t st) {
+  if (n_seqs <= 0) return 0;
+  if (!sizes_ok(H, 1, d, dv, 1) || n_seqs > 65535) return DRYFT_ERR_UNSUPPORTED;
+  const int dp = (d + 3) / 4 * 4, dvp = (dv + WALK_COLS - 1) / WALK_COLS * WALK_COLS;
+  switch (rows_per_lane(d)) {
+    case 1: return walk_launch<1>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
+    case 2: return walk_launch<2>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
+    case 4: return walk_launch<4>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
+    default: return walk_launch<8>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
+  }
+}
+
+DRYFT_API int dryft_delta_norm(int is_bf16, const float* o, const void* gate, int gate_ld, const float* w, float eps, int sigmoid_gate,
+                               const int* tok_slot, void* out, int n, int H, int dv, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (H < 1 || dv < 1) return DRYFT_ERR_UNSUPPORTED;
+  const long long blocks = ((long long)n * H + NORM_WARPS - 1) / NORM_WARPS;
+  if (blocks > 0x7fffffffLL) return DRYFT_ERR_UNSUPPORTED;
+  typedef __nv_bfloat16 bf;
+  if (is_bf16)
+    delta_norm_kernel<bf><<<(unsigned)blocks, NORM_WARPS * 32, 0, st>>>(o, (const bf*)gate, gate_ld, w, eps, sigmoid_gate, tok_slot, (bf*)out, n, H, dv);
+  else
+    delta_norm_kernel<float><<<(unsigned)blocks, NORM_WARPS * 32, 0, st>>>(o, (const float*)gate, gate_ld, w, eps, sigmoid_gate, tok_slot, (float*)out, n, H, dv);
+  return launch_status();
+}
+
+DRYFT_API int dryft_delta_decode(int is_bf16, int per_channel, const void* proj, int ld, int x_off, int b_off, const void* dec, int dec_ld,
+                                 const void* gate, int gate_ld, const float* conv_w, int taps, void* ring, const float* a_log,
+                                 const float* dt_bias, const float* norm_w, float eps, int sigmoid_gate, const int* tok_slot,
+                                 const int* tok_pos, int n, int H, int G, int d, int dv, float* state, void* out, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (!sizes_ok(H, G, d, dv, taps) || n > 65535 || (taps > 1 && ring == nullptr)) return DRYFT_ERR_UNSUPPORTED;
+  const int dp = (d + 3) / 4 * 4;
+#define DRYFT_DEC(T, R, CH)                                                                                                          \
+  return decode_launch<T, R, CH>(proj, ld, x_off, b_off, dec, dec_ld, gate, gate_ld, conv_w, taps, ring, a_log, dt_bias, norm_w, eps, \
+                                 sigmoid_gate, tok_slot, tok_pos, n, H, G, d, dv, dp, state, out, st)
+#define DRYFT_DEC_R(T, CH)                  \
+  switch (rows_per_lane(d)) {               \
+    case 1: DRYFT_DEC(T, 1, CH);            \
+    case 2: DRYFT_DEC(T, 2, CH);            \
+    case 4: DRYFT_DEC(T, 4, CH);            \
+    default: DRYFT_DEC(T, 8, CH);           \
+  }
+  if (is_bf16) {
+    if (per_channel) { DRYFT_DEC_R(__nv_bfloat16, true) } else { DRYFT_DEC_R(__nv_bfloat16, false) }
+  } else {
+    if (per_channel) { DRYFT_DEC_R(float, true) } else { DRYFT_DEC_R(float, false) }
+  }
+#undef DRYFT_DEC_R
+#undef DRYFT_DEC
+}

@@ -5,12 +5,15 @@
 // for every block of P positions that lies wholly before the window (block b = positions bP .. bP + P - 1, seen when
 // bP + P - 1 <= i - size): the mean of the block's P cached keys and the mean of its P cached values, kept in pages of
 // their own, one row per block.  Tokens and blocks share one softmax, whose denominator also holds exp(sink_h), a
-// number per head without key or value.  Scores, weights and sums are 32-bit; q, k, v and the pooled rows have the
+// number per head without key or value.  `keep` > 0: the first `keep` tokens of the sequence stay visible whatever the window
+// (each key once; their cached rows are those of their true positions).  Scores, weights and sums are 32-bit; q, k, v and the pooled rows have the
 // activation type T.
 //
 //   pool_attn_prep    per token: q, k (+ bias) rotated over their first `rot` dims (dims i and i + rot/2 turn together by
 //                     the angle pos * inv_freq[i], evaluated in 32-bit), THEN divided by their root mean square over D
 //                     (no weight; skipped when eps < 0); v (+ bias); k and v written into the cache at the token's position.  One warp a vector.
+//                     With convolution weights (shortconv.cuh) q, k and v first pass a short causal convolution per channel
+//                     of [q | k | v], and a decode step stores its own projected values in the convolution's ring.
 //   pool_attn_prep_tok  the same per token for projections that are normed as a whole: q (all H * D values at once) and k (all
 //                     G * D) are divided by their root mean square and multiplied by a weight per entry BEFORE the rotation,
 //                     and the rotation pairs either dims i and i + rot/2 or (interleaved) dims 2i and 2i + 1.  One block a
@@ -23,7 +26,7 @@
 //                     joins there and the output is written, else partial (max, sum, weighted sum) go to memory and
 //   pool_attn_combine joins the splits and the sink.
 // Tokens with slot -1 (padding) are skipped.  No block waits on another block.
-#include "common.cuh"
+#include "shortconv.cuh"
 #include <math.h>
 
 #ifndef DRYFT_QK_DIM
@@ -55,7 +58,8 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
     const T* __restrict__ proj, int ld, const float* __restrict__ qb, const float* __restrict__ kb, const float* __restrict__ vb,
     const float* __restrict__ inv_freq, const float* __restrict__ inv_freq_lo, int rot, const int* __restrict__ tok_slot,
     const int* __restrict__ tok_pos, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, const int* __restrict__ page_table, int max_pages,
-    int page_size, int n_tokens, int H, int G, float eps, int write_kv) {
+    int page_size, int n_tokens, int H, int G, float eps, int write_kv, const float* __restrict__ conv_w, int taps, T* __restrict__ ring,
+    int store_ring) {
   __shared__ float sm[PREP_WARPS][D > DV ? D : DV];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int per_tok = H + (write_kv ? 2 * G : 0);
@@ -66,6 +70,16 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
   if (slot < 0) return;
   const int pos = tok_pos[t];
   const T* row = proj + (size_t)t * ld;
+  const int CH = H * D + G * (D + DV);
+  int back = 0;              // rows before this one that belong to its sequence and this step, as far as the convolution looks
+  if (conv_w != nullptr)
+    while (back < taps - 1 && t - back - 1 >= 0 && tok_slot[t - back - 1] == slot) ++back;
+  // channel c of [q | k | v]: the projected value, or the convolution over it
+  auto input = [&](int c) {
+    if (conv_w == nullptr) return to_f32<T>(row[c]);
+    if (store_ring) ring[((size_t)slot * taps + pos % taps) * CH + c] = row[c];
+    return conv1<T>(conv_w, proj, ld, ring, taps, CH, slot, t, pos, back, c);
+  };
   size_t cache_row = 0;
   if (vec >= H) {
     const int g = (vec - H) % G;
@@ -73,18 +87,17 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
     cache_row = ((size_t)page * G + g) * page_size + pos % page_size;
   }
   if (vec >= H + G) {     // a value vector: bias, cache
-    const int g = vec - H - G;
-    const T* src = row + (size_t)H * D + (size_t)G * D + (size_t)g * DV;
+    const int g = vec - H - G, src = H * D + G * D + g * DV;
     for (int c = lane; c < DV; c += 32)
-      v_pages[cache_row * DV + c] = from_f32<T>(to_f32<T>(src[c]) + (vb != nullptr ? vb[g * DV + c] : 0.f));
+      v_pages[cache_row * DV + c] = from_f32<T>(input(src + c) + (vb != nullptr ? vb[g * DV + c] : 0.f));
     return;
   }
   const bool is_q = vec < H;
   const int hd = is_q ? vec : vec - H;
-  const T* src = row + (is_q ? (size_t)hd * D : (size_t)H * D + (size_t)hd * D);
+  const int src = is_q ? hd * D : H * D + hd * D;
   const float* bias = is_q ? qb : kb;
   float* s = sm[warp];
-  for (int c = lane; c < D; c += 32) s[c] = to_f32<T>(src[c]) + (bias != nullptr ? bias[hd * D + c] : 0.f);
+  for (int c = lane; c < D; c += 32) s[c] = input(src + c) + (bias != nullptr ? bias[hd * D + c] : 0.f);
   __syncwarp();
   const int half = rot / 2;
   const float fpos = (float)pos;
@@ -257,7 +270,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
     const T* __restrict__ q, const T* __restrict__ k_pages, const T* __restrict__ v_pages, const int* __restrict__ page_table,
     int max_pages, int page_size, const T* __restrict__ pk_pages, const T* __restrict__ pv_pages, const int* __restrict__ pool_table,
     int pool_max_pages, const float* __restrict__ sink, const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
-    T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int G, int n_splits, float scale, int size, int P) {
+    T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int G, int n_splits, float scale, int size, int P, int keep) {
   __shared__ float qs[REP][D];
   __shared__ float wo[ROWS_WARPS][REP][DV];
   __shared__ float wml[ROWS_WARPS][REP][2];
@@ -269,7 +282,8 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
   const int i = tok_pos[t];
   const int lo = max(0, i - size + 1);
   const int nb = (P > 0 && i - size + 1 >= P) ? (i - size + 1) / P : 0;
-  const int nkeys = nb + (i - lo + 1);
+  const int nk = min(keep, lo);                   // kept tokens that the window has passed
+  const int nkeys = nb + nk + (i - lo + 1);
   int chunk = (nkeys + n_splits - 1) / n_splits;
   chunk = (chunk + 31) / 32 * 32;
   const int u0 = sp * chunk, u1 = min(nkeys, u0 + chunk);
@@ -296,7 +310,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
         kr = pk_pages + r * D;
         vr = pv_pages + r * DV;
       } else {
-        const int j = lo + (u - nb);
+        const int j = u - nb < nk ? u - nb : lo + (u - nb - nk);
         const int page = page_table[(size_t)slot * max_pages + j / page_size];
         const size_t r = ((size_t)page * G + g) * page_size + j % page_size;
         kr = k_pages + r * D;
@@ -405,13 +419,14 @@ __global__ void __launch_bounds__(128) pool_attn_combine_kernel(const float* __r
 template <typename T>
 int prep_launch(const void* proj, int ld, const float* qb, const float* kb, const float* vb, const float* inv_freq,
                 const float* inv_freq_lo, int rot, const int* tok_slot, const int* tok_pos, void* q_out, void* k_pages, void* v_pages, const int* page_table,
-                int max_pages, int page_size, int n, int H, int G, float eps, int write_kv, cudaStream_t st) {
+                int max_pages, int page_size, int n, int H, int G, float eps, int write_kv, const float* conv_w, int taps, void* ring,
+                int store_ring, cudaStream_t st) {
   const long long items = (long long)n * (H + (write_kv ? 2 * G : 0));
   const long long blocks = (items + PREP_WARPS - 1) / PREP_WARPS;
   if (blocks > 0x7fffffffLL) return DRYFT_ERR_UNSUPPORTED;
   pool_attn_prep_kernel<T><<<(unsigned)blocks, PREP_WARPS * 32, 0, st>>>(
       (const T*)proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, (T*)q_out, (T*)k_pages, (T*)v_pages, page_table, max_pages,
-      page_size, n, H, G, eps, write_kv);
+      page_size, n, H, G, eps, write_kv, conv_w, taps, (T*)ring, store_ring);
   return launch_status();
 }
 
@@ -419,11 +434,11 @@ template <typename T>
 int rows_launch(const void* q, const void* k_pages, const void* v_pages, const int* page_table, int max_pages, int page_size,
                 const void* pk, const void* pv, const int* pool_table, int pool_max_pages, const float* sink, const int* tok_slot,
                 const int* tok_pos, void* out, float* part_o, float* part_ml, int n, int G, int n_splits, float scale, int size, int P,
-                cudaStream_t st) {
+                int keep, cudaStream_t st) {
   dim3 grid(n, G, n_splits);
   pool_attn_rows_kernel<T><<<grid, ROWS_WARPS * 32, 0, st>>>((const T*)q, (const T*)k_pages, (const T*)v_pages, page_table, max_pages,
                                                             page_size, (const T*)pk, (const T*)pv, pool_table, pool_max_pages, sink,
-                                                            tok_slot, tok_pos, (T*)out, part_o, part_ml, G, n_splits, scale, size, P);
+                                                            tok_slot, tok_pos, (T*)out, part_o, part_ml, G, n_splits, scale, size, P, keep);
   int rc = launch_status();
   if (rc || n_splits == 1) return rc;
   dim3 cgrid(n, G * REP);
@@ -439,14 +454,16 @@ DRYFT_API int dryft_pool_attn_group() { return REP; }
 DRYFT_API int dryft_pool_attn_prep(int is_bf16, const void* proj, int ld, const float* qb, const float* kb, const float* vb,
                                    const float* inv_freq, const float* inv_freq_lo, int rot, const int* tok_slot, const int* tok_pos,
                                    void* q_out, void* k_pages, void* v_pages, const int* page_table, int max_pages, int page_size, int n, int H, int G, float eps,
-                                   int write_kv, cudaStream_t st) {
+                                   int write_kv, const float* conv_w, int taps, void* ring, int store_ring, cudaStream_t st) {
   if (n <= 0) return 0;
   if (H != G * REP || rot < 0 || rot % 2 || rot > D || (rot > 0 && inv_freq == nullptr) || (write_kv && page_size < 1))
     return DRYFT_ERR_UNSUPPORTED;
+  if (conv_w != nullptr && (taps < 1 || taps > DRYFT_CONV_MAX_TAPS || !write_kv || ((taps > 1 || store_ring) && ring == nullptr)))
+    return DRYFT_ERR_UNSUPPORTED;
   return is_bf16 ? prep_launch<__nv_bfloat16>(proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, q_out, k_pages, v_pages, page_table,
-                                              max_pages, page_size, n, H, G, eps, write_kv, st)
+                                              max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, st)
                  : prep_launch<float>(proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, q_out, k_pages, v_pages, page_table,
-                                      max_pages, page_size, n, H, G, eps, write_kv, st);
+                                      max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, st);
 }
 
 DRYFT_API int dryft_pool_attn_prep_tok(int is_bf16, const void* proj, int ld, const float* q_w, const float* k_w, float norm_eps,
@@ -487,14 +504,14 @@ DRYFT_API int dryft_pool_attn_blocks(int is_bf16, const void* k_pages, const voi
 DRYFT_API int dryft_pool_attn_rows(int is_bf16, const void* q, const void* k_pages, const void* v_pages, const int* page_table,
                                    int max_pages, int page_size, const void* pk, const void* pv, const int* pool_table,
                                    int pool_max_pages, const float* sink, const int* tok_slot, const int* tok_pos, void* out,
-                                   float* part_o, float* part_ml, int n, int G, int n_splits, float scale, int size, int P,
+                                   float* part_o, float* part_ml, int n, int G, int n_splits, float scale, int size, int P, int keep,
                                    cudaStream_t st) {
   if (n <= 0) return 0;
-  if (G < 1 || G > 65535 || n_splits < 1 || n_splits > 65535 || size < 1 || page_size < 1 || (P > 0 && pk == nullptr) ||
+  if (G < 1 || G > 65535 || n_splits < 1 || n_splits > 65535 || size < 1 || keep < 0 || page_size < 1 || (P > 0 && pk == nullptr) ||
       (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return DRYFT_ERR_UNSUPPORTED;
   return is_bf16 ? rows_launch<__nv_bfloat16>(q, k_pages, v_pages, page_table, max_pages, page_size, pk, pv, pool_table, pool_max_pages,
-                                              sink, tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, st)
+                                              sink, tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, st)
                  : rows_launch<float>(q, k_pages, v_pages, page_table, max_pages, page_size, pk, pv, pool_table, pool_max_pages, sink,
-                                      tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, st);
+                                      tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, st);
 }

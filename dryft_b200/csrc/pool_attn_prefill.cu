@@ -4,14 +4,15 @@
 // Grid (query tiles x query heads).  A tile is up to 64 consecutive query tokens of ONE sequence (tile_tok0 = first
 // packed token, tile_rows = how many).  The block's 4 warps own 16 query rows each.  The block walks one list of key
 // tiles of 64 rows: first the pages of POOLED rows (row b = the mean key and the mean value of positions bP .. bP+P-1)
-// up to the last block any row of the tile sees, then the token pages from the first position the tile's first row sees
+// up to the last block any row of the tile sees, then the pages of the sequence's first `keep` tokens that lie wholly before
+// the window's first page, then the token pages from the first position the tile's first row sees
 // to the tile's last position.  A tile is brought to shared memory with cp.async (two stages), so rows written by this
 // very step and by earlier steps are read the same way -- a prompt may be fed in portions.  Q K^T and P V run on
 // mma.sync.m16n8k16 (bf16 in, fp32 accumulate); scores, maxima, weights and sums are 32-bit, P is rounded to bfloat16 as
 // the second product's operand.  Value rows that no row of the tile may see (positions behind the tile's last, blocks
 // behind its last seen block) are filled with zeros on their way in: what a page's last holder left there is never
 // multiplied.
-// The query at position p sees the tokens j with 0 <= p - j < size and the blocks b with bP + P - 1 <= p - size
+// The query at position p sees the tokens j with 0 <= p - j < size or j < keep (j <= p) and the blocks b with bP + P - 1 <= p - size
 // (P = 0: no blocks).  The softmax's denominator also holds exp(sink_head): the running maximum starts at the sink and
 // the running sum at one (no sink: -inf and zero).
 //
@@ -93,7 +94,7 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     const int* __restrict__ tile_tok0, const int* __restrict__ tile_rows,
     const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     bf16* __restrict__ out,                                              // [N, nH * DV]
-    int nH, int nKV, float scale_log2, int size, int P) {
+    int nH, int nKV, float scale_log2, int size, int P, int keep) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);   // [BM][KS]
   bf16* ks = qs + BM * KS;                        // [2][BN][KS]
@@ -124,11 +125,13 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
   const int n_pool = (nb_tile + BN - 1) / BN;             // key tiles of pooled rows
   const int pg_first = max(0, pos0 - size + 1) / BN;      // the bound never decreases with the position
   const int pg_last = last_pos / BN;
-  const int n_tiles = n_pool + (pg_last - pg_first + 1);
+  const int n_kept = min(pg_first, (keep + BN - 1) / BN); // pages of kept tokens before the window's first page
+  const int n_tiles = n_pool + n_kept + (pg_last - pg_first + 1);
   const int* pt = page_table + (size_t)slot * max_pages;
   const int* ppt = pool_table + (size_t)slot * pool_max_pages;
 
-  // key tile `it` of the list: pooled page `it`, or token page pg_first + (it - n_pool)
+  // key tile `it` of the list: pooled page `it`, or a token page: the kept ones, then those of the window
+  auto token_page = [&](int it) { return it - n_pool < n_kept ? it - n_pool : pg_first + (it - n_pool - n_kept); };
   auto load_tile = [&](int it, int stage) {
     bf16* kd = ks + stage * BN * KS;
     bf16* vd = vs + stage * BN * VS;
@@ -136,7 +139,7 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
       const size_t pg = ((size_t)ppt[it] * nKV + kvh) * (size_t)BN;
       load_page(kd, vd, pk_pages + pg * KW, pv_pages + pg * DV, tid, it * BN, nb_tile);
     } else {
-      const int page = pg_first + (it - n_pool);
+      const int page = token_page(it);
       const size_t pg = ((size_t)pt[page] * nKV + kvh) * (size_t)BN;
       load_page(kd, vd, k_pages + pg * KW, v_pages + pg * DV, tid, page * BN, last_pos + 1);
     }
@@ -175,8 +178,9 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     const bf16* kst = ks + stage * BN * KS;
     const bf16* vst = vs + stage * BN * VS;
     const bool pooled = it < n_pool;
-    const int key0 = pooled ? it * BN : (pg_first + (it - n_pool)) * BN;   // first block, or first position, of the tile
-    // what each of the two rows sees of this tile: indices in [vlo, vhi)
+    const int key0 = pooled ? it * BN : token_page(it) * BN;   // first block, or first position, of the tile
+    // what each of the two rows sees of this tile: indices in [vlo, vhi), and below vkeep
+    const int vkeep = pooled ? 0 : keep;
     const int vlo0 = pooled ? 0 : lo0, vhi0 = pooled ? nb0 : qrow0 + 1;
     const int vlo1 = pooled ? 0 : lo1, vhi1 = pooled ? nb1 : qrow1 + 1;
 
@@ -205,7 +209,7 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int kp = key0 + j * 8 + 2 * t + (i & 1);
-        const bool vis = (i < 2) ? (kp >= vlo0 && kp < vhi0) : (kp >= vlo1 && kp < vhi1);
+        const bool vis = (i < 2) ? ((kp >= vlo0 || kp < vkeep) && kp < vhi0) : ((kp >= vlo1 || kp < vkeep) && kp < vhi1);
         const float v = vis ? s[j][i] * scale_log2 : -INFINITY;
         s[j][i] = v;
         if (i < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
@@ -283,9 +287,9 @@ DRYFT_API int dryft_pool_attn_prefill(const void* q, const void* k_pages, const 
                                       int page_size, const void* pk_pages, const void* pv_pages, const int* pool_table,
                                       int pool_max_pages, const float* sink, const int* tile_tok0, const int* tile_rows,
                                       const int* tok_slot, const int* tok_pos, void* out, int n_tiles, int nH, int nKV, float scale,
-                                      int size, int P, cudaStream_t st) {
+                                      int size, int P, int keep, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
-  if (nH != nKV * G || nH > 65535 || page_size != BN || size < 1 || P < 0) return DRYFT_ERR_UNSUPPORTED;
+  if (nH != nKV * G || nH > 65535 || page_size != BN || size < 1 || P < 0 || keep < 0) return DRYFT_ERR_UNSUPPORTED;
   if (P > 0 && (pk_pages == nullptr || pv_pages == nullptr || pool_table == nullptr)) return DRYFT_ERR_UNSUPPORTED;
   const size_t smem = smem_bytes();
   if (smem > 227 * 1024) return DRYFT_ERR_UNSUPPORTED;
@@ -300,6 +304,6 @@ DRYFT_API int dryft_pool_attn_prefill(const void* q, const void* k_pages, const 
   pool_attn_prefill_kernel<<<grid, THREADS, smem, st>>>((const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, page_table,
                                                        max_pages, (const bf16*)pk_pages, (const bf16*)pv_pages, pool_table,
                                                        pool_max_pages, sink, tile_tok0, tile_rows, tok_slot, tok_pos, (bf16*)out, nH,
-                                                       nKV, scale * 1.4426950408889634f, size, P);
+                                                       nKV, scale * 1.4426950408889634f, size, P, keep);
   return launch_status();
 }

@@ -6,6 +6,10 @@
 //                 and, when a norm weight is given, h[n] = T( x32[n] / sqrt(mean(x32[n]^2) + eps) * w ): the sum of a layer
 //                 and the norm of the next in one launch.  `src` (optional, 32-bit) replaces x32 as the sum's start
 //                 (x32[n] = src[n] + ...).
+//   stream_sum_ln the same sum of up to three terms, then up to two LAYER norms of the new row in the same launch:
+//                 h_i[n] = T( (x32[n] - mean) / sqrt(mean((x32[n] - mean)^2) + eps) * w_i + b_i ); the row stays in shared memory
+//                 (4 * width bytes), the mean is formed before the deviations are squared.  `rows` (optional): output row r
+//                 reads stream row rows[r] (no terms then: nothing is written to the stream).
 //   pack_pair     out[n] = T([a32[n] | b32[n]]): two 32-bit rows side by side as one operand row of a product
 //   softcap       z <- cap * tanh(z / cap) over 32-bit logits, in place
 //
@@ -49,6 +53,107 @@ __global__ void __launch_bounds__(THREADS) stream_sum_kernel(
   for (int c = threadIdx.x; c < width; c += THREADS) h[n * width + c] = from_f32<T>(x[c] * rinv * norm_w[c]);   // the thread's own writes
 }
 
+template <typename T> __device__ __forceinline__ float4 load4(const T* p);
+template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&raw.x), b = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
+  return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, float4 v);
+template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 raw;
+  raw.x = *reinterpret_cast<unsigned*>(&a);
+  raw.y = *reinterpret_cast<unsigned*>(&b);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
+
+// VEC 4 (widths that are a multiple of four) or 1
+template <typename T, int VEC>
+__global__ void __launch_bounds__(THREADS) stream_sum_ln_kernel(
+    float* __restrict__ x32, const int* __restrict__ rows, const T* __restrict__ y0, float s0, const T* __restrict__ y1, float s1,
+    const T* __restrict__ y2, float s2, const float* __restrict__ w0, const float* __restrict__ b0, T* __restrict__ h0,
+    const float* __restrict__ w1, const float* __restrict__ b1, T* __restrict__ h1, float eps, int width) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float scratch[33];
+  const size_t n = blockIdx.x;
+  float* x = x32 + (rows != nullptr ? (size_t)rows[n] : n) * width;
+  const bool adds = y0 != nullptr || y1 != nullptr || y2 != nullptr;
+  float sum = 0.f;
+  if (VEC == 4) {
+    for (int c = threadIdx.x * 4; c < width; c += THREADS * 4) {
+      float4 v = *reinterpret_cast<const float4*>(x + c);
+      auto term = [&](const T* y, float s) {
+        const float4 t = load4<T>(y + n * width + c);
+        v.x = fmaf(s, t.x, v.x); v.y = fmaf(s, t.y, v.y); v.z = fmaf(s, t.z, v.z); v.w = fmaf(s, t.w, v.w);
+      };
+      if (y0 != nullptr) term(y0, s0);
+      if (y1 != nullptr) term(y1, s1);
+      if (y2 != nullptr) term(y2, s2);
+      if (adds) *reinterpret_cast<float4*>(x + c) = v;
+      *reinterpret_cast<float4*>(row + c) = v;
+      sum += (v.x + v.y) + (v.z + v.w);
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += THREADS) {
+      float v = x[c];
+      if (y0 != nullptr) v = fmaf(s0, to_f32<T>(y0[n * width + c]), v);
+      if (y1 != nullptr) v = fmaf(s1, to_f32<T>(y1[n * width + c]), v);
+      if (y2 != nullptr) v = fmaf(s2, to_f32<T>(y2[n * width + c]), v);
+      if (adds) x[c] = v;
+      row[c] = v;
+      sum += v;
+    }
+  }
+  if (h0 == nullptr && h1 == nullptr) return;
+  const float mean = block_sum(sum, scratch) / (float)width;
+  float ss = 0.f;      // every thread reads the entries it wrote itself
+  if (VEC == 4) {
+    for (int c = threadIdx.x * 4; c < width; c += THREADS * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(row + c);
+      const float a = v.x - mean, b = v.y - mean, d = v.z - mean, e = v.w - mean;
+      ss = fmaf(a, a, fmaf(b, b, fmaf(d, d, fmaf(e, e, ss))));
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += THREADS) { const float d = row[c] - mean; ss = fmaf(d, d, ss); }
+  }
+  const float rinv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  if (VEC == 4) {
+    for (int c = threadIdx.x * 4; c < width; c += THREADS * 4) {
+      float4 v = *reinterpret_cast<const float4*>(row + c);
+      v.x = (v.x - mean) * rinv; v.y = (v.y - mean) * rinv; v.z = (v.z - mean) * rinv; v.w = (v.w - mean) * rinv;
+      auto out = [&](const float* w, const float* b, T* h) {
+        const float4 ww = *reinterpret_cast<const float4*>(w + c), bb = *reinterpret_cast<const float4*>(b + c);
+        store4<T>(h + n * width + c, make_float4(fmaf(v.x, ww.x, bb.x), fmaf(v.y, ww.y, bb.y), fmaf(v.z, ww.z, bb.z), fmaf(v.w, ww.w, bb.w)));
+      };
+      if (h0 != nullptr) out(w0, b0, h0);
+      if (h1 != nullptr) out(w1, b1, h1);
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += THREADS) {
+      const float v = (row[c] - mean) * rinv;
+      if (h0 != nullptr) h0[n * width + c] = from_f32<T>(fmaf(v, w0[c], b0[c]));
+      if (h1 != nullptr) h1[n * width + c] = from_f32<T>(fmaf(v, w1[c], b1[c]));
+    }
+  }
+}
+
+template <typename T, int VEC>
+int sum_ln_launch(float* x32, const int* rows, const void* y0, float s0, const void* y1, float s1, const void* y2, float s2, const float* w0,
+                  const float* b0, void* h0, const float* w1, const float* b1, void* h1, float eps, int n, int width, cudaStream_t st) {
+  const size_t smem = sizeof(float) * (size_t)width;
+  if (smem > 200 * 1024) return DRYFT_ERR_UNSUPPORTED;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(stream_sum_ln_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  stream_sum_ln_kernel<T, VEC><<<n, THREADS, smem, st>>>(x32, rows, (const T*)y0, s0, (const T*)y1, s1, (const T*)y2, s2, w0, b0, (T*)h0, w1, b1,
+                                                        (T*)h1, eps, width);
+  return launch_status();
+}
+
 template <typename T>
 __global__ void __launch_bounds__(THREADS) pack_pair_kernel(const float* __restrict__ a, const float* __restrict__ b,
                                                            T* __restrict__ out, int width) {
@@ -76,6 +181,21 @@ DRYFT_API int dryft_stream_sum(int is_bf16, float* x32, const float* src, const 
     stream_sum_kernel<float><<<n, THREADS, 0, st>>>(x32, src, (const float*)y0, s0, (const float*)y1, s1, (const float*)y2, s2,
                                                     (const float*)yr, top, sr, vec, norm_w, eps, (float*)h, width);
   return launch_status();
+}
+
+DRYFT_API int dryft_stream_sum_ln(int is_bf16, float* x32, const int* rows, const void* y0, float s0, const void* y1, float s1, const void* y2,
+                                  float s2, const float* w0, const float* b0, void* h0, const float* w1, const float* b1, void* h1, float eps,
+                                  int n, int width, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (width <= 0 || (rows != nullptr && (y0 != nullptr || y1 != nullptr || y2 != nullptr)) || (h0 != nullptr && (w0 == nullptr || b0 == nullptr)) ||
+      (h1 != nullptr && (w1 == nullptr || b1 == nullptr)))
+    return DRYFT_ERR_UNSUPPORTED;
+  const bool vec = width % 4 == 0;
+  if (is_bf16)
+    return vec ? sum_ln_launch<__nv_bfloat16, 4>(x32, rows, y0, s0, y1, s1, y2, s2, w0, b0, h0, w1, b1, h1, eps, n, width, st)
+               : sum_ln_launch<__nv_bfloat16, 1>(x32, rows, y0, s0, y1, s1, y2, s2, w0, b0, h0, w1, b1, h1, eps, n, width, st);
+  return vec ? sum_ln_launch<float, 4>(x32, rows, y0, s0, y1, s1, y2, s2, w0, b0, h0, w1, b1, h1, eps, n, width, st)
+             : sum_ln_launch<float, 1>(x32, rows, y0, s0, y1, s1, y2, s2, w0, b0, h0, w1, b1, h1, eps, n, width, st);
 }
 
 DRYFT_API int dryft_pack_pair(int is_bf16, const float* a, const float* b, void* out, int n, int width, cudaStream_t st) {

@@ -99,7 +99,15 @@ class DecoderModel:
             block = self.blocks[st.layer]
             if st.enter is not None:
                 res = self.joints[st.enter[0]].enter(res, x0, st.enter[1], getattr(block, "norm_mixer", None))
-            if getattr(block, "takes_next_norm", False):
+            if getattr(block, "takes_next_norms", False):
+                # both norms that read the stream next (an arrangement whose mixer and feed-forward read the same stream)
+                if i + 1 < len(sched):
+                    b = self.blocks[sched[i + 1].layer] if sched[i + 1].enter is None else None
+                    nxts = (getattr(b, "norm_mixer", None), getattr(b, "norm_ffn", None) if getattr(b, "takes_next_norms", False) else None)
+                else:
+                    nxts = (self.final_norm, None)
+                res = block.forward(res, ctx, cache.entry(i), cache.state(i), owns_cache=st.cache_from is None, next_norms=nxts)
+            elif getattr(block, "takes_next_norm", False):
                 # the norm that reads the stream next: the following run step's first norm, or the final norm -- unless a
                 # joint transforms the stream in between
                 if i + 1 < len(sched):

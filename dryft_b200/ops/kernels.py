@@ -1764,10 +1764,10 @@ def pool_attention_lib(qk_dim: int, v_dim: int, group: int) -> ctypes.CDLL:
                                        {"DRYFT_QK_DIM": qk_dim, "DRYFT_V_DIM": v_dim, "DRYFT_GROUP": group})
             lib = _load(path)
             lib.dryft_pool_attn_prep.argtypes = [_i, _p, _i, _p, _p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f,
-                                                 _i, _p]
+                                                 _i, _p, _i, _p, _i, _p]
             lib.dryft_pool_attn_blocks.argtypes = [_i, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _i, _i, _i, _p]
             lib.dryft_pool_attn_rows.argtypes = [_i, _p, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f,
-                                                 _i, _i, _p]
+                                                 _i, _i, _i, _p]
             lib.dryft_pool_attn_prep_tok.argtypes = [_i, _p, _i, _p, _p, _f, _p, _p, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i,
                                                      _f, _i, _p]
             for fn in ("dryft_pool_attn_prep", "dryft_pool_attn_prep_tok", "dryft_pool_attn_blocks", "dryft_pool_attn_rows"):
@@ -1797,7 +1797,7 @@ def pool_attention_prefill_lib(qk_dim: int, v_dim: int, group: int, page: int = 
                                        {"DRYFT_QK_DIM": qk_dim, "DRYFT_V_DIM": v_dim, "DRYFT_GROUP": group, "DRYFT_PAGE": page})
             lib = _load(path)
             lib.dryft_pool_attn_prefill.argtypes = [_p, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f,
-                                                    _i, _i, _p]
+                                                    _i, _i, _i, _p]
             lib.dryft_pool_attn_prefill.restype = _i
             if (lib.dryft_pool_attn_prefill_qk_dim(), lib.dryft_pool_attn_prefill_v_dim()) != (qk_dim, v_dim):
                 raise KernelError("pooled-window prompt attention: the library was built for another head shape")
@@ -1806,9 +1806,9 @@ def pool_attention_prefill_lib(qk_dim: int, v_dim: int, group: int, page: int = 
 
 
 def pool_attn_prefill(q, k_pages, v_pages, page_table, pooled, sink, tile_tok0, tile_rows, tok_slot, tok_pos, out, n_tiles: int,
-                      scale: float, size: int, pool: int) -> None:
+                      scale: float, size: int, pool: int, keep: int = 0) -> None:
     """Prompt attention (bfloat16) of ``q [n, H, D]``, tile by tile of up to 64 tokens of one sequence, over the last ``size``
-    cached tokens and the pooled rows of the blocks of ``pool`` positions wholly before them (``pooled = (pk_pages, pv_pages,
+    cached tokens, the sequence's first ``keep`` tokens and the pooled rows of the blocks of ``pool`` positions wholly before them (``pooled = (pk_pages, pv_pages,
     pool_table)``; ``pool = 0``: none); the softmax's denominator also holds ``exp(sink[head])`` (if given)."""
     n, n_heads, d = q.shape
     n_kv, page = k_pages.shape[1], k_pages.shape[2]
@@ -1830,13 +1830,14 @@ def pool_attn_prefill(q, k_pages, v_pages, page_table, pooled, sink, tile_tok0, 
     _ok(lib.dryft_pool_attn_prefill(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1], page, _ptr(pk),
                                     _ptr(pv), _ptr(pt), pt.shape[1] if pt is not None else 0, _ptr(sink), _ptr(tile_tok0),
                                     _ptr(tile_rows), _ptr(tok_slot), _ptr(tok_pos), _ptr(out), int(n_tiles), n_heads, n_kv,
-                                    float(scale), int(size), int(pool), _stream()),
+                                    float(scale), int(size), int(pool), int(keep), _stream()),
         f"pool_attn_prefill (window {size}, blocks of {pool})")
 
 
 def pool_attn_prep(proj, q_bias, k_bias, v_bias, inv_freq, inv_freq_lo, rot: int, tok_slot, tok_pos, q_out, k_pages, v_pages,
-                   page_table, n_heads: int, n_kv: int, eps: float, write_kv: bool) -> None:
-    """Per token of ``proj [n, H*D (+ G*D + G*DV)]``: bias, rotation of the first ``rot`` dims (rotate-half), division by the
+                   page_table, n_heads: int, n_kv: int, eps: float, write_kv: bool, conv_w=None, ring=None, store_ring: bool = False) -> None:
+    """Per token of ``proj [n, H*D (+ G*D + G*DV)]``: (with ``conv_w [H*D + G*(D+DV), taps]``: a short causal convolution per
+    channel, earlier steps' values from ``ring [slots, taps, channels]``; ``store_ring``: a decode step stores its own there), bias, rotation of the first ``rot`` dims (rotate-half), division by the
     root mean square over the head (no weight; ``eps < 0``: not divided) for q and k; v plus its bias; k and v into the cache
     pages."""
     n, ld = proj.shape
@@ -1855,11 +1856,19 @@ def pool_attn_prep(proj, q_bias, k_bias, v_bias, inv_freq, inv_freq_lo, rot: int
         _need(inv_freq, "inv_freq", torch.float32, (rot // 2,))
         if inv_freq_lo is not None:
             _need(inv_freq_lo, "inv_freq_lo", torch.float32, (rot // 2,))
+    taps = 0
+    if conv_w is not None:
+        ch = n_heads * d + n_kv * (d + dv)
+        _need(conv_w, "conv_w", torch.float32, (ch, None))
+        taps = conv_w.shape[1]
+        if taps > 1:
+            _need(ring, "ring", proj.dtype, (None, taps, ch))
     lib = pool_attention_lib(d, dv, n_heads // n_kv)
     _ok(lib.dryft_pool_attn_prep(_act(proj, "proj"), _ptr(proj), ld, _ptr(q_bias), _ptr(k_bias), _ptr(v_bias), _ptr(inv_freq),
                                  _ptr(inv_freq_lo), int(rot), _ptr(tok_slot), _ptr(tok_pos), _ptr(q_out), _ptr(k_pages), _ptr(v_pages),
                                  _ptr(page_table), page_table.shape[1], k_pages.shape[2], n, n_heads, n_kv, float(eps),
-                                 int(write_kv), _stream()), f"pool_attn_prep ({n_heads}/{n_kv} heads of {d})")
+                                 int(write_kv), _ptr(conv_w), taps, _ptr(ring if taps > 1 else None), int(store_ring and taps > 1),
+                                 _stream()), f"pool_attn_prep ({n_heads}/{n_kv} heads of {d})")
 
 
 def pool_attn_prep_tok(proj, q_norm_w, k_norm_w, norm_eps: float, inv_freq, inv_freq_lo, rot: int, interleaved: bool, tok_slot, tok_pos,
@@ -1910,8 +1919,8 @@ def pool_attn_blocks(k_pages, v_pages, page_table, pk_pages, pv_pages, pool_tabl
 
 
 def pool_attn_rows(q, k_pages, v_pages, page_table, pooled, sink, tok_slot, tok_pos, out, scale: float, size: int, pool: int,
-                   n_splits: int = 1, part_o=None, part_ml=None) -> None:
-    """Row-wise attention of ``q [n, H, D]`` over the last ``size`` cached tokens and, beside them, the pooled row of every block
+                   n_splits: int = 1, part_o=None, part_ml=None, keep: int = 0) -> None:
+    """Row-wise attention of ``q [n, H, D]`` over the last ``size`` cached tokens, the sequence's first ``keep`` tokens and, beside them, the pooled row of every block
     of ``pool`` positions that lies wholly before them (``pooled = (pk_pages, pv_pages, pool_table)``; ``pool = 0``: none), one
     softmax whose denominator also holds ``exp(sink[head])`` (if given).  ``out [n, H, DV]``."""
     n, n_heads, d = q.shape
@@ -1936,7 +1945,7 @@ def pool_attn_rows(q, k_pages, v_pages, page_table, pooled, sink, tok_slot, tok_
     _ok(lib.dryft_pool_attn_rows(_act(q, "q"), _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1], page,
                                  _ptr(pk), _ptr(pv), _ptr(pt), pt.shape[1] if pt is not None else 0, _ptr(sink), _ptr(tok_slot),
                                  _ptr(tok_pos), _ptr(out), _ptr(part_o), _ptr(part_ml), n, n_kv, int(n_splits), float(scale), int(size),
-                                 int(pool), _stream()), f"pool_attn_rows (window {size}, blocks of {pool})",
+                                 int(pool), int(keep), _stream()), f"pool_attn_rows (window {size}, blocks of {pool})",
         n_kernels=2 if n_splits > 1 else 1)
 
 
@@ -1944,6 +1953,7 @@ def pool_attn_rows(q, k_pages, v_pages, page_table, pooled, sink, tok_slot, tok_
 def stream_par_lib() -> ctypes.CDLL:
     return _single_lib("stream_par", {
         "dryft_stream_sum": [_i, _p, _p, _p, _f, _p, _f, _p, _f, _p, _i, _f, _p, _p, _f, _p, _i, _i, _p],
+        "dryft_stream_sum_ln": [_i, _p, _p, _p, _f, _p, _f, _p, _f, _p, _p, _p, _p, _p, _p, _f, _i, _i, _p],
         "dryft_pack_pair": [_i, _p, _p, _p, _i, _i, _p],
         "dryft_softcap": [_p, _ll, _f, _p],
     })
@@ -1989,6 +1999,39 @@ def stream_sum(x32, terms=(), *, rows=None, top: int = 0, rows_scale: float = 1.
                                           _ptr(terms[1][0]), terms[1][1], _ptr(terms[2][0]), terms[2][1], _ptr(rows), int(top),
                                           float(rows_scale), _ptr(vec), _ptr(norm_w), float(eps), _ptr(h if norm_w is not None else None),
                                           n, width, _stream()), "stream_sum")
+
+
+def stream_sum_ln(x32, terms=(), *, norms=(), eps: float = 0.0, rows=None, n_rows: Optional[int] = None) -> None:
+    """``x32[n] += sum_i scale_i * y_i[n]`` in 32-bit for up to three ``terms`` ``(y_i, scale_i)`` of the activation type, and up to two
+    layer norms of the new rows: ``norms`` lists ``(weight, bias, out)`` (``out [n, width]`` of the activation type).  ``rows``
+    (int32): output row ``r`` reads stream row ``rows[r]``; there are no terms then and the stream stays as it is."""
+    width = x32.shape[1]
+    n = x32.shape[0] if rows is None else (n_rows if n_rows is not None else rows.numel())
+    _need(x32, "x32", torch.float32)
+    terms = [(y, float(sc)) for y, sc in terms if y is not None]
+    norms = [nm for nm in norms if nm is not None]
+    if len(terms) > 3 or len(norms) > 2 or (rows is not None and terms):
+        raise KernelError("stream_sum_ln: at most three terms (none with gathered rows) and two norms")
+    act = None
+    for y, _ in terms:
+        _need(y, "term", act, (n, width))
+        act = y.dtype
+    for w, b, out in norms:
+        _need(w, "norm weight", torch.float32, (width,))
+        _need(b, "norm bias", torch.float32, (width,))
+        _need(out, "norm result", act, (n, width))
+        act = out.dtype
+    if rows is not None:
+        _need(rows, "rows", torch.int32)
+        if rows.numel() < n:
+            raise KernelError(f"stream_sum_ln: {n} rows asked for, {rows.numel()} named")
+    if act not in (None, torch.float32, torch.bfloat16):
+        raise KernelError(f"stream_sum_ln: terms are float32 or bfloat16, got {act}")
+    terms += [(None, 0.0)] * (3 - len(terms))
+    (w0, b0, h0), (w1, b1, h1) = (list(norms) + [(None, None, None)] * 2)[:2]
+    _ok(stream_par_lib().dryft_stream_sum_ln(int(act == torch.bfloat16), _ptr(x32), _ptr(rows), _ptr(terms[0][0]), terms[0][1], _ptr(terms[1][0]),
+                                             terms[1][1], _ptr(terms[2][0]), terms[2][1], _ptr(w0), _ptr(b0), _ptr(h0), _ptr(w1), _ptr(b1), _ptr(h1),
+                                             float(eps), n, width, _stream()), "stream_sum_ln")
 
 
 def pack_pair(a32, b32, out) -> None:
@@ -2050,3 +2093,111 @@ def selscan(xc, low, b_off: int, c_off: int, dtp, dt_bias, a_log, d_skip, zrows,
                                     _ptr(a_log), _ptr(d_skip), _ptr(zrows), zrows.shape[1], int(z_off), _ptr(cu_q), _ptr(seq_slot),
                                     int(n_seqs), cht, n_chunks, inner, n_state, _ptr(state), _ptr(cstate), _ptr(cdt), _ptr(out), _stream()),
         f"selscan ({inner} channels, state {n_state})", n_kernels=3 if chunked else 1)
+
+
+# ----------------------------------------------------------------------------- short convolutions with a ring memory
+CONV_MAX_TAPS = 16
+
+
+def shortconv_lib() -> ctypes.CDLL:
+    return _single_lib("shortconv", {"dryft_conv_ring_store": [_i, _p, _i, _p, _p, _p, _p, _i, _i, _i, _p]})
+
+
+def conv_ring_store(proj, col: int, cu_q, seq_slot, tok_pos, ring, n_seqs: int) -> None:
+    """After a step of many tokens: the projected values (``proj`` columns ``col ..``) of each sequence's last ``taps - 1`` tokens
+    go to row ``position % taps`` of its slot's ``ring [slots, taps, channels]``."""
+    n, ld = proj.shape
+    _need(proj, "proj")
+    _need(ring, "ring", proj.dtype, (None, None, None))
+    taps, ch = ring.shape[1], ring.shape[2]
+    if col < 0 or col + ch > ld:
+        raise KernelError(f"conv_ring_store: {ch} channels from column {col} of a row of {ld}")
+    x = ctypes.c_void_p(proj.data_ptr() + col * proj.element_size())
+    _ok(shortconv_lib().dryft_conv_ring_store(_act(proj, "proj"), x, ld, _ptr(cu_q), _ptr(seq_slot), _ptr(tok_pos), _ptr(ring), taps, ch,
+                                              int(n_seqs), _stream()), f"conv_ring_store ({ch} channels, {taps} taps)")
+
+
+# ----------------------------------------------------------------------------- gated delta rule
+DELTA_MAX_DIM = 256
+DELTA_COLS = 16      # value columns a block of the walk takes
+
+
+def delta_lib() -> ctypes.CDLL:
+    return _single_lib("delta", {
+        "dryft_delta_prep": [_i, _i, _p, _i, _i, _i, _p, _i, _p, _i, _p, _p, _p, _p, _p, _i, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _p],
+        "dryft_delta_walk": [_p, _p, _p, _p, _i, _i, _i, _i, _p, _p, _p],
+        "dryft_delta_norm": [_i, _p, _p, _i, _p, _f, _i, _p, _p, _i, _i, _i, _p],
+        "dryft_delta_decode": [_i, _i, _p, _i, _i, _i, _p, _i, _p, _i, _p, _i, _p, _p, _p, _p, _f, _i, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p],
+    })
+
+
+def delta_state_rows(dim: int) -> int:
+    """Floats a value column of the state takes: the key size rounded up to whole 16-byte pieces."""
+    return (dim + 3) // 4 * 4
+
+
+def _rows_of(t, name: str, dtype, n: int, cols: int):
+    """A column slice of a row-major matrix (or a whole one): pointer and row stride."""
+    if not isinstance(t, torch.Tensor) or not t.is_cuda or t.dtype != dtype or t.dim() != 2 or t.shape[0] != n or t.shape[1] < cols or t.stride(1) != 1:
+        raise KernelError(f"{name}: expected {n} rows of at least {cols} {dtype} values on the device")
+    return ctypes.c_void_p(t.data_ptr()), t.stride(0)
+
+
+def _delta_common(proj, x_off, b_off, dec, conv_w, ring, a_log, dt_bias, heads, kv_heads, dim, vdim, per_channel):
+    n, ld = proj.shape
+    _need(proj, "proj")
+    ch = 2 * kv_heads * dim + heads * vdim
+    if x_off < 0 or x_off + ch > ld or b_off < 0 or b_off + heads > ld:
+        raise KernelError(f"delta rule: {ch} channels from column {x_off}, {heads} logits from column {b_off} of a row of {ld}")
+    _need(conv_w, "conv_w", torch.float32, (ch, None))
+    taps = conv_w.shape[1]
+    if taps > 1:
+        _need(ring, "ring", proj.dtype, (None, taps, ch))
+    count = heads * dim if per_channel else heads
+    _need(a_log, "a_log", torch.float32, (heads,))
+    _need(dt_bias, "dt_bias", torch.float32, (count,))
+    dec_ptr, dec_ld = _rows_of(dec, "dec", proj.dtype, n, count)
+    return n, ld, taps, dec_ptr, dec_ld
+
+
+def delta_tokens(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, dt_bias, norm_w, eps: float, sigmoid_gate: bool, ctx, state,
+                 out, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool) -> None:
+    """The gated delta rule over a step of many tokens (``csrc/delta.cu``): records of four tokens each, the walk over them from
+    each slot's ``state [slots, H, DV, dp]``, then norm and gate into ``out [n, H*DV]``.  ``ctx``: the step's context (its
+    tiles say which tokens belong together).  Three launches; the convolution's ring is not advanced (``conv_ring_store``)."""
+    n, ld, taps, dec_ptr, dec_ld = _delta_common(proj, x_off, b_off, dec, conv_w, ring, a_log, dt_bias, heads, kv_heads, dim, vdim, per_channel)
+    dp, dvp = delta_state_rows(dim), (vdim + DELTA_COLS - 1) // DELTA_COLS * DELTA_COLS
+    _need(state, "state", torch.float32, (None, heads, vdim, dp))
+    _need(norm_w, "norm_w", torch.float32, (vdim,))
+    _need(out, "out", proj.dtype, (n, heads * vdim))
+    gate_ptr, gate_ld = _rows_of(gate, "gate", proj.dtype, n, heads * vdim)
+    if ctx.tile_size % 4:
+        raise KernelError(f"delta rule: prompt tiles of {ctx.tile_size} tokens (a multiple of 4 is needed)")
+    rec = torch.empty(((n + 3 * ctx.n_seqs) // 4 + 1, heads, 13 * dp + 28), dtype=torch.float32, device=proj.device)
+    vbuf = torch.empty((n, heads, dvp), dtype=torch.float32, device=proj.device)
+    o = torch.empty((n, heads * vdim), dtype=torch.float32, device=proj.device)
+    lib, bf = delta_lib(), _act(proj, "proj")
+    what = f"delta rule ({heads}/{kv_heads} heads of {dim} x {vdim}, {taps} taps)"
+    _ok(lib.dryft_delta_prep(bf, int(per_channel), _ptr(proj), ld, int(x_off), int(b_off), dec_ptr, dec_ld, _ptr(conv_w), taps,
+                             _ptr(ring if taps > 1 else None), _ptr(a_log), _ptr(dt_bias), _ptr(ctx.tile_tok0), _ptr(ctx.tile_rows),
+                             int(ctx.n_tiles), int(ctx.tile_size), _ptr(ctx.cu_q), int(ctx.n_seqs), _ptr(ctx.tok_slot), _ptr(ctx.tok_pos),
+                             heads, kv_heads, dim, vdim, _ptr(rec), _ptr(vbuf), _stream()), what)
+    _ok(lib.dryft_delta_walk(_ptr(rec), _ptr(vbuf), _ptr(ctx.cu_q), _ptr(ctx.seq_slot), int(ctx.n_seqs), heads, dim, vdim, _ptr(state),
+                             _ptr(o), _stream()), what)
+    _ok(lib.dryft_delta_norm(bf, _ptr(o), gate_ptr, gate_ld, _ptr(norm_w), float(eps), int(sigmoid_gate), _ptr(ctx.tok_slot), _ptr(out), n,
+                             heads, vdim, _stream()), what)
+
+
+def delta_decode(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, dt_bias, norm_w, eps: float, sigmoid_gate: bool, tok_slot,
+                 tok_pos, state, out, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool) -> None:
+    """The gated delta rule for one token per sequence, all of it (convolution, state, read-out, norm, gate, the ring's new row)
+    in one launch."""
+    n, ld, taps, dec_ptr, dec_ld = _delta_common(proj, x_off, b_off, dec, conv_w, ring, a_log, dt_bias, heads, kv_heads, dim, vdim, per_channel)
+    _need(state, "state", torch.float32, (None, heads, vdim, delta_state_rows(dim)))
+    _need(norm_w, "norm_w", torch.float32, (vdim,))
+    _need(out, "out", proj.dtype, (n, heads * vdim))
+    gate_ptr, gate_ld = _rows_of(gate, "gate", proj.dtype, n, heads * vdim)
+    _ok(delta_lib().dryft_delta_decode(_act(proj, "proj"), int(per_channel), _ptr(proj), ld, int(x_off), int(b_off), dec_ptr, dec_ld, gate_ptr,
+                                       gate_ld, _ptr(conv_w), taps, _ptr(ring if taps > 1 else None), _ptr(a_log), _ptr(dt_bias),
+                                       _ptr(norm_w), float(eps), int(sigmoid_gate), _ptr(tok_slot), _ptr(tok_pos), n, heads, kv_heads, dim,
+                                       vdim, _ptr(state), _ptr(out), _stream()), f"delta_decode ({heads}/{kv_heads} heads of {dim} x {vdim})")

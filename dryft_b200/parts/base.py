@@ -39,13 +39,16 @@ class TensorInfo(NamedTuple):
     """One checkpoint tensor a part expects.  ``kind``: "matrix" (a product's weight), "vector"
     (norm weights and other small tensors, kept in 32-bit on the device) or "table" (embedding).  ``mean``: what random
     weights of this tensor are drawn around (default: 1 for vectors, 0 for everything else).  ``eye``: random weights of a
-    square tensor are drawn around ``eye`` times the identity (a mixing matrix that starts near "every stream keeps itself")."""
+    square tensor are drawn around ``eye`` times the identity (a mixing matrix that starts near "every stream keeps itself").
+    ``free``: dimensions the configuration does not give (the rank of a low-rank map): the checkpoint's tensor decides, and the
+    number in ``shape`` is what random weights use; a part asks ``weights.shape(name)``."""
 
     shape: Tuple[int, ...]
     kind: str
     optional: bool = False
     mean: Optional[float] = None
     eye: float = 0.0
+    free: Tuple[int, ...] = ()
 
 
 @dataclass
@@ -144,9 +147,12 @@ class Residual:
     conn: Optional[Any] = None
     closer: Optional[Any] = None
     # ``x`` already normed by ``hn_norm`` (in the activation type): left by the kernel that formed ``x`` for the layer
-    # whose first norm that is, which then skips its own norm launch
+    # whose first norm that is, which then skips its own norm launch; ``hn2`` / ``hn2_norm``: the same for the norm in front of
+    # that layer's feed-forward where both read the same ``x``
     hn: Optional[torch.Tensor] = None
     hn_norm: Optional[Any] = None
+    hn2: Optional[torch.Tensor] = None
+    hn2_norm: Optional[Any] = None
 
 
 def fused_rms(norm) -> Optional[Tuple[torch.Tensor, float]]:

@@ -280,6 +280,82 @@ class ParallelBlock:
         return Residual(x, hn=hn, hn_norm=next_norm if hn is not None else None)
 
 
+@register_connection("scaled_sum")
+class ScaledSum:
+    """A constant ``mult`` that the sublayers' results take on their way into the stream: ``x + mult * y``."""
+
+    @staticmethod
+    def tensors(params: Mapping, prefix: str) -> Dict[str, TensorInfo]:
+        return {}
+
+    def __init__(self, params: Mapping, prefix: str, weights, rt: Runtime):
+        self.mult = float(params.get("mult", 1.0))
+
+
+@register_block("parallel_norms")
+class ParallelNormsBlock:
+    """Mixer and feed-forward side by side, each behind a layer norm of its own of the same 32-bit stream:
+
+        x <- x + mult * (mixer(norm_mixer(x)) + ffn(norm_ffn(x)))
+
+    ``extra["sum"]`` (a ``scaled_sum``) gives ``mult`` (1 without it).  The norms must offer ``layer_params``; both read the same
+    row, so the kernel that forms a layer's sum leaves the row normed twice, for the mixer and for the feed-forward of the
+    layer that runs next (``csrc/stream_par.cu:stream_sum_ln``): a layer is two norm-less chains of products and one sum.  A mixer that
+    offers ``forward_terms`` hands over its results unsummed; in a step of few rows the feed-forward runs beside the mixer on a
+    stream of its own.  A layer without a feed-forward has no second norm."""
+
+    takes_next_norms = True     # forward accepts (the norm before the next mixer, the norm before the next feed-forward or None)
+
+    def __init__(self, norm_mixer, mixer, norm_ffn, ffn, extra: Optional[Mapping] = None):
+        for nm in (norm_mixer, norm_ffn):
+            if nm is not None and not hasattr(nm, "layer_params"):
+                raise ValueError("the 'parallel_norms' arrangement needs norms that offer layer_params")
+        if (ffn is None) != (norm_ffn is None):
+            raise ValueError("the 'parallel_norms' arrangement: a feed-forward and its norm go together (one of them is missing)")
+        self.norm_mixer, self.mixer, self.norm_ffn, self.ffn = norm_mixer, mixer, norm_ffn, ffn
+        self.extra = dict(extra or {})
+        self.mult = float(self.extra["sum"].mult) if "sum" in self.extra else 1.0
+        K.stream_par_lib()
+
+    @staticmethod
+    def _sum_and_norms(x: torch.Tensor, terms, norms, dtype) -> list:
+        """``x`` plus the terms, in place, and the norms of the result (None for a norm that is None or of another kind)."""
+        params = [nm.layer_params() if nm is not None and hasattr(nm, "layer_params") else None for nm in norms]
+        eps = next((p[2] for p in params if p is not None), 0.0)
+        outs = [torch.empty(x.shape, dtype=dtype, device=x.device) if p is not None and p[2] == eps else None for p in params]
+        K.stream_sum_ln(x, terms, norms=[(p[0], p[1], o) for p, o in zip(params, outs) if o is not None], eps=eps)
+        return outs
+
+    def forward(self, res: Residual, ctx: StepContext, cache, state, owns_cache: bool = True, next_norms=(None, None)) -> Residual:
+        x, rt = res.x, self.mixer.rt
+        if x.dtype != torch.float32:
+            raise ValueError("the 'parallel_norms' arrangement keeps its stream in float32; the embedding must start one")
+        if res.delta is not None:
+            x.add_(res.delta)
+        hm = res.hn if (res.hn is not None and res.hn_norm is self.norm_mixer) else None
+        hf = res.hn2 if (res.hn2 is not None and res.hn2_norm is self.norm_ffn) else None
+        if hm is None or (self.ffn is not None and hf is None):
+            hm, hf = self._sum_and_norms(x, (), (self.norm_mixer, self.norm_ffn), rt.dtype)
+            if self.ffn is not None and hf is None:      # another eps than the mixer's norm: a launch of its own
+                hf = self.norm_ffn.forward(x)
+
+        def mix():
+            terms = getattr(self.mixer, "forward_terms", None)
+            return list(terms(hm, ctx, cache, state, owns_cache)) if terms is not None else [(self.mixer.forward(hm, ctx, cache, state, owns_cache), 1.0)]
+
+        def feed():
+            return [(self.ffn.forward(hf, ctx), 1.0)]
+
+        if self.ffn is None:
+            terms = mix()
+        else:
+            a, f = rt.run_branches([mix, feed], first_stream=0) if rt.branches(x.shape[0]) else (mix(), feed())
+            terms = a + f
+        outs = self._sum_and_norms(x, [(y, s * self.mult) for y, s in terms], next_norms, rt.dtype)
+        return Residual(x, hn=outs[0], hn_norm=next_norms[0] if outs[0] is not None else None,
+                        hn2=outs[1], hn2_norm=next_norms[1] if outs[1] is not None else None)
+
+
 @register_connection("loop_mix")
 class LoopMix:
     """How a stretch of layers that runs several times is entered: ``x <- W [x | x0] + step[t]`` with ``x0`` the embedding's

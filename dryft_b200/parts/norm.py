@@ -114,3 +114,43 @@ class OffsetRMSNorm:
         K.gated_postnorm(y, x32, self._factor, keep, self.eps, h, gate=gate, gate_b=gate_bias, wts=wts, top=top, shared=shared,
                          shared_gate=shared_gate)
         return x32 if h is None else h
+
+
+@register_norm("layernorm")
+class LayerNorm:
+    """``(x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b`` of a 32-bit stream, all of it in 32-bit and rounded once
+    (``csrc/stream_par.cu``).  ``layer_params`` declares that arithmetic: an arrangement whose sum kernel has the row in hand
+    forms this norm, and a second one of the same row, on the side.  ``params``: ``size``, ``eps``, ``name`` (default
+    ``weight``) and ``bias`` (default ``bias``), the tensors' names behind the prefix."""
+
+    @staticmethod
+    def tensors(params: Mapping, prefix: str) -> Dict[str, TensorInfo]:
+        return {prefix + params.get("name", "weight"): TensorInfo((params["size"],), "vector"),
+                prefix + params.get("bias", "bias"): TensorInfo((params["size"],), "vector", False, 0.0)}
+
+    def __init__(self, params: Mapping, prefix: str, weights, rt: Runtime):
+        self.size = int(params["size"])
+        self.eps = float(params["eps"])
+        self.rt = rt
+        self.weight = weights.load(prefix + params.get("name", "weight"), "vector")  # float32 [size]
+        self.bias = weights.load(prefix + params.get("bias", "bias"), "vector")
+        K.stream_par_lib()
+
+    def layer_params(self):
+        return self.weight, self.bias, self.eps
+
+    def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None) -> torch.Tensor:
+        n = n_rows if n_rows is not None else (rows.numel() if rows is not None else x.shape[0])
+        out = torch.empty((n, self.size), dtype=self.rt.dtype, device=x.device)
+        K.stream_sum_ln(x if x.dtype == torch.float32 else x.to(torch.float32), norms=[(self.weight, self.bias, out)], eps=self.eps, rows=rows,
+                        n_rows=n)
+        return out
+
+    def add_forward(self, x: torch.Tensor, delta: torch.Tensor, rows: Optional[torch.Tensor] = None,
+                    n_rows: Optional[int] = None) -> torch.Tensor:
+        """``x += delta`` (in place, whatever ``rows`` says) and the norm of the sum: the pre-norm arrangement's use."""
+        if x.dtype == torch.float32:
+            x.add_(delta)
+        else:
+            K.residual_add(x, delta)
+        return self.forward(x, rows, n_rows)

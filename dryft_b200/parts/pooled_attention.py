@@ -16,6 +16,12 @@ Per step, with ``h`` the mixer's input:
           riding in the input product)
     out = W_o (heads concatenated)
 
+``keep_first``: with a ``window``, the sequence's first ``keep_first`` tokens stay visible to every later query (each once, with
+their true positions).  ``conv_taps``: q, k and v pass a short causal convolution per channel right behind the projection
+(weights ``q_conv`` .. ``[channels, taps]``, no bias, zeros before the sequence's start); its last ``taps - 1`` inputs are
+per-sequence state.  ``value_gate``: the concatenated heads are multiplied element by element by ``sigmoid(W_g h)``, ``W_g
+[heads * v_dim, hidden]`` riding in the input product.
+
 ``proj_norm``: q and k pass an RMS norm over the WHOLE projection (all heads' rows at once, weights ``q_norm [heads * qk_dim]``
 and ``k_norm [kv_heads * qk_dim]``, ``eps`` inside the root) before the rotation.  The rotation's layout is the position
 part's (``half``: dims ``i`` and ``i + R/2``; ``interleaved``: dims ``2i`` and ``2i + 1``).
@@ -42,7 +48,7 @@ from .linear import linear
 
 _ROLES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight", "q_bias": "q_proj.bias",
           "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "sink": "sink", "q_norm": "q_norm.weight", "k_norm": "k_norm.weight",
-          "gate": "g_proj.weight"}
+          "gate": "g_proj.weight", "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight"}
 NO_WINDOW = 1 << 30   # "every earlier token" as a window size
 
 
@@ -76,6 +82,12 @@ class PooledWindowAttention:
                 t[nm["k_norm"]] = TensorInfo((nkv * d,), "vector")
         if params.get("head_gate", False):
             t[nm["gate"]] = TensorInfo((nh, w), "matrix")
+        if params.get("value_gate", False):
+            t[nm["gate"]] = TensorInfo((nh * dv, w), "matrix")
+        taps = params.get("conv_taps")
+        if taps:
+            for role, ch in (("q_conv", nh * d), ("k_conv", nkv * d), ("v_conv", nkv * dv)):
+                t[nm[role]] = TensorInfo((ch, int(taps)), "vector", False, 1.0 / int(taps))
         return t
 
     def __init__(self, params: Mapping, prefix: str, weights, rt: Runtime):
@@ -96,6 +108,14 @@ class PooledWindowAttention:
         self.q_dim, self.o_dim = self.n_heads * self.qk_dim, self.n_heads * self.v_dim
         nm = _names(params, prefix)
         self.head_gate = bool(params.get("head_gate", False))
+        self.value_gate = bool(params.get("value_gate", False))
+        if self.head_gate and self.value_gate:
+            raise ValueError("pooled_window_attention: a gate per head or a gate per value, not both")
+        self.keep = int(params.get("keep_first", 0) or 0) if win is not None else 0
+        self.taps = int(params.get("conv_taps") or 0)
+        if self.keep < 0 or not 0 <= self.taps <= K.CONV_MAX_TAPS or (self.taps and not self.own_kv):
+            raise ValueError(f"pooled_window_attention: {self.keep} kept tokens, {self.taps} taps (at most {K.CONV_MAX_TAPS}; a layer that "
+                             "reads another's keys and values has no convolution)")
         names, rows = [nm["q"]], [self.q_dim]
         if self.own_kv:
             names += [nm["k"], nm["v"]]
@@ -104,11 +124,18 @@ class PooledWindowAttention:
         if self.head_gate:                 # the gate's logits are columns of the input product
             names.append(nm["gate"])
             rows.append(self.n_heads)
+        elif self.value_gate:
+            names.append(nm["gate"])
+            rows.append(self.o_dim)
         self.w_in = weights.load_fused(names, rows, self.hidden) if len(names) > 1 else weights.load(nm["q"], "matrix")
         self.proj_norm = bool(params.get("proj_norm", False))
         self.q_norm_w = weights.load(nm["q_norm"], "vector") if self.proj_norm else None
         self.k_norm_w = weights.load(nm["k_norm"], "vector") if self.proj_norm and self.own_kv else None
         self.w_o = weights.load(nm["o"], "matrix")
+        self.conv_w = None
+        if self.taps:
+            self.conv_w = torch.cat([weights.load(nm[r], "vector") for r in ("q_conv", "k_conv", "v_conv")]).contiguous()
+            K.shortconv_lib()
         bias = bool(params.get("bias", False))
         self.q_bias = weights.load(nm["q_bias"], "vector") if bias else None
         self.k_bias = weights.load(nm["k_bias"], "vector") if bias and self.own_kv else None
@@ -120,10 +147,12 @@ class PooledWindowAttention:
         self.interleaved = bool(getattr(self.position, "interleaved", False))
         # the per-token preparation with one block a token takes the norm over whole projections and both rotation layouts
         self.prep_by_token = self.proj_norm or self.interleaved
+        if self.prep_by_token and self.taps:
+            raise ValueError("pooled_window_attention: the convolution does not go with a norm over the whole projection or the interleaved layout")
         if self.prep_by_token and bias:
             raise ValueError("pooled_window_attention: biases do not go with a norm over the whole projection or the interleaved layout")
-        if self.head_gate:
-            K.latent_attn_lib()            # the per-head gate kernel lives beside the other gated attention
+        if self.head_gate or self.value_gate:
+            K.latent_attn_lib()            # the gate kernel lives beside the other gated attention
         self.rot = int(getattr(self.position, "rotary_dim", 0) or 0) if getattr(self.position, "inv_freq", None) is not None else 0
         K.pool_attention_lib(self.qk_dim, self.v_dim, self.group)   # build (or find) the kernels of this head shape now
         self.use_prefill_kernel = rt.is_bf16 and K.pool_attention_prefill_supported(self.qk_dim, self.v_dim, self.group)
@@ -145,14 +174,17 @@ class PooledWindowAttention:
         if self.size >= NO_WINDOW:
             return KVNeed(self.n_kv, self.qk_dim, None, self.v_dim)
         # rows that must stay: the window's, and those of the block that is still to be summarised
-        return KVNeed(self.n_kv, self.qk_dim, max(self.size, self.pool), self.v_dim, None, True, self.pool or None)
+        return KVNeed(self.n_kv, self.qk_dim, max(self.size, self.pool), self.v_dim, None, True, self.pool or None, self.keep)
 
-    def state_need(self) -> Optional[StateNeed]:
-        return None
+    def state_need(self):
+        if self.taps < 2:
+            return None
+        # the projected values of the last tokens, in the type the product leaves: row (position % taps) of a ring
+        return {"conv": StateNeed((self.taps, self.conv_w.shape[0]), self.rt.dtype)}
 
     def _n_splits(self, n_rows: int, max_kv: int) -> int:
         """Keys of a row split over enough blocks to fill the device, a block taking at least 128 keys."""
-        keys = min(max(1, max_kv), self.size) + (max(1, max_kv) // self.pool if self.pool else 0)
+        keys = min(max(1, max_kv), self.size) + self.keep + (max(1, max_kv) // self.pool if self.pool else 0)
         want = math.ceil(2 * self.rt.sm_count / max(1, n_rows * self.n_kv))
         return max(1, min(32, want, (keys + 127) // 128))
 
@@ -173,7 +205,10 @@ class PooledWindowAttention:
         else:
             K.pool_attn_prep(proj, self.q_bias, self.k_bias, self.v_bias, pos.inv_freq if self.rot else None,
                              getattr(pos, "inv_freq_lo", None) if self.rot else None, self.rot, ctx.tok_slot, ctx.tok_pos, q, cache.k,
-                             cache.v, cache.page_table, self.n_heads, self.n_kv, self.eps if self.unit_norm else -1.0, owns_cache)
+                             cache.v, cache.page_table, self.n_heads, self.n_kv, self.eps if self.unit_norm else -1.0, owns_cache,
+                             conv_w=self.conv_w, ring=state["conv"] if self.taps > 1 else None, store_ring=ctx.decode)
+            if self.taps > 1 and not ctx.decode:
+                K.conv_ring_store(proj, 0, ctx.cu_q, ctx.seq_slot, ctx.tok_pos, state["conv"], ctx.n_seqs)
         pooled = None
         if self.pool:
             pc = cache.pooled
@@ -186,7 +221,7 @@ class PooledWindowAttention:
         o = torch.empty((n, self.n_heads, self.v_dim), dtype=h.dtype, device=dev)
         if self.use_prefill_kernel and not ctx.decode and ctx.n_tiles > 0 and cache.k.shape[2] == 64:
             K.pool_attn_prefill(q, cache.k, cache.v, cache.page_table, pooled, self.sink, ctx.tile_tok0, ctx.tile_rows, ctx.tok_slot,
-                                ctx.tok_pos, o, ctx.n_tiles, self.scale, self.size, self.pool)
+                                ctx.tok_pos, o, ctx.n_tiles, self.scale, self.size, self.pool, keep=self.keep)
         else:
             s = self._n_splits(n, ctx.max_kv)
             part_o = part_ml = None
@@ -194,8 +229,10 @@ class PooledWindowAttention:
                 part_o = torch.empty((n, self.n_heads, s, self.v_dim), dtype=torch.float32, device=dev)
                 part_ml = torch.empty((n, self.n_heads, s, 2), dtype=torch.float32, device=dev)
             K.pool_attn_rows(q, cache.k, cache.v, cache.page_table, pooled, self.sink, ctx.tok_slot, ctx.tok_pos, o, self.scale,
-                             self.size, self.pool, s, part_o, part_ml)
+                             self.size, self.pool, s, part_o, part_ml, keep=self.keep)
         o = o.view(n, self.o_dim)
         if self.head_gate:
             K.head_gate_rows(o, proj, self.gate_col, o, self.n_heads, self.v_dim)     # in place: an entry reads only itself
+        elif self.value_gate:       # a gate per value: every value is a "head" of its own to the same kernel
+            K.head_gate_rows(o, proj, self.gate_col, o, self.o_dim, 1)
         return linear(o, self.w_o, self.rt)

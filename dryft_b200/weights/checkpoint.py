@@ -93,8 +93,10 @@ class Checkpoint:
     def check(self, expected: Mapping[str, TensorInfo]) -> None:
         missing = [n for n, info in expected.items() if n not in self._where and not info.optional]
         unexpected = [n for n in self._where if n not in expected]
-        wrong = [(n, info.shape, self.shapes[n]) for n, info in expected.items()
-                 if n in self._where and tuple(info.shape) != self.shapes[n]]
+        def fits(info: TensorInfo, found: tuple) -> bool:      # a free dimension may have any size
+            return len(found) == len(info.shape) and all(i in info.free or a == b for i, (a, b) in enumerate(zip(info.shape, found)))
+
+        wrong = [(n, info.shape, self.shapes[n]) for n, info in expected.items() if n in self._where and not fits(info, self.shapes[n])]
         other = [f"{n}: dtype of the stored tensor is not supported" for n in expected
                  if n in self._where and (self.dtypes[n] is None or self.dtypes[n] == torch.bool)]
         if missing or unexpected or wrong or other:

@@ -43,6 +43,10 @@ class WeightSource:
     def stored_dtype(self, name: str) -> torch.dtype:
         raise NotImplementedError
 
+    def shape(self, name: str) -> tuple:
+        """The stored tensor's shape (for sizes the configuration does not give)."""
+        raise NotImplementedError
+
     def _read(self, name: str) -> torch.Tensor:
         """The stored tensor, on any device."""
         raise NotImplementedError
@@ -79,6 +83,9 @@ class CheckpointSource(WeightSource):
 
     def stored_dtype(self, name: str) -> torch.dtype:
         return self.ckpt.dtypes[name]
+
+    def shape(self, name: str) -> tuple:
+        return self.ckpt.shapes[name]
 
     def _read(self, name: str) -> torch.Tensor:
         return self.ckpt.read(name)
@@ -128,6 +135,9 @@ class RandomSource(WeightSource):
 
     def stored_dtype(self, name: str) -> torch.dtype:
         return self.store_dtype
+
+    def shape(self, name: str) -> tuple:
+        return tuple(self.expected[name].shape)
 
     def _read(self, name: str) -> torch.Tensor:
         return random_tensor(name, self.expected[name], self.seed, self.std, self.draw_device).to(self.store_dtype)
