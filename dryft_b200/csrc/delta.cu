@@ -31,7 +31,8 @@
 //   delta_walk    one block per (16 value columns, head, sequence), a warp four columns: quads in order from the slot's state,
 //                 records and v brought to shared memory a few quads ahead by cp.async; the 32 sums of a warp and quad are
 //                 formed by one butterfly that leaves lane l with sum l.  Leaves o [n, H*dv] and the slot's state.
-//   delta_norm    one warp per (token, head): the norm over dv, the weight and the gate.
+//   delta_norm    one warp per (token, head): the norm over dv, the weight and the gate.  Further blocks store the convolution's
+//                 last inputs in the ring (this launch runs behind the one that reads it).
 //   delta_decode  one token per sequence: one block per (head, sequence) does all of it, the ring's new row included.
 // Sequences with slot -1 (padding) are skipped (their output rows are zeros).  No block waits on another block; the only waits
 // are cp.async.wait_group and __syncthreads.
@@ -44,16 +45,42 @@ constexpr int QUAD = 4;
 constexpr int PREP_THREADS = 256;
 constexpr int V_SPLIT = 4;            // blocks a tile's quads are dealt to while v is convolved
 constexpr int WALK_WARPS = 4;
-constexpr int CPW = 4;                // value columns a warp of the walk owns
-constexpr int WALK_COLS = WALK_WARPS * CPW;
+constexpr int WALK_STAGES = 4;        // quads of the walk in shared memory at once
+constexpr long long FEW_COLUMNS = 8 * 148;
+constexpr int V_PAD = 16;             // rows of the convolved v are padded to whole blocks of columns
 constexpr int SCAL = 28;              // numbers of a record behind its vectors
 constexpr int DEC_COLS = 8;           // value columns a warp of the decode kernel holds at once
 constexpr int DEC_THREADS = 512;
 constexpr unsigned FULL = 0xffffffffu;
 
-__device__ __forceinline__ float sigmoidf_(float v) { return 1.f / (1.f + expf(-v)); }
-__device__ __forceinline__ float siluf_(float v) { return v / (1.f + expf(-v)); }
+constexpr float LOG2E = 1.4426950408889634f, LN2 = 0.6931471805599453f;
+
+// two to the power x, one instruction (2 ulp)
+__device__ __forceinline__ float exp2_(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float sigmoidf_(float v) { return __fdividef(1.f, 1.f + exp2_(-LOG2E * v)); }
+__device__ __forceinline__ float siluf_(float v) { return v * sigmoidf_(v); }
 __device__ __forceinline__ float softplusf_(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+template <typename T> __device__ __forceinline__ float4 load4(const T* p);
+template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&raw.x), b = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
+  return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, float4 v);
+template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 raw;
+  raw.x = *reinterpret_cast<unsigned*>(&a);
+  raw.y = *reinterpret_cast<unsigned*>(&b);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
 
 __device__ __forceinline__ int seq_of(const int* __restrict__ cu_q, int n_seqs, int t) {
   int lo = 0, hi = n_seqs - 1;        // largest b with cu_q[b] <= t
@@ -130,7 +157,7 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
     const T* __restrict__ proj, int ld, int x_off, int b_off, const T* __restrict__ dec, int dec_ld, const float* __restrict__ conv_w,
     int taps, const T* __restrict__ ring, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
     const int* __restrict__ tile_tok0, const int* __restrict__ tile_rows, const int* __restrict__ cu_q, int n_seqs,
-    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, int H, int G, int d, int dv, int dp, int dvp,
+    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, int H, int G, int d, int dv, int dvp,
     float* __restrict__ rec, float* __restrict__ vbuf) {
   const int tile = blockIdx.x;
   const int tok0 = tile_tok0[tile], rows = tile_rows[tile];
@@ -160,8 +187,9 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
 
   const int h = blockIdx.y, g = h / (H / G);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const float rate = -expf(a_log[h]);
-  const size_t RS = (size_t)13 * dp + SCAL;
+  const float rate = -LOG2E * expf(a_log[h]);      // log decays in powers of two
+  constexpr int dr = 32 * DR;      // a record's vectors are padded with zeros to whole warps
+  constexpr size_t RS = (size_t)13 * dr + SCAL;
   for (int qd = warp; qd < nq; qd += PREP_THREADS / 32) {
     const int i0 = i_tile + qd * QUAD, m = min(QUAD, n - i0);
     float q[QUAD][DR], k[QUAD][DR], lg[QUAD][DR];
@@ -172,6 +200,16 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
       for (int i = 0; i < QUAD; ++i)
         head_lg[i] = i < m ? rate * softplusf_(to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h]) + dt_bias[h]) : 0.f;
     }
+    float z[QUAD][DR];                 // the decays' pre-activations, requested first
+    if (CHAN) {
+#pragma unroll
+      for (int i = 0; i < QUAD; ++i)
+#pragma unroll
+        for (int r = 0; r < DR; ++r) {
+          const int c = lane + 32 * r;
+          z[i][r] = c < d && i < m ? to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h * d + c]) : 0.f;
+        }
+    }
 #pragma unroll
     for (int r = 0; r < DR; ++r) {
       const int c = lane + 32 * r;
@@ -181,13 +219,20 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
         conv4<T>(ak, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, (G + g) * d + c);
       }
 #pragma unroll
+      for (int i = 0; i < QUAD; ++i) { q[i][r] = aq[i]; k[i][r] = ak[i]; }
+    }
+#pragma unroll
+    for (int r = 0; r < DR; ++r) {
+      const int c = lane + 32 * r;
+      const float bias = CHAN && c < d ? dt_bias[h * d + c] : 0.f;
+#pragma unroll
       for (int i = 0; i < QUAD; ++i) {
         const bool on = c < d && i < m;
-        q[i][r] = on ? siluf_(aq[i]) : 0.f;
-        k[i][r] = on ? siluf_(ak[i]) : 0.f;
+        q[i][r] = on ? siluf_(q[i][r]) : 0.f;
+        k[i][r] = on ? siluf_(k[i][r]) : 0.f;
         sq[i] = fmaf(q[i][r], q[i][r], sq[i]);
         sk[i] = fmaf(k[i][r], k[i][r], sk[i]);
-        if (CHAN) lg[i][r] = on ? rate * softplusf_(to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h * d + c]) + dt_bias[h * d + c]) : 0.f;
+        if (CHAN) lg[i][r] = on ? rate * softplusf_(z[i][r] + bias) : 0.f;
         else lg[i][r] = head_lg[i];
       }
     }
@@ -209,7 +254,7 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
       const float l1 = lg[1][r], l2 = lg[2][r], l3 = lg[3][r];
       const float g0 = lg[0][r], g1 = g0 + l1, g2 = g1 + l2, g3 = g2 + l3;
       // decays from token j to token i of the quad: sums of the log decays in between, so e^0 = 1 where nothing decays
-      const float e10 = expf(l1), e21 = expf(l2), e20 = expf(l1 + l2), e32 = expf(l3), e31 = expf(l2 + l3), e30 = expf(l1 + l2 + l3);
+      const float e10 = exp2_(l1), e21 = exp2_(l2), e20 = exp2_(l1 + l2), e32 = exp2_(l3), e31 = exp2_(l2 + l3), e30 = exp2_(l1 + l2 + l3);
       A[0] = fmaf(k[1][r] * k[0][r], e10, A[0]);
       A[1] = fmaf(k[2][r] * k[0][r], e20, A[1]); A[2] = fmaf(k[2][r] * k[1][r], e21, A[2]);
       A[3] = fmaf(k[3][r] * k[0][r], e30, A[3]); A[4] = fmaf(k[3][r] * k[1][r], e31, A[4]); A[5] = fmaf(k[3][r] * k[2][r], e32, A[5]);
@@ -218,13 +263,13 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
       P[3] = fmaf(q[2][r] * k[0][r], e20, P[3]); P[4] = fmaf(q[2][r] * k[1][r], e21, P[4]); P[5] = fmaf(q[2][r], k[2][r], P[5]);
       P[6] = fmaf(q[3][r] * k[0][r], e30, P[6]); P[7] = fmaf(q[3][r] * k[1][r], e31, P[7]);
       P[8] = fmaf(q[3][r] * k[2][r], e32, P[8]); P[9] = fmaf(q[3][r], k[3][r], P[9]);
-      if (c < dp) {
-        const float x0 = expf(g0), x1 = expf(g1), x2 = expf(g2), x3 = expf(g3);
-        rc[c] = beta[0] * k[0][r] * x0; rc[dp + c] = beta[1] * k[1][r] * x1;
-        rc[2 * dp + c] = beta[2] * k[2][r] * x2; rc[3 * dp + c] = beta[3] * k[3][r] * x3;
-        rc[4 * dp + c] = q[0][r] * x0; rc[5 * dp + c] = q[1][r] * x1; rc[6 * dp + c] = q[2][r] * x2; rc[7 * dp + c] = q[3][r] * x3;
-        rc[8 * dp + c] = k[0][r] * e30; rc[9 * dp + c] = k[1][r] * e31; rc[10 * dp + c] = k[2][r] * e32; rc[11 * dp + c] = k[3][r];
-        rc[12 * dp + c] = c < d ? expm1f(g3) : 0.f;
+      {
+        const float x0 = exp2_(g0), x1 = exp2_(g1), x2 = exp2_(g2), x3 = exp2_(g3);
+        rc[c] = beta[0] * k[0][r] * x0; rc[dr + c] = beta[1] * k[1][r] * x1;
+        rc[2 * dr + c] = beta[2] * k[2][r] * x2; rc[3 * dr + c] = beta[3] * k[3][r] * x3;
+        rc[4 * dr + c] = q[0][r] * x0; rc[5 * dr + c] = q[1][r] * x1; rc[6 * dr + c] = q[2][r] * x2; rc[7 * dr + c] = q[3][r] * x3;
+        rc[8 * dr + c] = k[0][r] * e30; rc[9 * dr + c] = k[1][r] * e31; rc[10 * dr + c] = k[2][r] * e32; rc[11 * dr + c] = k[3][r];
+        rc[12 * dr + c] = c < d ? expm1f(LN2 * g3) : 0.f;
       }
     }
 #pragma unroll
@@ -232,7 +277,7 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
 #pragma unroll
     for (int i = 0; i < 10; ++i) P[i] = warp_sum(P[i]);
     if (lane == 0) {
-      float4* s = reinterpret_cast<float4*>(rc + 13 * dp);
+      float4* s = reinterpret_cast<float4*>(rc + 13 * dr);
       s[0] = make_float4(beta[0], beta[1], beta[2], beta[3]);
       s[1] = make_float4(beta[1] * A[0], beta[2] * A[1], beta[2] * A[2], beta[3] * A[3]);
       s[2] = make_float4(beta[3] * A[4], beta[3] * A[5], 0.f, 0.f);
@@ -244,36 +289,69 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
   }
 }
 
-template <int RPL> struct WalkStages { static constexpr int value = RPL >= 8 ? 3 : 4; };   // quads in shared memory at once
+// two neighbouring rows at once: fused multiply-adds on register pairs (each half rounds like the single one)
+typedef unsigned long long pair_t;
+__device__ __forceinline__ pair_t fma2(pair_t a, pair_t b, pair_t c) {
+  pair_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ pair_t mul2(pair_t a, pair_t b) {
+  pair_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ pair_t pack2(float lo, float hi) {
+  pair_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float sum2(pair_t a) {
+  float lo, hi;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(a));
+  return lo + hi;
+}
 
-template <int RPL>
+// A group of L lanes owns CPG value columns; lane l of the group holds the rows 4 (l + L m) .. + 3 for m < RPL / 4 (vectors of
+// 16 bytes, neighbouring lanes side by side).  Records hold vectors of L * RPL floats, so no lane needs a bound.
+template <int L, int RPL, int CPG>
 __global__ void __launch_bounds__(WALK_WARPS * 32) delta_walk_kernel(
     const float* __restrict__ rec, const float* __restrict__ vbuf, const int* __restrict__ cu_q, const int* __restrict__ seq_slot,
     int H, int dv, int dp, int dvp, float* __restrict__ state, float* __restrict__ o) {
-  constexpr int NST = WalkStages<RPL>::value;
+  constexpr int DR = L * RPL, RS = 13 * DR + SCAL;
+  constexpr int COLS = WALK_WARPS * (32 / L) * CPG;         // value columns of the block
+  constexpr int NV = QUAD * COLS / 4;                       // 16-byte pieces of a quad's v
+  constexpr int STAGE = RS + QUAD * COLS;
+  constexpr int NST = WALK_STAGES;
+  constexpr int VALS = 8 * CPG, DUP = L / VALS;             // sums a group forms; lanes that end up with the same one
+  constexpr int THREADS = WALK_WARPS * 32;
+  static_assert(VALS <= L, "a lane is left with one sum");
   extern __shared__ __align__(16) float stage_mem[];
-  __shared__ __align__(16) float sums[WALK_WARPS][16];
   const int b = blockIdx.z, h = blockIdx.y;
   const int slot = seq_slot[b];
   const int t0 = cu_q[b], n = cu_q[b + 1] - t0;
   if (slot < 0 || n <= 0) return;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int blk0 = blockIdx.x * WALK_COLS, col0 = blk0 + warp * CPW;
-  const int RS = 13 * dp + SCAL;
-  const int stage_floats = RS + QUAD * WALK_COLS;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gl = lane % L;
+  const int blk0 = blockIdx.x * COLS, lcol = (warp * (32 / L) + lane / L) * CPG, col0 = blk0 + lcol;
   const int nq = (n + QUAD - 1) / QUAD;
   const float* rc0 = rec + (quad_base(t0, b) * H + h) * (size_t)RS;
   const size_t rstep = (size_t)H * RS;
+  const float* v0 = vbuf + (size_t)t0 * H * dvp + (size_t)h * dvp + blk0;
+  const size_t vstep = (size_t)H * dvp;
 
   auto issue = [&](int j) {      // record and v rows of quad j -> its stage
     if (j < nq) {
-      float* sm = stage_mem + (j % NST) * stage_floats;
+      float* sm = stage_mem + (j % NST) * STAGE;
       const float* src = rc0 + (size_t)j * rstep;
-      for (int i = tid * 4; i < RS; i += WALK_WARPS * 32 * 4) cp_async16(sm + i, src + i);
-      for (int i = tid; i < QUAD * (WALK_COLS / 4); i += WALK_WARPS * 32) {
-        const int r = i / (WALK_COLS / 4), c = (i % (WALK_COLS / 4)) * 4;
+#pragma unroll
+      for (int k = 0; k < (RS / 4 + THREADS - 1) / THREADS; ++k) {
+        const int i = (tid + k * THREADS) * 4;
+        if (i < RS) cp_async16(sm + i, src + i);
+      }
+      if (tid < NV) {
+        const int r = tid / (COLS / 4), c = (tid % (COLS / 4)) * 4;
         const int t = min(j * QUAD + r, n - 1);      // a quad's missing tokens have beta = 0: any finite row will do
-        cp_async16(sm + RS + r * WALK_COLS + c, vbuf + (size_t)(t0 + t) * H * dvp + (size_t)h * dvp + blk0 + c);
+        cp_async16(sm + RS + r * COLS + c, v0 + (size_t)t * vstep + c);
       }
     }
     cp_async_commit();
@@ -281,92 +359,131 @@ __global__ void __launch_bounds__(WALK_WARPS * 32) delta_walk_kernel(
 #pragma unroll
   for (int j = 0; j < NST - 1; ++j) issue(j);
 
-  float S[CPW][RPL];
+  pair_t S[CPG][RPL / 2];
   float* sp = state + (((size_t)slot * H + h) * dv + col0) * dp;
-  const int row0 = lane * RPL;
 #pragma unroll
-  for (int c = 0; c < CPW; ++c) {
-    if (col0 + c < dv) load_rows<RPL>(S[c], sp + (size_t)c * dp, row0, dp);
-    else
+  for (int c = 0; c < CPG; ++c)
 #pragma unroll
-      for (int r = 0; r < RPL; ++r) S[c][r] = 0.f;
-  }
+    for (int m = 0; m < RPL / 4; ++m) {
+      const int row = 4 * (gl + L * m);
+      ulonglong2 x = make_ulonglong2(0ull, 0ull);
+      if (col0 + c < dv && row < dp) x = *reinterpret_cast<const ulonglong2*>(sp + (size_t)c * dp + row);
+      S[c][2 * m] = x.x;
+      S[c][2 * m + 1] = x.y;
+    }
+
+  const int id = gl / DUP, o_tok = id / CPG & 3, o_col = id % CPG;
+  const bool o_on = id >= 4 * CPG && gl % DUP == 0 && col0 + o_col < dv;
+  float* op = o + (size_t)(t0 + o_tok) * H * dv + (size_t)h * dv + col0 + o_col;
 
   for (int j = 0; j < nq; ++j) {
     cp_async_wait<NST - 2>();
     __syncthreads();               // quad j is in shared memory; everyone is done with quad j - 1
     issue(j + NST - 1);
-    const float* sm = stage_mem + (j % NST) * stage_floats;
-    float x[32];
+    const float* sm = stage_mem + (j % NST) * STAGE;
+    const float* vec = sm + 4 * gl;
+    float x[VALS];                 // index: (token, or 4 + token for the query) * CPG + column
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      float kt[RPL];
-      load_rows<RPL>(kt, sm + i * dp, row0, dp);
+      pair_t kt[RPL / 2];
 #pragma unroll
-      for (int c = 0; c < CPW; ++c) {
-        float a = kt[0] * S[c][0];
+      for (int m = 0; m < RPL / 4; ++m) {
+        const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(vec + i * DR + 4 * L * m);
+        kt[2 * m] = t.x;
+        kt[2 * m + 1] = t.y;
+      }
 #pragma unroll
-        for (int r = 1; r < RPL; ++r) a = fmaf(kt[r], S[c][r], a);
-        x[i * CPW + c] = a;
+      for (int c = 0; c < CPG; ++c) {
+        pair_t a = mul2(kt[0], S[c][0]);
+#pragma unroll
+        for (int r = 1; r < RPL / 2; ++r) a = fma2(kt[r], S[c][r], a);
+        x[i * CPG + c] = sum2(a);
       }
     }
-    const float mine = butterfly<32>(x, lane);     // lane l < 16: key sum of token l / 4, column l % 4; above: query sums
-    if (lane < 16) sums[warp][lane] = mine;
-    __syncwarp();
-    const float* sc = sm + 13 * dp;
+    // one butterfly over the group: lane gl is left with the sum of index gl / DUP
+    {
+      int off = L / 2;
+#pragma unroll
+      for (int m = VALS / 2; m > 0; m >>= 1, off >>= 1) {
+        const bool up = (gl & off) != 0;
+#pragma unroll
+        for (int i = 0; i < VALS / 2; ++i) {
+          if (i < m) {
+            const float send = up ? x[i] : x[i + m], keep = up ? x[i + m] : x[i];
+            x[i] = keep + __shfl_xor_sync(FULL, send, off);
+          }
+        }
+      }
+#pragma unroll
+      for (int w = DUP / 2; w > 0; w >>= 1) x[0] += __shfl_xor_sync(FULL, x[0], w);
+    }
+    const float mine = x[0];
+    const float* sc = sm + 13 * DR;
     const float4 be = *reinterpret_cast<const float4*>(sc), a0 = *reinterpret_cast<const float4*>(sc + 4),
                  a1 = *reinterpret_cast<const float4*>(sc + 8);
-    float u[QUAD][CPW];
-    {
-      const float bi[4] = {be.x, be.y, be.z, be.w};
-      const float A[6] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y};
+    const float bi[4] = {be.x, be.y, be.z, be.w};
+    const float A[6] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y};
+    float u[QUAD][CPG];
 #pragma unroll
-      for (int i = 0; i < QUAD; ++i) {
-        const float4 dk = *reinterpret_cast<const float4*>(&sums[warp][i * 4]);
-        const float4 vv = *reinterpret_cast<const float4*>(sm + RS + i * WALK_COLS + warp * CPW);
-        u[i][0] = fmaf(bi[i], vv.x, -dk.x); u[i][1] = fmaf(bi[i], vv.y, -dk.y);
-        u[i][2] = fmaf(bi[i], vv.z, -dk.z); u[i][3] = fmaf(bi[i], vv.w, -dk.w);
+    for (int i = 0; i < QUAD; ++i)
 #pragma unroll
-        for (int jj = 0; jj < i; ++jj)
+      for (int c = 0; c < CPG; ++c) {
+        const float dk = __shfl_sync(FULL, mine, (i * CPG + c) * DUP, L);
+        u[i][c] = fmaf(bi[i], sm[RS + i * COLS + lcol + c], -dk);
 #pragma unroll
-          for (int c = 0; c < CPW; ++c) u[i][c] = fmaf(-A[i * (i - 1) / 2 + jj], u[jj][c], u[i][c]);
+        for (int jj = 0; jj < i; ++jj) u[i][c] = fmaf(-A[i * (i - 1) / 2 + jj], u[jj][c], u[i][c]);
       }
-    }
     {
-      float gm[RPL];
-      load_rows<RPL>(gm, sm + 12 * dp, row0, dp);
+      pair_t gm[RPL / 2];
 #pragma unroll
-      for (int c = 0; c < CPW; ++c)
+      for (int m = 0; m < RPL / 4; ++m) {
+        const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(vec + 12 * DR + 4 * L * m);
+        gm[2 * m] = t.x;
+        gm[2 * m + 1] = t.y;
+      }
 #pragma unroll
-        for (int r = 0; r < RPL; ++r) S[c][r] = fmaf(S[c][r], gm[r], S[c][r]);
+      for (int c = 0; c < CPG; ++c)
+#pragma unroll
+        for (int r = 0; r < RPL / 2; ++r) S[c][r] = fma2(S[c][r], gm[r], S[c][r]);
     }
 #pragma unroll
     for (int i = 0; i < QUAD; ++i) {
-      float kb[RPL];
-      load_rows<RPL>(kb, sm + (8 + i) * dp, row0, dp);
+      pair_t kb[RPL / 2];
 #pragma unroll
-      for (int c = 0; c < CPW; ++c)
+      for (int m = 0; m < RPL / 4; ++m) {
+        const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(vec + (8 + i) * DR + 4 * L * m);
+        kb[2 * m] = t.x;
+        kb[2 * m + 1] = t.y;
+      }
 #pragma unroll
-        for (int r = 0; r < RPL; ++r) S[c][r] = fmaf(kb[r], u[i][c], S[c][r]);
+      for (int c = 0; c < CPG; ++c) {
+        const pair_t uu = pack2(u[i][c], u[i][c]);
+#pragma unroll
+        for (int r = 0; r < RPL / 2; ++r) S[c][r] = fma2(kb[r], uu, S[c][r]);
+      }
     }
-    if (lane >= 16) {
-      const int i = (lane >> 2) & 3, c = lane & 3;
-      const float4 Pr = *reinterpret_cast<const float4*>(sc + 12 + i * 4);
+    {      // the lanes that hold a query's sum finish its output
+      const float4 Pr = *reinterpret_cast<const float4*>(sc + 12 + o_tok * 4);
       const float pr[4] = {Pr.x, Pr.y, Pr.z, Pr.w};
       float val = mine;
 #pragma unroll
       for (int jj = 0; jj < QUAD; ++jj) {
-        const float uc = c < 2 ? (c == 0 ? u[jj][0] : u[jj][1]) : (c == 2 ? u[jj][2] : u[jj][3]);
+        float uc = u[jj][0];
+#pragma unroll
+        for (int cc = 1; cc < CPG; ++cc) uc = o_col == cc ? u[jj][cc] : uc;
         val = fmaf(pr[jj], uc, val);
       }
-      const int t = j * QUAD + i;
-      if (t < n && col0 + c < dv) o[(size_t)(t0 + t) * H * dv + (size_t)h * dv + col0 + c] = val;
+      if (o_on && j * QUAD + o_tok < n) op[(size_t)j * QUAD * H * dv] = val;
     }
   }
   cp_async_wait<0>();
 #pragma unroll
-  for (int c = 0; c < CPW; ++c)
-    if (col0 + c < dv) store_rows<RPL>(S[c], sp + (size_t)c * dp, row0, dp);
+  for (int c = 0; c < CPG; ++c)
+#pragma unroll
+    for (int m = 0; m < RPL / 4; ++m) {
+      const int row = 4 * (gl + L * m);
+      if (col0 + c < dv && row < dp) *reinterpret_cast<ulonglong2*>(sp + (size_t)c * dp + row) = make_ulonglong2(S[c][2 * m], S[c][2 * m + 1]);
+    }
 }
 
 constexpr int NORM_WARPS = 4;
@@ -375,7 +492,19 @@ template <typename T>
 __global__ void __launch_bounds__(NORM_WARPS * 32) delta_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_ld,
                                                                     const float* __restrict__ w, float eps, int sigmoid_gate,
                                                                     const int* __restrict__ tok_slot, T* __restrict__ out, int n, int H,
-                                                                    int dv) {
+                                                                    int dv, int norm_blocks, const T* __restrict__ x, int ld,
+                                                                    const int* __restrict__ cu_q, const int* __restrict__ seq_slot,
+                                                                    const int* __restrict__ tok_pos, T* __restrict__ ring, int taps, int CH) {
+  if ((int)blockIdx.x >= norm_blocks) {      // the ring: a thread a (sequence, channel)
+    const int cb = (CH + NORM_WARPS * 32 - 1) / (NORM_WARPS * 32), i = (int)blockIdx.x - norm_blocks;
+    const int b = i / cb, c = (i % cb) * NORM_WARPS * 32 + threadIdx.x, slot = seq_slot[b];
+    const int t1 = cu_q[b + 1], nb = t1 - cu_q[b];
+    if (slot < 0 || nb <= 0 || c >= CH) return;
+    const int last = tok_pos[t1 - 1];
+    for (int k = 0; k < taps - 1 && k < nb; ++k)
+      ring[((size_t)slot * taps + (last - k) % taps) * CH + c] = x[(size_t)(t1 - 1 - k) * ld + c];
+    return;
+  }
   const int lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * NORM_WARPS + (threadIdx.x >> 5);
   if (item >= (long long)n * H) return;
@@ -388,6 +517,30 @@ __global__ void __launch_bounds__(NORM_WARPS * 32) delta_norm_kernel(const float
   const float* src = o + (size_t)t * H * dv + (size_t)h * dv;
   const T* gt = gate + (size_t)t * gate_ld + (size_t)h * dv;
   float ss = 0.f;
+  // heads of up to 256 values in steps of four, rows on their vectors' boundaries: a lane keeps its values in registers
+  if (dv % 4 == 0 && dv <= 256 && gate_ld % 4 == 0 && reinterpret_cast<uintptr_t>(gate) % (4 * sizeof(T)) == 0) {
+    float4 v[2], z[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int c = 4 * (lane + 32 * k);
+      v[k] = z[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < dv) { v[k] = *reinterpret_cast<const float4*>(src + c); z[k] = load4<T>(gt + c); }
+    }
+#pragma unroll
+    for (int k = 0; k < 2; ++k) ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+    const float rinv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int c = 4 * (lane + 32 * k);
+      if (c < dv) {
+        const float4 ww = *reinterpret_cast<const float4*>(w + c);
+        auto act = [&](float x) { return sigmoid_gate ? sigmoidf_(x) : siluf_(x); };
+        store4<T>(dst + c, make_float4(v[k].x * rinv * ww.x * act(z[k].x), v[k].y * rinv * ww.y * act(z[k].y),
+                                       v[k].z * rinv * ww.z * act(z[k].z), v[k].w * rinv * ww.w * act(z[k].w)));
+      }
+    }
+    return;
+  }
   for (int c = lane; c < dv; c += 32) { const float v = src[c]; ss = fmaf(v, v, ss); }
   const float rinv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
   for (int c = lane; c < dv; c += 32) {
@@ -428,13 +581,14 @@ __global__ void __launch_bounds__(DEC_THREADS) delta_decode_kernel(
   const bool first = h % (H / G) == 0;                       // one head of a group stores the group's q and k in the ring
   const T* x = proj + x_off;
   T* ring_row = ring + ((size_t)slot * taps + pos % taps) * CH;
+  const ConvRows<T> conv(conv_w, x, ld, ring, taps, CH, slot, t, pos, 0);
   float aq = 0.f, ak = 0.f, aqk = 0.f;
   for (int c = tid; c < dp; c += nthr) {
     float q = 0.f, k = 0.f, gmc = 0.f;
     if (c < d) {
       const int cq = g * d + c, ck = (G + g) * d + c;
-      q = siluf_(conv1<T>(conv_w, x, ld, ring, taps, CH, slot, t, pos, 0, cq));
-      k = siluf_(conv1<T>(conv_w, x, ld, ring, taps, CH, slot, t, pos, 0, ck));
+      q = siluf_(conv(cq));
+      k = siluf_(conv(ck));
       if (first && taps > 1) { ring_row[cq] = x[(size_t)t * ld + cq]; ring_row[ck] = x[(size_t)t * ld + ck]; }
       const int gi = CHAN ? h * d + c : h;
       gmc = expm1f(-expf(a_log[h]) * softplusf_(to_f32<T>(dec[(size_t)t * dec_ld + gi]) + dt_bias[gi]));
@@ -444,7 +598,7 @@ __global__ void __launch_bounds__(DEC_THREADS) delta_decode_kernel(
   }
   for (int c = tid; c < dv; c += nthr) {
     const int cv = 2 * G * d + h * dv + c;
-    vs[c] = siluf_(conv1<T>(conv_w, x, ld, ring, taps, CH, slot, t, pos, 0, cv));
+    vs[c] = siluf_(conv(cv));
     if (taps > 1) ring_row[cv] = x[(size_t)t * ld + cv];
   }
   const float rq = 1.f / (sqrtf((float)d) * sqrtf(block_sum(aq, scratch) + UNIT_EPS));
@@ -507,27 +661,29 @@ __global__ void __launch_bounds__(DEC_THREADS) delta_decode_kernel(
 template <typename T, int DR, bool CHAN>
 int prep_launch(const void* proj, int ld, int x_off, int b_off, const void* dec, int dec_ld, const float* conv_w, int taps,
                 const void* ring, const float* a_log, const float* dt_bias, const int* tile_tok0, const int* tile_rows, int n_tiles,
-                const int* cu_q, int n_seqs, const int* tok_slot, const int* tok_pos, int H, int G, int d, int dv, int dp, int dvp,
+                const int* cu_q, int n_seqs, const int* tok_slot, const int* tok_pos, int H, int G, int d, int dv, int dvp,
                 float* rec, float* vbuf, cudaStream_t st) {
   const long long vb = ((long long)H * dvp + PREP_THREADS - 1) / PREP_THREADS * V_SPLIT;
   if (H + vb > 65535) return DRYFT_ERR_UNSUPPORTED;
   dim3 grid(n_tiles, (unsigned)(H + vb));
   delta_prep_kernel<T, DR, CHAN><<<grid, PREP_THREADS, 0, st>>>(
       (const T*)proj, ld, x_off, b_off, (const T*)dec, dec_ld, conv_w, taps, (const T*)ring, a_log, dt_bias, tile_tok0, tile_rows, cu_q,
-      n_seqs, tok_slot, tok_pos, H, G, d, dv, dp, dvp, rec, vbuf);
+      n_seqs, tok_slot, tok_pos, H, G, d, dv, dvp, rec, vbuf);
   return launch_status();
 }
 
-template <int RPL>
+template <int L, int RPL, int CPG>
 int walk_launch(const float* rec, const float* vbuf, const int* cu_q, const int* seq_slot, int n_seqs, int H, int dv, int dp, int dvp,
                 float* state, float* o, cudaStream_t st) {
-  const size_t smem = sizeof(float) * WalkStages<RPL>::value * ((size_t)13 * dp + SCAL + QUAD * WALK_COLS);
+  constexpr int COLS = WALK_WARPS * (32 / L) * CPG;
+  static_assert(V_PAD % COLS == 0, "a block's columns lie within a padded row of v");
+  const size_t smem = sizeof(float) * WALK_STAGES * (size_t)(13 * L * RPL + SCAL + QUAD * COLS);
   if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(delta_walk_kernel<RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(delta_walk_kernel<L, RPL, CPG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  dim3 grid((dv + WALK_COLS - 1) / WALK_COLS, H, n_seqs);
-  delta_walk_kernel<RPL><<<grid, WALK_WARPS * 32, smem, st>>>(rec, vbuf, cu_q, seq_slot, H, dv, dp, dvp, state, o);
+  dim3 grid((dv + COLS - 1) / COLS, H, n_seqs);
+  delta_walk_kernel<L, RPL, CPG><<<grid, WALK_WARPS * 32, smem, st>>>(rec, vbuf, cu_q, seq_slot, H, dv, dp, dvp, state, o);
   return launch_status();
 }
 
@@ -560,10 +716,10 @@ DRYFT_API int dryft_delta_prep(int is_bf16, int per_channel, const void* proj, i
                                cudaStream_t st) {
   if (n_tiles <= 0) return 0;
   if (!sizes_ok(H, G, d, dv, taps) || tile_size % QUAD || (taps > 1 && ring == nullptr)) return DRYFT_ERR_UNSUPPORTED;
-  const int dp = (d + 3) / 4 * 4, dvp = (dv + WALK_COLS - 1) / WALK_COLS * WALK_COLS;
+  const int dvp = (dv + V_PAD - 1) / V_PAD * V_PAD;
 #define DRYFT_PREP(T, DR, CH)                                                                                                       \
   return prep_launch<T, DR, CH>(proj, ld, x_off, b_off, dec, dec_ld, conv_w, taps, ring, a_log, dt_bias, tile_tok0, tile_rows, n_tiles, \
-                                cu_q, n_seqs, tok_slot, tok_pos, H, G, d, dv, dp, dvp, rec, vbuf, st)
+                                cu_q, n_seqs, tok_slot, tok_pos, H, G, d, dv, dvp, rec, vbuf, st)
 #define DRYFT_PREP_R(T, CH)                  \
   switch (rows_per_lane(d)) {                \
     case 1: DRYFT_PREP(T, 1, CH);            \
@@ -584,26 +740,37 @@ DRYFT_API int dryft_delta_walk(const float* rec, const float* vbuf, const int* c
                                float* state, float* o, cudaStream_t st) {
   if (n_seqs <= 0) return 0;
   if (!sizes_ok(H, 1, d, dv, 1) || n_seqs > 65535) return DRYFT_ERR_UNSUPPORTED;
-  const int dp = (d + 3) / 4 * 4, dvp = (dv + WALK_COLS - 1) / WALK_COLS * WALK_COLS;
-  switch (rows_per_lane(d)) {
-    case 1: return walk_launch<1>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
-    case 2: return walk_launch<2>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
-    case 4: return walk_launch<4>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
-    default: return walk_launch<8>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st);
+  const int dp = (d + 3) / 4 * 4, dvp = (dv + V_PAD - 1) / V_PAD * V_PAD;
+#define DRYFT_WALK(L, R, C) return walk_launch<L, R, C>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st)
+  switch (rows_per_lane(d)) {      // L * RPL = 32 * rows_per_lane: the length of a record's vectors
+    case 1: DRYFT_WALK(8, 4, 1);
+    case 2: DRYFT_WALK(8, 8, 1);
+    case 4:      // few columns for the device (at most eight an SM): two a warp instead of four
+      if ((long long)n_seqs * H * dv <= FEW_COLUMNS) DRYFT_WALK(32, 4, 2);
+      DRYFT_WALK(32, 4, 4);
+    default: DRYFT_WALK(32, 8, 4);
   }
+#undef DRYFT_WALK
 }
 
 DRYFT_API int dryft_delta_norm(int is_bf16, const float* o, const void* gate, int gate_ld, const float* w, float eps, int sigmoid_gate,
-                               const int* tok_slot, void* out, int n, int H, int dv, cudaStream_t st) {
+                               const int* tok_slot, void* out, int n, int H, int G, int d, int dv, const void* proj, int ld, int x_off,
+                               const int* cu_q, const int* seq_slot, int n_seqs, const int* tok_pos, void* ring, int taps, cudaStream_t st) {
   if (n <= 0) return 0;
-  if (H < 1 || dv < 1) return DRYFT_ERR_UNSUPPORTED;
-  const long long blocks = ((long long)n * H + NORM_WARPS - 1) / NORM_WARPS;
-  if (blocks > 0x7fffffffLL) return DRYFT_ERR_UNSUPPORTED;
+  if (!sizes_ok(H, G, d, dv, taps)) return DRYFT_ERR_UNSUPPORTED;
+  const int CH = 2 * G * d + H * dv;
+  const long long nblk = ((long long)n * H + NORM_WARPS - 1) / NORM_WARPS;
+  const long long rblk = taps > 1 ? (long long)n_seqs * ((CH + NORM_WARPS * 32 - 1) / (NORM_WARPS * 32)) : 0;
+  if (nblk + rblk > 0x7fffffffLL) return DRYFT_ERR_UNSUPPORTED;
   typedef __nv_bfloat16 bf;
+  const unsigned grid = (unsigned)(nblk + rblk);
   if (is_bf16)
-    delta_norm_kernel<bf><<<(unsigned)blocks, NORM_WARPS * 32, 0, st>>>(o, (const bf*)gate, gate_ld, w, eps, sigmoid_gate, tok_slot, (bf*)out, n, H, dv);
+    delta_norm_kernel<bf><<<grid, NORM_WARPS * 32, 0, st>>>(o, (const bf*)gate, gate_ld, w, eps, sigmoid_gate, tok_slot, (bf*)out, n, H, dv,
+                                                            (int)nblk, (const bf*)proj + x_off, ld, cu_q, seq_slot, tok_pos, (bf*)ring, taps, CH);
   else
-    delta_norm_kernel<float><<<(unsigned)blocks, NORM_WARPS * 32, 0, st>>>(o, (const float*)gate, gate_ld, w, eps, sigmoid_gate, tok_slot, (float*)out, n, H, dv);
+    delta_norm_kernel<float><<<grid, NORM_WARPS * 32, 0, st>>>(o, (const float*)gate, gate_ld, w, eps, sigmoid_gate, tok_slot, (float*)out, n, H,
+                                                               dv, (int)nblk, (const float*)proj + x_off, ld, cu_q, seq_slot, tok_pos,
+                                                               (float*)ring, taps, CH);
   return launch_status();
 }
 

@@ -24,7 +24,7 @@
 //                     rows and tokens (one list of keys; a lane a key for the scores, a lane a value column for the
 //                     weighted sum), online softmax per warp, warps combined in shared memory; with one split the sink
 //                     joins there and the output is written, else partial (max, sum, weighted sum) go to memory and
-//   pool_attn_combine joins the splits and the sink.
+//   pool_attn_combine joins the splits and the sink.  With `gate` logits every output value is multiplied by the sigmoid of its own.
 // Tokens with slot -1 (padding) are skipped.  No block waits on another block.
 #include "shortconv.cuh"
 #include <math.h>
@@ -75,10 +75,12 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
   if (conv_w != nullptr)
     while (back < taps - 1 && t - back - 1 >= 0 && tok_slot[t - back - 1] == slot) ++back;
   // channel c of [q | k | v]: the projected value, or the convolution over it
+  const ConvRows<T> conv(conv_w, proj, ld, ring, conv_w != nullptr ? taps : 4, CH, slot, t, pos, back);
+  T* ring_row = store_ring ? ring + ((size_t)slot * taps + pos % taps) * CH : nullptr;
   auto input = [&](int c) {
     if (conv_w == nullptr) return to_f32<T>(row[c]);
-    if (store_ring) ring[((size_t)slot * taps + pos % taps) * CH + c] = row[c];
-    return conv1<T>(conv_w, proj, ld, ring, taps, CH, slot, t, pos, back, c);
+    if (store_ring) ring_row[c] = row[c];
+    return conv(c);
   };
   size_t cache_row = 0;
   if (vec >= H) {
@@ -265,12 +267,18 @@ template <typename T> __device__ __forceinline__ void dot_row(const T* __restric
   }
 }
 
+// the factor of output value c of a token's head: the sigmoid of its logit in [n, H * DV] (no gate: one)
+template <typename T> __device__ __forceinline__ float gate_at(const T* __restrict__ gate, int gate_ld, int t, int head, int c) {
+  return gate == nullptr ? 1.f : 1.f / (1.f + expf(-to_f32<T>(gate[(size_t)t * gate_ld + (size_t)head * DV + c])));
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
     const T* __restrict__ q, const T* __restrict__ k_pages, const T* __restrict__ v_pages, const int* __restrict__ page_table,
     int max_pages, int page_size, const T* __restrict__ pk_pages, const T* __restrict__ pv_pages, const int* __restrict__ pool_table,
     int pool_max_pages, const float* __restrict__ sink, const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
-    T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int G, int n_splits, float scale, int size, int P, int keep) {
+    T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int G, int n_splits, float scale, int size, int P, int keep, const T* __restrict__ gate,
+    int gate_ld) {
   __shared__ float qs[REP][D];
   __shared__ float wo[ROWS_WARPS][REP][DV];
   __shared__ float wml[ROWS_WARPS][REP][2];
@@ -382,7 +390,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
       const float Mx = fmaxf(M, sk);
       const float f = M == -INFINITY ? 0.f : expf(M - Mx);
       const float den = L * f + (sk == -INFINITY ? 0.f : expf(sk - Mx));
-      out[((size_t)t * H + head) * DV + c] = from_f32<T>(den > 0.f ? O * f / den : 0.f);
+      out[((size_t)t * H + head) * DV + c] = from_f32<T>(den > 0.f ? O * f / den * gate_at<T>(gate, gate_ld, t, head, c) : 0.f);
     } else {
       const size_t pi = ((size_t)t * H + head) * n_splits + sp;
       part_o[pi * DV + c] = O;
@@ -394,7 +402,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
 template <typename T>
 __global__ void __launch_bounds__(128) pool_attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                                 const float* __restrict__ sink, const int* __restrict__ tok_slot,
-                                                                T* __restrict__ out, int H, int n_splits) {
+                                                                T* __restrict__ out, int H, int n_splits, const T* __restrict__ gate, int gate_ld) {
   const int t = blockIdx.x, head = blockIdx.y;
   if (tok_slot[t] < 0) return;
   const size_t base = ((size_t)t * H + head) * n_splits;
@@ -412,7 +420,7 @@ __global__ void __launch_bounds__(128) pool_attn_combine_kernel(const float* __r
       const float ms = part_ml[(base + s) * 2];
       if (ms != -INFINITY) O = fmaf(part_o[(base + s) * DV + c], expf(ms - Mx), O);
     }
-    out[((size_t)t * H + head) * DV + c] = from_f32<T>(den > 0.f ? O / den : 0.f);
+    out[((size_t)t * H + head) * DV + c] = from_f32<T>(den > 0.f ? O / den * gate_at<T>(gate, gate_ld, t, head, c) : 0.f);
   }
 }
 
@@ -434,15 +442,15 @@ template <typename T>
 int rows_launch(const void* q, const void* k_pages, const void* v_pages, const int* page_table, int max_pages, int page_size,
                 const void* pk, const void* pv, const int* pool_table, int pool_max_pages, const float* sink, const int* tok_slot,
                 const int* tok_pos, void* out, float* part_o, float* part_ml, int n, int G, int n_splits, float scale, int size, int P,
-                int keep, cudaStream_t st) {
+                int keep, const void* gate, int gate_ld, cudaStream_t st) {
   dim3 grid(n, G, n_splits);
   pool_attn_rows_kernel<T><<<grid, ROWS_WARPS * 32, 0, st>>>((const T*)q, (const T*)k_pages, (const T*)v_pages, page_table, max_pages,
                                                             page_size, (const T*)pk, (const T*)pv, pool_table, pool_max_pages, sink,
-                                                            tok_slot, tok_pos, (T*)out, part_o, part_ml, G, n_splits, scale, size, P, keep);
+                                                            tok_slot, tok_pos, (T*)out, part_o, part_ml, G, n_splits, scale, size, P, keep, (const T*)gate, gate_ld);
   int rc = launch_status();
   if (rc || n_splits == 1) return rc;
   dim3 cgrid(n, G * REP);
-  pool_attn_combine_kernel<T><<<cgrid, 128, 0, st>>>(part_o, part_ml, sink, tok_slot, (T*)out, G * REP, n_splits);
+  pool_attn_combine_kernel<T><<<cgrid, 128, 0, st>>>(part_o, part_ml, sink, tok_slot, (T*)out, G * REP, n_splits, (const T*)gate, gate_ld);
   return launch_status();
 }
 }  // namespace
@@ -505,13 +513,13 @@ DRYFT_API int dryft_pool_attn_rows(int is_bf16, const void* q, const void* k_pag
                                    int max_pages, int page_size, const void* pk, const void* pv, const int* pool_table,
                                    int pool_max_pages, const float* sink, const int* tok_slot, const int* tok_pos, void* out,
                                    float* part_o, float* part_ml, int n, int G, int n_splits, float scale, int size, int P, int keep,
-                                   cudaStream_t st) {
+                                   const void* gate, int gate_ld, cudaStream_t st) {
   if (n <= 0) return 0;
   if (G < 1 || G > 65535 || n_splits < 1 || n_splits > 65535 || size < 1 || keep < 0 || page_size < 1 || (P > 0 && pk == nullptr) ||
       (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return DRYFT_ERR_UNSUPPORTED;
   return is_bf16 ? rows_launch<__nv_bfloat16>(q, k_pages, v_pages, page_table, max_pages, page_size, pk, pv, pool_table, pool_max_pages,
-                                              sink, tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, st)
+                                              sink, tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, gate, gate_ld, st)
                  : rows_launch<float>(q, k_pages, v_pages, page_table, max_pages, page_size, pk, pv, pool_table, pool_max_pages, sink,
-                                      tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, st);
+                                      tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, gate, gate_ld, st);
 }

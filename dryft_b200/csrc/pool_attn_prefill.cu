@@ -94,7 +94,8 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     const int* __restrict__ tile_tok0, const int* __restrict__ tile_rows,
     const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     bf16* __restrict__ out,                                              // [N, nH * DV]
-    int nH, int nKV, float scale_log2, int size, int P, int keep) {
+    int nH, int nKV, float scale_log2, int size, int P, int keep,
+    const bf16* __restrict__ gate, int gate_ld) {                        // gate logits [N, nH * DV] of row stride gate_ld, or null
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);   // [BM][KS]
   bf16* ks = qs + BM * KS;                        // [2][BN][KS]
@@ -269,13 +270,27 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   const float f0 = l0 > 0.f ? 1.f / l0 : 0.f, f1 = l1 > 0.f ? 1.f / l1 : 0.f;
   const int r0 = warp * 16 + g, r1 = r0 + 8;
+  const bool gate_pairs = (gate_ld & 1) == 0 && (reinterpret_cast<uintptr_t>(gate) & 3) == 0;   // two logits a load
 #pragma unroll
   for (int j = 0; j < DT; ++j) {
     const int d = j * 8 + 2 * t;
+    float g00 = f0, g01 = f0, g10 = f1, g11 = f1;
+    if (gate != nullptr) {       // each value times the sigmoid of its own logit
+      auto factors = [&](int r, float& lo, float& hi) {
+        const bf16* gp = gate + (size_t)(tok0 + r) * gate_ld + (size_t)h * DV + d;
+        __nv_bfloat162 z;
+        if (gate_pairs) z = *reinterpret_cast<const __nv_bfloat162*>(gp);
+        else z = __halves2bfloat162(gp[0], gp[1]);
+        lo *= __fdividef(1.f, 1.f + exp2f(-1.4426950408889634f * __low2float(z)));
+        hi *= __fdividef(1.f, 1.f + exp2f(-1.4426950408889634f * __high2float(z)));
+      };
+      if (r0 < rows) factors(r0, g00, g01);
+      if (r1 < rows) factors(r1, g10, g11);
+    }
     if (r0 < rows)
-      *reinterpret_cast<unsigned*>(out + ((size_t)(tok0 + r0) * nH + h) * DV + d) = pack_bf16(o_acc[j][0] * f0, o_acc[j][1] * f0);
+      *reinterpret_cast<unsigned*>(out + ((size_t)(tok0 + r0) * nH + h) * DV + d) = pack_bf16(o_acc[j][0] * g00, o_acc[j][1] * g01);
     if (r1 < rows)
-      *reinterpret_cast<unsigned*>(out + ((size_t)(tok0 + r1) * nH + h) * DV + d) = pack_bf16(o_acc[j][2] * f1, o_acc[j][3] * f1);
+      *reinterpret_cast<unsigned*>(out + ((size_t)(tok0 + r1) * nH + h) * DV + d) = pack_bf16(o_acc[j][2] * g10, o_acc[j][3] * g11);
   }
 }
 }  // namespace
@@ -287,7 +302,7 @@ DRYFT_API int dryft_pool_attn_prefill(const void* q, const void* k_pages, const 
                                       int page_size, const void* pk_pages, const void* pv_pages, const int* pool_table,
                                       int pool_max_pages, const float* sink, const int* tile_tok0, const int* tile_rows,
                                       const int* tok_slot, const int* tok_pos, void* out, int n_tiles, int nH, int nKV, float scale,
-                                      int size, int P, int keep, cudaStream_t st) {
+                                      int size, int P, int keep, const void* gate, int gate_ld, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
   if (nH != nKV * G || nH > 65535 || page_size != BN || size < 1 || P < 0 || keep < 0) return DRYFT_ERR_UNSUPPORTED;
   if (P > 0 && (pk_pages == nullptr || pv_pages == nullptr || pool_table == nullptr)) return DRYFT_ERR_UNSUPPORTED;
@@ -304,6 +319,6 @@ DRYFT_API int dryft_pool_attn_prefill(const void* q, const void* k_pages, const 
   pool_attn_prefill_kernel<<<grid, THREADS, smem, st>>>((const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, page_table,
                                                        max_pages, (const bf16*)pk_pages, (const bf16*)pv_pages, pool_table,
                                                        pool_max_pages, sink, tile_tok0, tile_rows, tok_slot, tok_pos, (bf16*)out, nH,
-                                                       nKV, scale * 1.4426950408889634f, size, P, keep);
+                                                       nKV, scale * 1.4426950408889634f, size, P, keep, (const bf16*)gate, gate_ld);
   return launch_status();
 }

@@ -24,21 +24,27 @@ __device__ __forceinline__ float conv_input(const T* __restrict__ x, int ld, con
 template <typename T>
 __device__ __forceinline__ void conv4(float (&acc)[4], const float* __restrict__ w, const T* __restrict__ x, int ld,
                                       const T* __restrict__ ring, int taps, int CH, int slot, int t0, int p0, int i0, int n, int c) {
-#pragma unroll
-  for (int k = 0; k < 4; ++k) acc[k] = 0.f;
   const float* wc = w + (size_t)c * taps;
   if (taps == 4) {      // the usual case, unrolled: seven inputs, four weights
-    const float w0 = wc[0], w1 = wc[1], w2 = wc[2], w3 = wc[3];
+    const float4 ww = *reinterpret_cast<const float4*>(wc);
     float u[7];
+    if (i0 >= 3 && i0 + 4 <= n) {      // all of them belong to this step: seven loads without a question
+      const T* src = x + (size_t)(t0 + i0 - 3) * ld + c;
 #pragma unroll
-    for (int s = 0; s < 7; ++s) {
-      const int i = i0 - 3 + s;
-      u[s] = i < n ? conv_input<T>(x, ld, ring, taps, CH, slot, t0, p0, i, c) : 0.f;
+      for (int s = 0; s < 7; ++s) u[s] = to_f32<T>(src[(size_t)s * ld]);
+    } else {
+#pragma unroll
+      for (int s = 0; s < 7; ++s) {
+        const int i = i0 - 3 + s;
+        u[s] = i < n ? conv_input<T>(x, ld, ring, taps, CH, slot, t0, p0, i, c) : 0.f;
+      }
     }
 #pragma unroll
-    for (int k = 0; k < 4; ++k) acc[k] = fmaf(w3, u[k + 3], fmaf(w2, u[k + 2], fmaf(w1, u[k + 1], w0 * u[k])));
+    for (int k = 0; k < 4; ++k) acc[k] = fmaf(ww.w, u[k + 3], fmaf(ww.z, u[k + 2], fmaf(ww.y, u[k + 1], ww.x * u[k])));
     return;
   }
+#pragma unroll
+  for (int k = 0; k < 4; ++k) acc[k] = 0.f;
   for (int s = 0; s < taps + 3; ++s) {
     const int i = i0 - (taps - 1) + s;
     if (i >= n) break;
@@ -51,19 +57,43 @@ __device__ __forceinline__ void conv4(float (&acc)[4], const float* __restrict__
   }
 }
 
-// the convolution's result of ONE token (packed row t at position p), of channel c: `back` of the rows before it belong to
-// its sequence and this step
-template <typename T>
-__device__ __forceinline__ float conv1(const float* __restrict__ w, const T* __restrict__ x, int ld, const T* __restrict__ ring,
-                                       int taps, int CH, int slot, int t, int p, int back, int c) {
-  const float* wc = w + (size_t)c * taps;
-  float acc = 0.f;
-  for (int j = 0; j < taps; ++j) {
-    const int d = taps - 1 - j;
-    float u = 0.f;
-    if (d <= back) u = to_f32<T>(x[(size_t)(t - d) * ld + c]);
-    else if (p - d >= 0) u = to_f32<T>(ring[((size_t)slot * taps + (p - d) % taps) * CH + c]);
-    acc = fmaf(wc[j], u, acc);
+// The rows that the convolution of ONE token (packed row t at position p) reads, worked out once for all its channels: `back`
+// of the rows before t belong to its sequence and this step, older ones lie in the ring, and a row before the sequence's
+// start counts as zeros (its weight is dropped; the pointer then names the token's own row).
+template <typename T> struct ConvRows {
+  const T* src[4];
+  float on[4];
+  const float* w;
+  const T* x;
+  const T* ring_slot;
+  int ld, taps, CH, t, p, back;
+
+  __device__ __forceinline__ ConvRows(const float* __restrict__ w_, const T* __restrict__ x_, int ld_, const T* __restrict__ ring, int taps_,
+                                      int CH_, int slot, int t_, int p_, int back_)
+      : w(w_), x(x_), ring_slot(ring + (size_t)slot * taps_ * CH_), ld(ld_), taps(taps_), CH(CH_), t(t_), p(p_), back(back_) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int d = 3 - j;
+      const bool seen = d <= back || p >= d;
+      on[j] = seen ? 1.f : 0.f;
+      src[j] = d <= back || !seen || taps != 4 ? x + (size_t)(t - (seen && d <= back ? d : 0)) * ld : ring_slot + (size_t)((p - d) & 3) * CH;
+    }
   }
-  return acc;
-}
+  __device__ __forceinline__ float operator()(int c) const {
+    const float* wc = w + (size_t)c * taps;
+    if (taps == 4) {
+      const float4 ww = *reinterpret_cast<const float4*>(wc);
+      const float u0 = to_f32<T>(src[0][c]), u1 = to_f32<T>(src[1][c]), u2 = to_f32<T>(src[2][c]), u3 = to_f32<T>(src[3][c]);
+      return fmaf(ww.w, u3, fmaf(ww.z * on[2], u2, fmaf(ww.y * on[1], u1, ww.x * on[0] * u0)));
+    }
+    float acc = 0.f;
+    for (int j = 0; j < taps; ++j) {
+      const int d = taps - 1 - j;
+      float u = 0.f;
+      if (d <= back) u = to_f32<T>(x[(size_t)(t - d) * ld + c]);
+      else if (p >= d) u = to_f32<T>(ring_slot[(size_t)((p - d) % taps) * CH + c]);
+      acc = fmaf(wc[j], u, acc);
+    }
+    return acc;
+  }
+};

@@ -1767,7 +1767,7 @@ def pool_attention_lib(qk_dim: int, v_dim: int, group: int) -> ctypes.CDLL:
                                                  _i, _p, _i, _p, _i, _p]
             lib.dryft_pool_attn_blocks.argtypes = [_i, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _i, _i, _i, _p]
             lib.dryft_pool_attn_rows.argtypes = [_i, _p, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f,
-                                                 _i, _i, _i, _p]
+                                                 _i, _i, _i, _p, _i, _p]
             lib.dryft_pool_attn_prep_tok.argtypes = [_i, _p, _i, _p, _p, _f, _p, _p, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i,
                                                      _f, _i, _p]
             for fn in ("dryft_pool_attn_prep", "dryft_pool_attn_prep_tok", "dryft_pool_attn_blocks", "dryft_pool_attn_rows"):
@@ -1797,7 +1797,7 @@ def pool_attention_prefill_lib(qk_dim: int, v_dim: int, group: int, page: int = 
                                        {"DRYFT_QK_DIM": qk_dim, "DRYFT_V_DIM": v_dim, "DRYFT_GROUP": group, "DRYFT_PAGE": page})
             lib = _load(path)
             lib.dryft_pool_attn_prefill.argtypes = [_p, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f,
-                                                    _i, _i, _i, _p]
+                                                    _i, _i, _i, _p, _i, _p]
             lib.dryft_pool_attn_prefill.restype = _i
             if (lib.dryft_pool_attn_prefill_qk_dim(), lib.dryft_pool_attn_prefill_v_dim()) != (qk_dim, v_dim):
                 raise KernelError("pooled-window prompt attention: the library was built for another head shape")
@@ -1805,11 +1805,17 @@ def pool_attention_prefill_lib(qk_dim: int, v_dim: int, group: int, page: int = 
         return lib
 
 
+def _gate_of(gate, dtype, n: int, cols: int):
+    """Pointer and row stride of optional gate logits."""
+    return (ctypes.c_void_p(0), 0) if gate is None else _rows_of(gate, "gate", dtype, n, cols)
+
+
 def pool_attn_prefill(q, k_pages, v_pages, page_table, pooled, sink, tile_tok0, tile_rows, tok_slot, tok_pos, out, n_tiles: int,
-                      scale: float, size: int, pool: int, keep: int = 0) -> None:
+                      scale: float, size: int, pool: int, keep: int = 0, gate=None) -> None:
     """Prompt attention (bfloat16) of ``q [n, H, D]``, tile by tile of up to 64 tokens of one sequence, over the last ``size``
     cached tokens, the sequence's first ``keep`` tokens and the pooled rows of the blocks of ``pool`` positions wholly before them (``pooled = (pk_pages, pv_pages,
-    pool_table)``; ``pool = 0``: none); the softmax's denominator also holds ``exp(sink[head])`` (if given)."""
+    pool_table)``; ``pool = 0``: none); the softmax's denominator also holds ``exp(sink[head])`` (if given).
+    ``gate [n, H * DV]`` (a column slice is fine): logits whose sigmoids multiply the output value by value."""
     n, n_heads, d = q.shape
     n_kv, page = k_pages.shape[1], k_pages.shape[2]
     dv = v_pages.shape[-1]
@@ -1830,7 +1836,7 @@ def pool_attn_prefill(q, k_pages, v_pages, page_table, pooled, sink, tile_tok0, 
     _ok(lib.dryft_pool_attn_prefill(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1], page, _ptr(pk),
                                     _ptr(pv), _ptr(pt), pt.shape[1] if pt is not None else 0, _ptr(sink), _ptr(tile_tok0),
                                     _ptr(tile_rows), _ptr(tok_slot), _ptr(tok_pos), _ptr(out), int(n_tiles), n_heads, n_kv,
-                                    float(scale), int(size), int(pool), int(keep), _stream()),
+                                    float(scale), int(size), int(pool), int(keep), *_gate_of(gate, q.dtype, n, n_heads * dv), _stream()),
         f"pool_attn_prefill (window {size}, blocks of {pool})")
 
 
@@ -1919,10 +1925,10 @@ def pool_attn_blocks(k_pages, v_pages, page_table, pk_pages, pv_pages, pool_tabl
 
 
 def pool_attn_rows(q, k_pages, v_pages, page_table, pooled, sink, tok_slot, tok_pos, out, scale: float, size: int, pool: int,
-                   n_splits: int = 1, part_o=None, part_ml=None, keep: int = 0) -> None:
+                   n_splits: int = 1, part_o=None, part_ml=None, keep: int = 0, gate=None) -> None:
     """Row-wise attention of ``q [n, H, D]`` over the last ``size`` cached tokens, the sequence's first ``keep`` tokens and, beside them, the pooled row of every block
     of ``pool`` positions that lies wholly before them (``pooled = (pk_pages, pv_pages, pool_table)``; ``pool = 0``: none), one
-    softmax whose denominator also holds ``exp(sink[head])`` (if given).  ``out [n, H, DV]``."""
+    softmax whose denominator also holds ``exp(sink[head])`` (if given).  ``out [n, H, DV]``; ``gate`` as in ``pool_attn_prefill``."""
     n, n_heads, d = q.shape
     n_kv, page = k_pages.shape[1], k_pages.shape[2]
     dv = v_pages.shape[-1]
@@ -1945,7 +1951,7 @@ def pool_attn_rows(q, k_pages, v_pages, page_table, pooled, sink, tok_slot, tok_
     _ok(lib.dryft_pool_attn_rows(_act(q, "q"), _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1], page,
                                  _ptr(pk), _ptr(pv), _ptr(pt), pt.shape[1] if pt is not None else 0, _ptr(sink), _ptr(tok_slot),
                                  _ptr(tok_pos), _ptr(out), _ptr(part_o), _ptr(part_ml), n, n_kv, int(n_splits), float(scale), int(size),
-                                 int(pool), int(keep), _stream()), f"pool_attn_rows (window {size}, blocks of {pool})",
+                                 int(pool), int(keep), *_gate_of(gate, q.dtype, n, n_heads * dv), _stream()), f"pool_attn_rows (window {size}, blocks of {pool})",
         n_kernels=2 if n_splits > 1 else 1)
 
 
@@ -2126,7 +2132,7 @@ def delta_lib() -> ctypes.CDLL:
     return _single_lib("delta", {
         "dryft_delta_prep": [_i, _i, _p, _i, _i, _i, _p, _i, _p, _i, _p, _p, _p, _p, _p, _i, _i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _p],
         "dryft_delta_walk": [_p, _p, _p, _p, _i, _i, _i, _i, _p, _p, _p],
-        "dryft_delta_norm": [_i, _p, _p, _i, _p, _f, _i, _p, _p, _i, _i, _i, _p],
+        "dryft_delta_norm": [_i, _p, _p, _i, _p, _f, _i, _p, _p, _i, _i, _i, _i, _i, _p, _i, _i, _p, _p, _i, _p, _p, _i, _p],
         "dryft_delta_decode": [_i, _i, _p, _i, _i, _i, _p, _i, _p, _i, _p, _i, _p, _p, _p, _p, _f, _i, _p, _p, _i, _i, _i, _i, _i, _p, _p, _p],
     })
 
@@ -2134,6 +2140,11 @@ def delta_lib() -> ctypes.CDLL:
 def delta_state_rows(dim: int) -> int:
     """Floats a value column of the state takes: the key size rounded up to whole 16-byte pieces."""
     return (dim + 3) // 4 * 4
+
+
+def delta_record_dim(dim: int) -> int:
+    """Floats a key vector takes in the walk's records: whole warps of 1, 2, 4 or 8 rows a lane."""
+    return 32 if dim <= 32 else 64 if dim <= 64 else 128 if dim <= 128 else 256
 
 
 def _rows_of(t, name: str, dtype, n: int, cols: int):
@@ -2164,7 +2175,8 @@ def delta_tokens(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, d
                  out, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool) -> None:
     """The gated delta rule over a step of many tokens (``csrc/delta.cu``): records of four tokens each, the walk over them from
     each slot's ``state [slots, H, DV, dp]``, then norm and gate into ``out [n, H*DV]``.  ``ctx``: the step's context (its
-    tiles say which tokens belong together).  Three launches; the convolution's ring is not advanced (``conv_ring_store``)."""
+    tiles say which tokens belong together).  Three launches; the last one also advances the convolution's
+    ``ring``."""
     n, ld, taps, dec_ptr, dec_ld = _delta_common(proj, x_off, b_off, dec, conv_w, ring, a_log, dt_bias, heads, kv_heads, dim, vdim, per_channel)
     dp, dvp = delta_state_rows(dim), (vdim + DELTA_COLS - 1) // DELTA_COLS * DELTA_COLS
     _need(state, "state", torch.float32, (None, heads, vdim, dp))
@@ -2173,7 +2185,7 @@ def delta_tokens(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, d
     gate_ptr, gate_ld = _rows_of(gate, "gate", proj.dtype, n, heads * vdim)
     if ctx.tile_size % 4:
         raise KernelError(f"delta rule: prompt tiles of {ctx.tile_size} tokens (a multiple of 4 is needed)")
-    rec = torch.empty(((n + 3 * ctx.n_seqs) // 4 + 1, heads, 13 * dp + 28), dtype=torch.float32, device=proj.device)
+    rec = torch.empty(((n + 3 * ctx.n_seqs) // 4 + 1, heads, 13 * delta_record_dim(dim) + 28), dtype=torch.float32, device=proj.device)
     vbuf = torch.empty((n, heads, dvp), dtype=torch.float32, device=proj.device)
     o = torch.empty((n, heads * vdim), dtype=torch.float32, device=proj.device)
     lib, bf = delta_lib(), _act(proj, "proj")
@@ -2185,7 +2197,8 @@ def delta_tokens(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, d
     _ok(lib.dryft_delta_walk(_ptr(rec), _ptr(vbuf), _ptr(ctx.cu_q), _ptr(ctx.seq_slot), int(ctx.n_seqs), heads, dim, vdim, _ptr(state),
                              _ptr(o), _stream()), what)
     _ok(lib.dryft_delta_norm(bf, _ptr(o), gate_ptr, gate_ld, _ptr(norm_w), float(eps), int(sigmoid_gate), _ptr(ctx.tok_slot), _ptr(out), n,
-                             heads, vdim, _stream()), what)
+                             heads, kv_heads, dim, vdim, _ptr(proj), ld, int(x_off), _ptr(ctx.cu_q), _ptr(ctx.seq_slot), int(ctx.n_seqs),
+                             _ptr(ctx.tok_pos), _ptr(ring if taps > 1 else None), taps, _stream()), what)
 
 
 def delta_decode(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, dt_bias, norm_w, eps: float, sigmoid_gate: bool, tok_slot,

@@ -122,8 +122,6 @@ class GatedDelta:
         self.conv_w = torch.cat([f32("q_conv"), f32("k_conv"), f32("v_conv")]).contiguous()
         self.a_log, self.dt_bias, self.norm_w = f32("a_log"), f32("dt_bias"), f32("norm")
         K.delta_lib()
-        if self.taps > 1:
-            K.shortconv_lib()
 
     def kv_need(self) -> Optional[KVNeed]:
         return None
@@ -154,6 +152,4 @@ class GatedDelta:
         else:
             K.delta_tokens(proj, 0, self.b_col, dec, gate, self.conv_w, ring, self.a_log, self.dt_bias, self.norm_w, self.eps,
                            self.sigmoid_gate, ctx, state["s"], out, *sizes)
-            if self.taps > 1:
-                K.conv_ring_store(proj, 0, ctx.cu_q, ctx.seq_slot, ctx.tok_pos, ring, ctx.n_seqs)
         return linear(out, self.w_o, self.rt)

@@ -151,8 +151,8 @@ class PooledWindowAttention:
             raise ValueError("pooled_window_attention: the convolution does not go with a norm over the whole projection or the interleaved layout")
         if self.prep_by_token and bias:
             raise ValueError("pooled_window_attention: biases do not go with a norm over the whole projection or the interleaved layout")
-        if self.head_gate or self.value_gate:
-            K.latent_attn_lib()            # the gate kernel lives beside the other gated attention
+        if self.head_gate:
+            K.latent_attn_lib()            # the per-head gate kernel lives beside the other gated attention
         self.rot = int(getattr(self.position, "rotary_dim", 0) or 0) if getattr(self.position, "inv_freq", None) is not None else 0
         K.pool_attention_lib(self.qk_dim, self.v_dim, self.group)   # build (or find) the kernels of this head shape now
         self.use_prefill_kernel = rt.is_bf16 and K.pool_attention_prefill_supported(self.qk_dim, self.v_dim, self.group)
@@ -219,9 +219,10 @@ class PooledWindowAttention:
                 K.pool_attn_blocks(cache.k, cache.v, cache.page_table, pc.k, pc.v, pc.page_table, ctx.tok_slot, ctx.tok_pos, n,
                                    self.pool, self.group)
         o = torch.empty((n, self.n_heads, self.v_dim), dtype=h.dtype, device=dev)
+        gate = proj[:, self.gate_col:self.gate_col + self.o_dim] if self.value_gate else None     # applied inside the attention
         if self.use_prefill_kernel and not ctx.decode and ctx.n_tiles > 0 and cache.k.shape[2] == 64:
             K.pool_attn_prefill(q, cache.k, cache.v, cache.page_table, pooled, self.sink, ctx.tile_tok0, ctx.tile_rows, ctx.tok_slot,
-                                ctx.tok_pos, o, ctx.n_tiles, self.scale, self.size, self.pool, keep=self.keep)
+                                ctx.tok_pos, o, ctx.n_tiles, self.scale, self.size, self.pool, keep=self.keep, gate=gate)
         else:
             s = self._n_splits(n, ctx.max_kv)
             part_o = part_ml = None
@@ -229,10 +230,8 @@ class PooledWindowAttention:
                 part_o = torch.empty((n, self.n_heads, s, self.v_dim), dtype=torch.float32, device=dev)
                 part_ml = torch.empty((n, self.n_heads, s, 2), dtype=torch.float32, device=dev)
             K.pool_attn_rows(q, cache.k, cache.v, cache.page_table, pooled, self.sink, ctx.tok_slot, ctx.tok_pos, o, self.scale,
-                             self.size, self.pool, s, part_o, part_ml, keep=self.keep)
+                             self.size, self.pool, s, part_o, part_ml, keep=self.keep, gate=gate)
         o = o.view(n, self.o_dim)
         if self.head_gate:
             K.head_gate_rows(o, proj, self.gate_col, o, self.n_heads, self.v_dim)     # in place: an entry reads only itself
-        elif self.value_gate:       # a gate per value: every value is a "head" of its own to the same kernel
-            K.head_gate_rows(o, proj, self.gate_col, o, self.o_dim, 1)
         return linear(o, self.w_o, self.rt)
