@@ -165,7 +165,7 @@ def delta_mixer(h: torch.Tensor, p: Mapping, w: Mapping[str, torch.Tensor], pre:
 def side_by_side_mixer(h, p, w, pre, eps):
     left = gated_window_attention(h, p["left"], w, pre + "left.")
     right = delta_mixer(h, p["right"], w, pre + "right.", eps, per_channel=False)
-    return float(p["left_scale"]) * left + float(p["right_scale"]) * right
+    return float(p.get("left_scale", 1.0)) * left + float(p.get("right_scale", 1.0)) * right
 
 
 # ----------------------------------------------------------------------------- feed-forward
@@ -196,7 +196,7 @@ def forward(config: Mapping, weights: Mapping[str, torch.Tensor], tokens: List[i
 
 def _forward(config, weights, tokens, tap):
     w = {k: v.to(F) for k, v in weights.items() if v.is_floating_point()}
-    eps, m = float(config["norm"]["eps"]), float(config["residual_mult"])
+    eps, m = float(config["norm"]["eps"]), float(config.get("residual_mult", 1.0))
     x = w["embed"][torch.tensor(tokens, dtype=torch.long)]
     for run, i in enumerate(run_order(config)):
         layer, pre = config["layers"][i], f"l{i}."
