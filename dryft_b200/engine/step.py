@@ -16,6 +16,8 @@ kernel skips them, so padding changes no result.
 
 from __future__ import annotations
 
+import gc
+from contextlib import contextmanager
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import numpy as np
@@ -199,6 +201,21 @@ class Stepper:
         return logits
 
 
+@contextmanager
+def _capturing(graph: torch.cuda.CUDAGraph):
+    """``torch.cuda.graph`` with the cycle collector held off: an engine dropped earlier (its parts refer to one another) that is
+    collected in the middle of a capture would destroy its own graphs and free its memory there, which CUDA forbids while a
+    stream captures -- and invalidates the capture."""
+    was_on = gc.isenabled()
+    gc.disable()
+    try:
+        with torch.cuda.graph(graph):
+            yield
+    finally:
+        if was_on:
+            gc.enable()
+
+
 class _PromptGraph:
     """A captured prompt step of one shape (its counts and, for models that tell such steps apart, whether every sequence
     starts at position 0): its own copy of the step's integers, its token metadata and the graph.
@@ -219,7 +236,7 @@ class _PromptGraph:
         torch.cuda.synchronize()
         self.graph = torch.cuda.CUDAGraph()
         before = K.launch_count
-        with torch.cuda.graph(self.graph):
+        with _capturing(self.graph):
             self.logits = self.st._run(self.ints, self.meta, self.shape, False, 0)
         self.n_kernels = K.launch_count - before
 
@@ -311,7 +328,7 @@ class _DecodeGraph:
             torch.cuda.synchronize()
             self.graph = torch.cuda.CUDAGraph()
             before = K.launch_count
-            with torch.cuda.graph(self.graph):
+            with _capturing(self.graph):
                 self.logits = self._body()
             self.n_kernels = K.launch_count - before
             self.seq_slot.copy_(host, non_blocking=True)
