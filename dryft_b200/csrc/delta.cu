@@ -16,21 +16,23 @@
 // columns, and the sums over the key channels are warp sums.  Decays are applied as S + S * (g - 1) with g - 1 = expm1(log g):
 // a decay close to one keeps its distance from one.
 //
-// A step of many tokens goes by quads of four tokens.  With G_i the sum of the log decays of a quad's tokens 0..i,
+// A step of many tokens goes by groups of eight tokens.  With G_i the sum of the log decays of a group's tokens 0..i,
 //
 //     u_i = beta_i (v_i - (k_i e^{G_i})^T S0) - sum_{j<i} beta_i A_ij u_j ,    A_ij = sum_c k_i k_j e^{G_i - G_j}
 //     o_i = (q_i e^{G_i})^T S0 + sum_{j<=i} P_ij u_j ,                         P_ij = sum_c q_i k_j e^{G_i - G_j}
-//     S4  = e^{G_3} S0 + sum_j (k_j e^{G_3 - G_j}) u_j^T
+//     S8  = e^{G_7} S0 + sum_j (k_j e^{G_7 - G_j}) u_j^T
 //
-// so the eight products with S0 of a quad do not wait for one another and their warp sums are formed together; every exponent
-// is a sum of log decays, hence never positive.
+// so the sixteen products with S0 of a group do not wait for one another and their warp sums are formed together; every
+// exponent is a sum of log decays, hence never positive.
 //
-//   delta_prep    one block per (tile of a sequence's tokens, head): a warp a quad; leaves a record per (quad, head):
-//                 [beta_i k_i e^{G_i}: 4 dp | q_i e^{G_i}: 4 dp | k_j e^{G_3-G_j}: 4 dp | expm1(G_3): dp | beta 4 |
-//                 beta_i A_ij: 6 (+2) | P: 4 x 4].  Further blocks convolve v into [n, H, dvp] floats.
-//   delta_walk    one block per (16 value columns, head, sequence), a warp four columns: quads in order from the slot's state,
-//                 records and v brought to shared memory a few quads ahead by cp.async; the 32 sums of a warp and quad are
-//                 formed by one butterfly that leaves lane l with sum l.  Leaves o [n, H*dv] and the slot's state.
+//   delta_prep    one block per (tile of a sequence's tokens, head): a warp a group; leaves a record per (group, head), vectors
+//                 of dr = 32, 64, 128 or 256 floats (the key size rounded up, zeros behind it):
+//                 [beta_i k_i e^{G_i}: 8 dr | q_i e^{G_i}: 8 dr | k_j e^{G_7-G_j}: 8 dr | expm1(G_7): dr | beta 8 |
+//                 beta_i A_ij: 28 | P: 8 x 8].  Further blocks convolve v into [n, H, dvp] floats.
+//   delta_walk    one block per (slice of value columns, head, sequence), the columns dealt to its warps: groups in order from
+//                 the slot's state, records and v brought to shared memory ahead by cp.async; the sums of a warp and
+//                 group are formed by one butterfly that leaves every lane one or two of them.  Leaves o [n, H*dv] and the
+//                 slot's state.
 //   delta_norm    one warp per (token, head): the norm over dv, the weight and the gate.  Further blocks store the convolution's
 //                 last inputs in the ring (this launch runs behind the one that reads it).
 //   delta_decode  one token per sequence: one block per (head, sequence) does all of it, the ring's new row included.
@@ -41,14 +43,16 @@
 
 namespace {
 constexpr float UNIT_EPS = 1e-6f;     // inside the root of the unit vectors' length: fixed by the rule
-constexpr int QUAD = 4;
-constexpr int PREP_THREADS = 256;
-constexpr int V_SPLIT = 4;            // blocks a tile's quads are dealt to while v is convolved
+constexpr int GRP = 8;                // tokens of a group
+constexpr int PAIRS = GRP * (GRP - 1) / 2;
+constexpr int VECS = 3 * GRP + 1;     // vectors of a record
+constexpr int SCAL = GRP + PAIRS + GRP * GRP;   // numbers behind them
+constexpr int PREP_THREADS = 128;
+constexpr int V_SPLIT = 4;            // blocks a tile's groups are dealt to while v is convolved
 constexpr int WALK_WARPS = 4;
-constexpr int WALK_STAGES = 4;        // quads of the walk in shared memory at once
+constexpr int WALK_STAGES = 4;        // records of the walk in shared memory at once
 constexpr long long FEW_COLUMNS = 8 * 148;
 constexpr int V_PAD = 16;             // rows of the convolved v are padded to whole blocks of columns
-constexpr int SCAL = 28;              // numbers of a record behind its vectors
 constexpr int DEC_COLS = 8;           // value columns a warp of the decode kernel holds at once
 constexpr int DEC_THREADS = 512;
 constexpr unsigned FULL = 0xffffffffu;
@@ -91,8 +95,8 @@ __device__ __forceinline__ int seq_of(const int* __restrict__ cu_q, int n_seqs, 
   return lo;
 }
 
-// the first quad's record of sequence b whose first packed token is t0: sequences take disjoint ranges in order
-__device__ __forceinline__ size_t quad_base(int t0, int b) { return (size_t)((t0 + 3 * b) / QUAD); }
+// the first group's record of sequence b whose first packed token is t0: sequences take disjoint ranges in order
+__device__ __forceinline__ size_t group_base(int t0, int b) { return (size_t)(((long long)t0 + (long long)(GRP - 1) * b) / GRP); }
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -132,33 +136,37 @@ __device__ __forceinline__ void store_rows(const float (&v)[RPL], float* p, int 
   }
 }
 
-// x[i] summed over the warp, i < N (a power of two up to 32); lane l is left with the sum of index l / (32 / N)
-template <int N>
-__device__ __forceinline__ float butterfly(float (&x)[N], int lane) {
-  int off = 16;
+// x[i] summed over the L lanes of a group, i < N (powers of two): lane l of the group is left with the sums of index
+// l * N / L .. in x[0 .. N / L - 1] (N >= L), or with the sum of index l / (L / N) in x[0]
+template <int N, int L>
+__device__ __forceinline__ void butterfly(float (&x)[N], int l) {
+  int n = N;
 #pragma unroll
-  for (int n = N / 2; n > 0; n >>= 1, off >>= 1) {
-    const bool up = (lane & off) != 0;
+  for (int off = L / 2; off > 0; off >>= 1) {
+    if (n > 1) {
+      n >>= 1;
+      const bool up = (l & off) != 0;
 #pragma unroll
-    for (int i = 0; i < N / 2; ++i) {
-      if (i < n) {
-        const float send = up ? x[i] : x[i + n], keep = up ? x[i + n] : x[i];
-        x[i] = keep + __shfl_xor_sync(FULL, send, off);
+      for (int i = 0; i < N / 2; ++i) {
+        if (i < n) {
+          const float send = up ? x[i] : x[i + n], keep = up ? x[i + n] : x[i];
+          x[i] = keep + __shfl_xor_sync(FULL, send, off);
+        }
       }
+    } else {
+      x[0] += __shfl_xor_sync(FULL, x[0], off);
     }
   }
-  float r = x[0];
-  for (; off > 0; off >>= 1) r += __shfl_xor_sync(FULL, r, off);
-  return r;
 }
 
-template <typename T, int DR, bool CHAN>
-__global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
+template <typename T, bool CHAN>
+__global__ void __launch_bounds__(PREP_THREADS, 3) delta_prep_kernel(
     const T* __restrict__ proj, int ld, int x_off, int b_off, const T* __restrict__ dec, int dec_ld, const float* __restrict__ conv_w,
     int taps, const T* __restrict__ ring, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
     const int* __restrict__ tile_tok0, const int* __restrict__ tile_rows, const int* __restrict__ cu_q, int n_seqs,
-    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, int H, int G, int d, int dv, int dvp,
+    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, int H, int G, int d, int dv, int dr, int dvp,
     float* __restrict__ rec, float* __restrict__ vbuf) {
+  extern __shared__ float own[];      // per warp: q, k and log decays of a group, [3][GRP][dr]; every lane reads what it wrote
   const int tile = blockIdx.x;
   const int tok0 = tile_tok0[tile], rows = tile_rows[tile];
   const int slot = tok_slot[tok0];
@@ -167,19 +175,21 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
   const int t0 = cu_q[b], n = cu_q[b + 1] - t0, p0 = tok_pos[t0], i_tile = tok0 - t0;
   const T* x = proj + x_off;
   const int CH = 2 * G * d + H * dv;
-  const int nq = (rows + QUAD - 1) / QUAD;
+  const int ng = (rows + GRP - 1) / GRP;
 
   if ((int)blockIdx.y >= H) {      // v: a thread a column of [H, dvp]
     const int part = (int)blockIdx.y - H;
     const int col = (part / V_SPLIT) * PREP_THREADS + threadIdx.x;
     if (col >= H * dvp) return;
     const int h = col / dvp, c = col % dvp;
-    for (int qd = part % V_SPLIT; qd < nq; qd += V_SPLIT) {
-      const int i0 = i_tile + qd * QUAD;
-      float acc[4] = {0.f, 0.f, 0.f, 0.f};
-      if (c < dv) conv4<T>(acc, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, 2 * G * d + h * dv + c);
+    for (int gi = part % V_SPLIT; gi < ng; gi += V_SPLIT) {
+      const int i0 = i_tile + gi * GRP;
+      float acc[GRP];
 #pragma unroll
-      for (int k = 0; k < QUAD; ++k)
+      for (int k = 0; k < GRP; ++k) acc[k] = 0.f;
+      if (c < dv) conv_run<T, GRP>(acc, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, 2 * G * d + h * dv + c);
+#pragma unroll
+      for (int k = 0; k < GRP; ++k)
         if (i0 + k < n) vbuf[(size_t)(t0 + i0 + k) * H * dvp + col] = c < dv ? siluf_(acc[k]) : 0.f;
     }
     return;
@@ -188,103 +198,108 @@ __global__ void __launch_bounds__(PREP_THREADS) delta_prep_kernel(
   const int h = blockIdx.y, g = h / (H / G);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float rate = -LOG2E * expf(a_log[h]);      // log decays in powers of two
-  constexpr int dr = 32 * DR;      // a record's vectors are padded with zeros to whole warps
-  constexpr size_t RS = (size_t)13 * dr + SCAL;
-  for (int qd = warp; qd < nq; qd += PREP_THREADS / 32) {
-    const int i0 = i_tile + qd * QUAD, m = min(QUAD, n - i0);
-    float q[QUAD][DR], k[QUAD][DR], lg[QUAD][DR];
-    float sq[QUAD] = {0.f, 0.f, 0.f, 0.f}, sk[QUAD] = {0.f, 0.f, 0.f, 0.f};
-    float head_lg[QUAD];
-    if (!CHAN) {
-#pragma unroll
-      for (int i = 0; i < QUAD; ++i)
-        head_lg[i] = i < m ? rate * softplusf_(to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h]) + dt_bias[h]) : 0.f;
+  const size_t RS = (size_t)VECS * dr + SCAL;
+  float* qs = own + (size_t)warp * 3 * GRP * dr;
+  float *ks = qs + GRP * dr, *ls = ks + GRP * dr;
+  for (int gi = warp; gi < ng; gi += PREP_THREADS / 32) {
+    const int i0 = i_tile + gi * GRP, m = min(GRP, n - i0);
+    // lane i < GRP: beta of token i, and its log decay where there is one per head
+    float beta = 0.f, head_lg = 0.f;
+    if (lane < m) {
+      beta = sigmoidf_(to_f32<T>(proj[(size_t)(t0 + i0 + lane) * ld + b_off + h]));
+      if (!CHAN) head_lg = rate * softplusf_(to_f32<T>(dec[(size_t)(t0 + i0 + lane) * dec_ld + h]) + dt_bias[h]);
     }
-    float z[QUAD][DR];                 // the decays' pre-activations, requested first
-    if (CHAN) {
+    float ss[2 * GRP];        // sums of squares: q of each token, then k
 #pragma unroll
-      for (int i = 0; i < QUAD; ++i)
+    for (int i = 0; i < 2 * GRP; ++i) ss[i] = 0.f;
+    for (int c = lane; c < dr; c += 32) {
+      float aq[GRP], ak[GRP], z[GRP];
 #pragma unroll
-        for (int r = 0; r < DR; ++r) {
-          const int c = lane + 32 * r;
-          z[i][r] = c < d && i < m ? to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h * d + c]) : 0.f;
-        }
-    }
-#pragma unroll
-    for (int r = 0; r < DR; ++r) {
-      const int c = lane + 32 * r;
-      float aq[4] = {0.f, 0.f, 0.f, 0.f}, ak[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int i = 0; i < GRP; ++i) aq[i] = ak[i] = z[i] = 0.f;
       if (c < d) {
-        conv4<T>(aq, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, g * d + c);
-        conv4<T>(ak, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, (G + g) * d + c);
+        if (CHAN) {
+#pragma unroll
+          for (int i = 0; i < GRP; ++i)
+            if (i < m) z[i] = to_f32<T>(dec[(size_t)(t0 + i0 + i) * dec_ld + h * d + c]);
+        }
+        conv_run<T, GRP>(aq, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, g * d + c);
+        conv_run<T, GRP>(ak, conv_w, x, ld, ring, taps, CH, slot, t0, p0, i0, n, (G + g) * d + c);
       }
-#pragma unroll
-      for (int i = 0; i < QUAD; ++i) { q[i][r] = aq[i]; k[i][r] = ak[i]; }
-    }
-#pragma unroll
-    for (int r = 0; r < DR; ++r) {
-      const int c = lane + 32 * r;
       const float bias = CHAN && c < d ? dt_bias[h * d + c] : 0.f;
 #pragma unroll
-      for (int i = 0; i < QUAD; ++i) {
+      for (int i = 0; i < GRP; ++i) {
         const bool on = c < d && i < m;
-        q[i][r] = on ? siluf_(q[i][r]) : 0.f;
-        k[i][r] = on ? siluf_(k[i][r]) : 0.f;
-        sq[i] = fmaf(q[i][r], q[i][r], sq[i]);
-        sk[i] = fmaf(k[i][r], k[i][r], sk[i]);
-        if (CHAN) lg[i][r] = on ? rate * softplusf_(z[i][r] + bias) : 0.f;
-        else lg[i][r] = head_lg[i];
+        const float qv = on ? siluf_(aq[i]) : 0.f, kv = on ? siluf_(ak[i]) : 0.f;
+        ss[i] = fmaf(qv, qv, ss[i]);
+        ss[GRP + i] = fmaf(kv, kv, ss[GRP + i]);
+        qs[i * dr + c] = qv;
+        ks[i * dr + c] = kv;
+        if (CHAN) ls[i * dr + c] = on ? rate * softplusf_(z[i] + bias) : 0.f;
       }
     }
-    const float qscale = 1.f / sqrtf((float)d);
-    float beta[QUAD];
+    butterfly<2 * GRP, 32>(ss, lane);      // lane l: sum l / 2
+    const float len = (lane < 16 ? 1.f / sqrtf((float)d) : 1.f) / sqrtf(ss[0] + UNIT_EPS);
+    float rq[GRP], rk[GRP], be[GRP], hl[GRP];
 #pragma unroll
-    for (int i = 0; i < QUAD; ++i) {
-      const float rq = qscale / sqrtf(warp_sum(sq[i]) + UNIT_EPS), rk = 1.f / sqrtf(warp_sum(sk[i]) + UNIT_EPS);
-      beta[i] = i < m ? sigmoidf_(to_f32<T>(proj[(size_t)(t0 + i0 + i) * ld + b_off + h])) : 0.f;
-#pragma unroll
-      for (int r = 0; r < DR; ++r) { q[i][r] *= rq; k[i][r] *= rk; }
+    for (int i = 0; i < GRP; ++i) {
+      rq[i] = __shfl_sync(FULL, len, 2 * i);
+      rk[i] = __shfl_sync(FULL, len, 16 + 2 * i);
+      be[i] = __shfl_sync(FULL, beta, i);
+      hl[i] = CHAN ? 0.f : __shfl_sync(FULL, head_lg, i);
     }
-    float A[6] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f};      // (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
-    float P[10] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};   // (0,0) (1,0) (1,1) (2,0) ...
-    float* rc = rec + ((quad_base(t0, b) + (size_t)(i0 / QUAD)) * H + h) * RS;
+    float sums[64];           // A_ij (i(i-1)/2 + j), then P_ij (i(i+1)/2 + j)
 #pragma unroll
-    for (int r = 0; r < DR; ++r) {
-      const int c = lane + 32 * r;
-      const float l1 = lg[1][r], l2 = lg[2][r], l3 = lg[3][r];
-      const float g0 = lg[0][r], g1 = g0 + l1, g2 = g1 + l2, g3 = g2 + l3;
-      // decays from token j to token i of the quad: sums of the log decays in between, so e^0 = 1 where nothing decays
-      const float e10 = exp2_(l1), e21 = exp2_(l2), e20 = exp2_(l1 + l2), e32 = exp2_(l3), e31 = exp2_(l2 + l3), e30 = exp2_(l1 + l2 + l3);
-      A[0] = fmaf(k[1][r] * k[0][r], e10, A[0]);
-      A[1] = fmaf(k[2][r] * k[0][r], e20, A[1]); A[2] = fmaf(k[2][r] * k[1][r], e21, A[2]);
-      A[3] = fmaf(k[3][r] * k[0][r], e30, A[3]); A[4] = fmaf(k[3][r] * k[1][r], e31, A[4]); A[5] = fmaf(k[3][r] * k[2][r], e32, A[5]);
-      P[0] = fmaf(q[0][r], k[0][r], P[0]);
-      P[1] = fmaf(q[1][r] * k[0][r], e10, P[1]); P[2] = fmaf(q[1][r], k[1][r], P[2]);
-      P[3] = fmaf(q[2][r] * k[0][r], e20, P[3]); P[4] = fmaf(q[2][r] * k[1][r], e21, P[4]); P[5] = fmaf(q[2][r], k[2][r], P[5]);
-      P[6] = fmaf(q[3][r] * k[0][r], e30, P[6]); P[7] = fmaf(q[3][r] * k[1][r], e31, P[7]);
-      P[8] = fmaf(q[3][r] * k[2][r], e32, P[8]); P[9] = fmaf(q[3][r], k[3][r], P[9]);
-      {
-        const float x0 = exp2_(g0), x1 = exp2_(g1), x2 = exp2_(g2), x3 = exp2_(g3);
-        rc[c] = beta[0] * k[0][r] * x0; rc[dr + c] = beta[1] * k[1][r] * x1;
-        rc[2 * dr + c] = beta[2] * k[2][r] * x2; rc[3 * dr + c] = beta[3] * k[3][r] * x3;
-        rc[4 * dr + c] = q[0][r] * x0; rc[5 * dr + c] = q[1][r] * x1; rc[6 * dr + c] = q[2][r] * x2; rc[7 * dr + c] = q[3][r] * x3;
-        rc[8 * dr + c] = k[0][r] * e30; rc[9 * dr + c] = k[1][r] * e31; rc[10 * dr + c] = k[2][r] * e32; rc[11 * dr + c] = k[3][r];
-        rc[12 * dr + c] = c < d ? expm1f(LN2 * g3) : 0.f;
+    for (int i = 0; i < 64; ++i) sums[i] = 0.f;
+    float* rc = rec + ((group_base(t0, b) + (size_t)(i0 / GRP)) * H + h) * RS;
+    for (int c = lane; c < dr; c += 32) {
+      float q[GRP], k[GRP], l[GRP];
+#pragma unroll
+      for (int i = 0; i < GRP; ++i) {
+        q[i] = qs[i * dr + c] * rq[i];
+        k[i] = ks[i * dr + c] * rk[i];
+        l[i] = CHAN ? ls[i * dr + c] : hl[i];
       }
+      float cum = 0.f;
+#pragma unroll
+      for (int i = 0; i < GRP; ++i) {
+        cum += l[i];
+        const float e = exp2_(cum);
+        rc[i * dr + c] = be[i] * k[i] * e;
+        rc[(GRP + i) * dr + c] = q[i] * e;
+      }
+      rc[3 * GRP * dr + c] = c < d ? expm1f(LN2 * cum) : 0.f;
+#pragma unroll
+      for (int i = 0; i < GRP; ++i) {
+        float* P = sums + PAIRS + i * (i + 1) / 2;
+        P[i] = fmaf(q[i], k[i], P[i]);
+        float s = 0.f;          // from token j to token i: the log decays in between
+#pragma unroll
+        for (int j = i - 1; j >= 0; --j) {
+          s += l[j + 1];
+          const float t = k[j] * exp2_(s);
+          sums[i * (i - 1) / 2 + j] = fmaf(k[i], t, sums[i * (i - 1) / 2 + j]);
+          P[j] = fmaf(q[i], t, P[j]);
+          if (i == GRP - 1) rc[(2 * GRP + j) * dr + c] = t;
+        }
+      }
+      rc[(3 * GRP - 1) * dr + c] = k[GRP - 1];
     }
+    butterfly<64, 32>(sums, lane);         // lane l: sums 2 l and 2 l + 1
+    float* sc = rc + (size_t)VECS * dr;
+    if (lane < GRP) sc[lane] = beta;
 #pragma unroll
-    for (int i = 0; i < 6; ++i) A[i] = warp_sum(A[i]);
-#pragma unroll
-    for (int i = 0; i < 10; ++i) P[i] = warp_sum(P[i]);
-    if (lane == 0) {
-      float4* s = reinterpret_cast<float4*>(rc + 13 * dr);
-      s[0] = make_float4(beta[0], beta[1], beta[2], beta[3]);
-      s[1] = make_float4(beta[1] * A[0], beta[2] * A[1], beta[2] * A[2], beta[3] * A[3]);
-      s[2] = make_float4(beta[3] * A[4], beta[3] * A[5], 0.f, 0.f);
-      s[3] = make_float4(P[0], 0.f, 0.f, 0.f);
-      s[4] = make_float4(P[1], P[2], 0.f, 0.f);
-      s[5] = make_float4(P[3], P[4], P[5], 0.f);
-      s[6] = make_float4(P[6], P[7], P[8], P[9]);
+    for (int e = 0; e < 2; ++e) {
+      const int idx = 2 * lane + e, p = idx < PAIRS ? idx : idx - PAIRS;
+      int i = 0;
+      while ((idx < PAIRS ? i * (i + 1) : (i + 1) * (i + 2)) / 2 <= p) ++i;      // the row of the triangle
+      const int j = p - (idx < PAIRS ? i * (i - 1) : i * (i + 1)) / 2;
+      const float bi = __shfl_sync(FULL, beta, i);
+      if (idx < PAIRS) {
+        sc[GRP + idx] = bi * sums[e];
+        sc[GRP + PAIRS + j * GRP + i] = 0.f;            // P above its diagonal
+      } else {
+        sc[GRP + PAIRS + i * GRP + j] = sums[e];
+      }
     }
   }
 }
@@ -312,35 +327,36 @@ __device__ __forceinline__ float sum2(pair_t a) {
   return lo + hi;
 }
 
-// A group of L lanes owns CPG value columns; lane l of the group holds the rows 4 (l + L m) .. + 3 for m < RPL / 4 (vectors of
-// 16 bytes, neighbouring lanes side by side).  Records hold vectors of L * RPL floats, so no lane needs a bound.
+// L lanes share CPG value columns; lane l of them holds the rows 4 (l + L m) .. + 3 for m < RPL / 4 (vectors of 16 bytes,
+// neighbouring lanes side by side).  Records hold vectors of L * RPL floats, so no lane needs a bound.
 template <int L, int RPL, int CPG>
 __global__ void __launch_bounds__(WALK_WARPS * 32) delta_walk_kernel(
     const float* __restrict__ rec, const float* __restrict__ vbuf, const int* __restrict__ cu_q, const int* __restrict__ seq_slot,
     int H, int dv, int dp, int dvp, float* __restrict__ state, float* __restrict__ o) {
-  constexpr int DR = L * RPL, RS = 13 * DR + SCAL;
+  constexpr int DR = L * RPL, RS = VECS * DR + SCAL;
   constexpr int COLS = WALK_WARPS * (32 / L) * CPG;         // value columns of the block
-  constexpr int NV = QUAD * COLS / 4;                       // 16-byte pieces of a quad's v
-  constexpr int STAGE = RS + QUAD * COLS;
+  constexpr int NV = GRP * COLS / 4;                        // 16-byte pieces of a group's v
+  constexpr int STAGE = RS + GRP * COLS;
   constexpr int NST = WALK_STAGES;
-  constexpr int VALS = 8 * CPG, DUP = L / VALS;             // sums a group forms; lanes that end up with the same one
+  constexpr int VALS = 2 * GRP * CPG, NPL = VALS / L;       // sums L lanes form, sums a lane is left with
   constexpr int THREADS = WALK_WARPS * 32;
-  static_assert(VALS <= L, "a lane is left with one sum");
+  static_assert(VALS >= L && NV <= THREADS, "every lane is left with a sum; a thread a piece of v");
   extern __shared__ __align__(16) float stage_mem[];
+  __shared__ __align__(16) float ksum[WALK_WARPS][32 / L][GRP * CPG];
   const int b = blockIdx.z, h = blockIdx.y;
   const int slot = seq_slot[b];
   const int t0 = cu_q[b], n = cu_q[b + 1] - t0;
   if (slot < 0 || n <= 0) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gl = lane % L;
   const int blk0 = blockIdx.x * COLS, lcol = (warp * (32 / L) + lane / L) * CPG, col0 = blk0 + lcol;
-  const int nq = (n + QUAD - 1) / QUAD;
-  const float* rc0 = rec + (quad_base(t0, b) * H + h) * (size_t)RS;
+  const int ng = (n + GRP - 1) / GRP;
+  const float* rc0 = rec + (group_base(t0, b) * H + h) * (size_t)RS;
   const size_t rstep = (size_t)H * RS;
   const float* v0 = vbuf + (size_t)t0 * H * dvp + (size_t)h * dvp + blk0;
   const size_t vstep = (size_t)H * dvp;
 
-  auto issue = [&](int j) {      // record and v rows of quad j -> its stage
-    if (j < nq) {
+  auto issue = [&](int j) {      // record and v rows of group j -> its stage
+    if (j < ng) {
       float* sm = stage_mem + (j % NST) * STAGE;
       const float* src = rc0 + (size_t)j * rstep;
 #pragma unroll
@@ -350,7 +366,7 @@ __global__ void __launch_bounds__(WALK_WARPS * 32) delta_walk_kernel(
       }
       if (tid < NV) {
         const int r = tid / (COLS / 4), c = (tid % (COLS / 4)) * 4;
-        const int t = min(j * QUAD + r, n - 1);      // a quad's missing tokens have beta = 0: any finite row will do
+        const int t = min(j * GRP + r, n - 1);      // a group's missing tokens have beta = 0: any finite row will do
         cp_async16(sm + RS + r * COLS + c, v0 + (size_t)t * vstep + c);
       }
     }
@@ -371,27 +387,29 @@ __global__ void __launch_bounds__(WALK_WARPS * 32) delta_walk_kernel(
       S[c][2 * m] = x.x;
       S[c][2 * m + 1] = x.y;
     }
+  // the sums this lane is left with: index -> (token, or GRP + token for the query; column)
+  const int tok0 = gl * NPL / CPG;
+  float* op = o + (size_t)t0 * H * dv + (size_t)h * dv + col0;
 
-  const int id = gl / DUP, o_tok = id / CPG & 3, o_col = id % CPG;
-  const bool o_on = id >= 4 * CPG && gl % DUP == 0 && col0 + o_col < dv;
-  float* op = o + (size_t)(t0 + o_tok) * H * dv + (size_t)h * dv + col0 + o_col;
-
-  for (int j = 0; j < nq; ++j) {
+  for (int j = 0; j < ng; ++j) {
     cp_async_wait<NST - 2>();
-    __syncthreads();               // quad j is in shared memory; everyone is done with quad j - 1
+    __syncthreads();               // group j is in shared memory; everyone is done with group j - 1
     issue(j + NST - 1);
     const float* sm = stage_mem + (j % NST) * STAGE;
     const float* vec = sm + 4 * gl;
-    float x[VALS];                 // index: (token, or 4 + token for the query) * CPG + column
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      pair_t kt[RPL / 2];
+    auto rows = [&](pair_t (&r)[RPL / 2], int i) {
 #pragma unroll
       for (int m = 0; m < RPL / 4; ++m) {
         const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(vec + i * DR + 4 * L * m);
-        kt[2 * m] = t.x;
-        kt[2 * m + 1] = t.y;
+        r[2 * m] = t.x;
+        r[2 * m + 1] = t.y;
       }
+    };
+    float x[VALS];
+#pragma unroll
+    for (int i = 0; i < 2 * GRP; ++i) {
+      pair_t kt[RPL / 2];
+      rows(kt, i);
 #pragma unroll
       for (int c = 0; c < CPG; ++c) {
         pair_t a = mul2(kt[0], S[c][0]);
@@ -400,80 +418,59 @@ __global__ void __launch_bounds__(WALK_WARPS * 32) delta_walk_kernel(
         x[i * CPG + c] = sum2(a);
       }
     }
-    // one butterfly over the group: lane gl is left with the sum of index gl / DUP
-    {
-      int off = L / 2;
+    // what the update will read is on its way while the sums are formed
+    pair_t gm[RPL / 2], kb[GRP][RPL / 2];
+    rows(gm, 3 * GRP);
 #pragma unroll
-      for (int m = VALS / 2; m > 0; m >>= 1, off >>= 1) {
-        const bool up = (gl & off) != 0;
+    for (int i = 0; i < GRP; ++i) rows(kb[i], 2 * GRP + i);
+    butterfly<VALS, L>(x, gl);
+    if (tok0 < GRP) {
 #pragma unroll
-        for (int i = 0; i < VALS / 2; ++i) {
-          if (i < m) {
-            const float send = up ? x[i] : x[i + m], keep = up ? x[i + m] : x[i];
-            x[i] = keep + __shfl_xor_sync(FULL, send, off);
-          }
-        }
-      }
-#pragma unroll
-      for (int w = DUP / 2; w > 0; w >>= 1) x[0] += __shfl_xor_sync(FULL, x[0], w);
+      for (int e = 0; e < NPL; ++e) ksum[warp][lane / L][gl * NPL + e] = x[e];
     }
-    const float mine = x[0];
-    const float* sc = sm + 13 * DR;
-    const float4 be = *reinterpret_cast<const float4*>(sc), a0 = *reinterpret_cast<const float4*>(sc + 4),
-                 a1 = *reinterpret_cast<const float4*>(sc + 8);
-    const float bi[4] = {be.x, be.y, be.z, be.w};
-    const float A[6] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y};
-    float u[QUAD][CPG];
+    __syncwarp();
+    const float* sc = sm + VECS * DR;
+    const float* ksm = ksum[warp][lane / L];
+    float u[GRP][CPG];
 #pragma unroll
-    for (int i = 0; i < QUAD; ++i)
+    for (int i = 0; i < GRP; ++i) {
 #pragma unroll
-      for (int c = 0; c < CPG; ++c) {
-        const float dk = __shfl_sync(FULL, mine, (i * CPG + c) * DUP, L);
-        u[i][c] = fmaf(bi[i], sm[RS + i * COLS + lcol + c], -dk);
+      for (int c = 0; c < CPG; ++c) u[i][c] = fmaf(sc[i], sm[RS + i * COLS + lcol + c], -ksm[i * CPG + c]);
 #pragma unroll
-        for (int jj = 0; jj < i; ++jj) u[i][c] = fmaf(-A[i * (i - 1) / 2 + jj], u[jj][c], u[i][c]);
+      for (int jj = 0; jj < i; ++jj) {
+        const float a = sc[GRP + i * (i - 1) / 2 + jj];
+#pragma unroll
+        for (int c = 0; c < CPG; ++c) u[i][c] = fmaf(-a, u[jj][c], u[i][c]);
       }
-    {
-      pair_t gm[RPL / 2];
-#pragma unroll
-      for (int m = 0; m < RPL / 4; ++m) {
-        const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(vec + 12 * DR + 4 * L * m);
-        gm[2 * m] = t.x;
-        gm[2 * m + 1] = t.y;
-      }
-#pragma unroll
-      for (int c = 0; c < CPG; ++c)
-#pragma unroll
-        for (int r = 0; r < RPL / 2; ++r) S[c][r] = fma2(S[c][r], gm[r], S[c][r]);
     }
 #pragma unroll
-    for (int i = 0; i < QUAD; ++i) {
-      pair_t kb[RPL / 2];
+    for (int c = 0; c < CPG; ++c)
 #pragma unroll
-      for (int m = 0; m < RPL / 4; ++m) {
-        const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(vec + (8 + i) * DR + 4 * L * m);
-        kb[2 * m] = t.x;
-        kb[2 * m + 1] = t.y;
-      }
+      for (int r = 0; r < RPL / 2; ++r) S[c][r] = fma2(S[c][r], gm[r], S[c][r]);
+#pragma unroll
+    for (int i = 0; i < GRP; ++i) {
 #pragma unroll
       for (int c = 0; c < CPG; ++c) {
         const pair_t uu = pack2(u[i][c], u[i][c]);
 #pragma unroll
-        for (int r = 0; r < RPL / 2; ++r) S[c][r] = fma2(kb[r], uu, S[c][r]);
+        for (int r = 0; r < RPL / 2; ++r) S[c][r] = fma2(kb[i][r], uu, S[c][r]);
       }
     }
-    {      // the lanes that hold a query's sum finish its output
-      const float4 Pr = *reinterpret_cast<const float4*>(sc + 12 + o_tok * 4);
-      const float pr[4] = {Pr.x, Pr.y, Pr.z, Pr.w};
-      float val = mine;
+    // the lanes that hold queries' sums finish their outputs
 #pragma unroll
-      for (int jj = 0; jj < QUAD; ++jj) {
+    for (int e = 0; e < NPL; ++e) {
+      const int idx = gl * NPL + e, i = (idx / CPG) % GRP, oc = idx % CPG;
+      const float* pr = sc + GRP + PAIRS + i * GRP;
+      float val = x[e];
+#pragma unroll
+      for (int jj = 0; jj < GRP; ++jj) {
         float uc = u[jj][0];
 #pragma unroll
-        for (int cc = 1; cc < CPG; ++cc) uc = o_col == cc ? u[jj][cc] : uc;
+        for (int cc = 1; cc < CPG; ++cc) uc = oc == cc ? u[jj][cc] : uc;
         val = fmaf(pr[jj], uc, val);
       }
-      if (o_on && j * QUAD + o_tok < n) op[(size_t)j * QUAD * H * dv] = val;
+      const int t = j * GRP + i;
+      if (idx >= GRP * CPG && t < n && col0 + oc < dv) op[(size_t)t * H * dv + oc] = val;
     }
   }
   cp_async_wait<0>();
@@ -635,7 +632,8 @@ __global__ void __launch_bounds__(DEC_THREADS) delta_decode_kernel(
       xs[c] = a;
       xs[DEC_COLS + c] = q;
     }
-    const float mine = butterfly<2 * DEC_COLS>(xs, lane);    // lane l: sum l / 2 (key sums of the eight columns, then query sums)
+    butterfly<2 * DEC_COLS, 32>(xs, lane);
+    const float mine = xs[0];                                // lane l: sum l / 2 (key sums of the eight columns, then query sums)
     const int id = lane >> 1, c_own = id & (DEC_COLS - 1), col = base + c_own;
     const float uval = col < dv ? beta * (vs[col] - mine) : 0.f;
     const float u_own = __shfl_sync(FULL, uval, 2 * c_own);
@@ -658,17 +656,22 @@ __global__ void __launch_bounds__(DEC_THREADS) delta_decode_kernel(
   }
 }
 
-template <typename T, int DR, bool CHAN>
+template <typename T, bool CHAN>
 int prep_launch(const void* proj, int ld, int x_off, int b_off, const void* dec, int dec_ld, const float* conv_w, int taps,
                 const void* ring, const float* a_log, const float* dt_bias, const int* tile_tok0, const int* tile_rows, int n_tiles,
-                const int* cu_q, int n_seqs, const int* tok_slot, const int* tok_pos, int H, int G, int d, int dv, int dvp,
+                const int* cu_q, int n_seqs, const int* tok_slot, const int* tok_pos, int H, int G, int d, int dv, int dr, int dvp,
                 float* rec, float* vbuf, cudaStream_t st) {
   const long long vb = ((long long)H * dvp + PREP_THREADS - 1) / PREP_THREADS * V_SPLIT;
   if (H + vb > 65535) return DRYFT_ERR_UNSUPPORTED;
+  const size_t smem = sizeof(float) * (PREP_THREADS / 32) * 3 * GRP * (size_t)dr;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(delta_prep_kernel<T, CHAN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
   dim3 grid(n_tiles, (unsigned)(H + vb));
-  delta_prep_kernel<T, DR, CHAN><<<grid, PREP_THREADS, 0, st>>>(
+  delta_prep_kernel<T, CHAN><<<grid, PREP_THREADS, smem, st>>>(
       (const T*)proj, ld, x_off, b_off, (const T*)dec, dec_ld, conv_w, taps, (const T*)ring, a_log, dt_bias, tile_tok0, tile_rows, cu_q,
-      n_seqs, tok_slot, tok_pos, H, G, d, dv, dvp, rec, vbuf);
+      n_seqs, tok_slot, tok_pos, H, G, d, dv, dr, dvp, rec, vbuf);
   return launch_status();
 }
 
@@ -677,7 +680,7 @@ int walk_launch(const float* rec, const float* vbuf, const int* cu_q, const int*
                 float* state, float* o, cudaStream_t st) {
   constexpr int COLS = WALK_WARPS * (32 / L) * CPG;
   static_assert(V_PAD % COLS == 0, "a block's columns lie within a padded row of v");
-  const size_t smem = sizeof(float) * WALK_STAGES * (size_t)(13 * L * RPL + SCAL + QUAD * COLS);
+  const size_t smem = sizeof(float) * WALK_STAGES * (size_t)(VECS * L * RPL + SCAL + GRP * COLS);
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(delta_walk_kernel<L, RPL, CPG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
@@ -715,24 +718,17 @@ DRYFT_API int dryft_delta_prep(int is_bf16, int per_channel, const void* proj, i
                                const int* tok_slot, const int* tok_pos, int H, int G, int d, int dv, float* rec, float* vbuf,
                                cudaStream_t st) {
   if (n_tiles <= 0) return 0;
-  if (!sizes_ok(H, G, d, dv, taps) || tile_size % QUAD || (taps > 1 && ring == nullptr)) return DRYFT_ERR_UNSUPPORTED;
-  const int dvp = (dv + V_PAD - 1) / V_PAD * V_PAD;
-#define DRYFT_PREP(T, DR, CH)                                                                                                       \
-  return prep_launch<T, DR, CH>(proj, ld, x_off, b_off, dec, dec_ld, conv_w, taps, ring, a_log, dt_bias, tile_tok0, tile_rows, n_tiles, \
-                                cu_q, n_seqs, tok_slot, tok_pos, H, G, d, dv, dvp, rec, vbuf, st)
-#define DRYFT_PREP_R(T, CH)                  \
-  switch (rows_per_lane(d)) {                \
-    case 1: DRYFT_PREP(T, 1, CH);            \
-    case 2: DRYFT_PREP(T, 2, CH);            \
-    case 4: DRYFT_PREP(T, 4, CH);            \
-    default: DRYFT_PREP(T, 8, CH);           \
-  }
+  if (!sizes_ok(H, G, d, dv, taps) || tile_size % GRP || (taps > 1 && ring == nullptr)) return DRYFT_ERR_UNSUPPORTED;
+  const int dr = 32 * rows_per_lane(d), dvp = (dv + V_PAD - 1) / V_PAD * V_PAD;
+#define DRYFT_PREP(T, CH)                                                                                                        \
+  return prep_launch<T, CH>(proj, ld, x_off, b_off, dec, dec_ld, conv_w, taps, ring, a_log, dt_bias, tile_tok0, tile_rows, n_tiles, \
+                            cu_q, n_seqs, tok_slot, tok_pos, H, G, d, dv, dr, dvp, rec, vbuf, st)
   if (is_bf16) {
-    if (per_channel) { DRYFT_PREP_R(__nv_bfloat16, true) } else { DRYFT_PREP_R(__nv_bfloat16, false) }
-  } else {
-    if (per_channel) { DRYFT_PREP_R(float, true) } else { DRYFT_PREP_R(float, false) }
+    if (per_channel) DRYFT_PREP(__nv_bfloat16, true);
+    DRYFT_PREP(__nv_bfloat16, false);
   }
-#undef DRYFT_PREP_R
+  if (per_channel) DRYFT_PREP(float, true);
+  DRYFT_PREP(float, false);
 #undef DRYFT_PREP
 }
 
@@ -744,10 +740,10 @@ DRYFT_API int dryft_delta_walk(const float* rec, const float* vbuf, const int* c
 #define DRYFT_WALK(L, R, C) return walk_launch<L, R, C>(rec, vbuf, cu_q, seq_slot, n_seqs, H, dv, dp, dvp, state, o, st)
   switch (rows_per_lane(d)) {      // L * RPL = 32 * rows_per_lane: the length of a record's vectors
     case 1: DRYFT_WALK(8, 4, 1);
-    case 2: DRYFT_WALK(8, 8, 1);
+    case 2: DRYFT_WALK(16, 4, 2);
     case 4:      // few columns for the device (at most eight an SM): two a warp instead of four
       if ((long long)n_seqs * H * dv <= FEW_COLUMNS) DRYFT_WALK(32, 4, 2);
-      DRYFT_WALK(32, 4, 4);
+      DRYFT_WALK(16, 8, 2);
     default: DRYFT_WALK(32, 8, 4);
   }
 #undef DRYFT_WALK

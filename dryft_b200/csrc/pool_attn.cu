@@ -11,9 +11,12 @@
 //
 //   pool_attn_prep    per token: q, k (+ bias) rotated over their first `rot` dims (dims i and i + rot/2 turn together by
 //                     the angle pos * inv_freq[i], evaluated in 32-bit), THEN divided by their root mean square over D
-//                     (no weight; skipped when eps < 0); v (+ bias); k and v written into the cache at the token's position.  One warp a vector.
+//                     (no weight; skipped when eps < 0); v (+ bias); k and v written into the cache at the token's position.  A warp a vector, or several of
+//                     one token in a step of many tokens.
 //                     With convolution weights (shortconv.cuh) q, k and v first pass a short causal convolution per channel
 //                     of [q | k | v], and a decode step stores its own projected values in the convolution's ring.
+//   pool_attn_prep_run  the same behind a convolution for steps of many tokens: a block a run of eight tokens, a warp a vector of
+//                     all of them.
 //   pool_attn_prep_tok  the same per token for projections that are normed as a whole: q (all H * D values at once) and k (all
 //                     G * D) are divided by their root mean square and multiplied by a weight per entry BEFORE the rotation,
 //                     and the rotation pairs either dims i and i + rot/2 or (interleaved) dims 2i and 2i + 1.  One block a
@@ -59,13 +62,13 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
     const float* __restrict__ inv_freq, const float* __restrict__ inv_freq_lo, int rot, const int* __restrict__ tok_slot,
     const int* __restrict__ tok_pos, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, const int* __restrict__ page_table, int max_pages,
     int page_size, int n_tokens, int H, int G, float eps, int write_kv, const float* __restrict__ conv_w, int taps, T* __restrict__ ring,
-    int store_ring) {
+    int store_ring, int per_warp) {
   __shared__ float sm[PREP_WARPS][D > DV ? D : DV];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int per_tok = H + (write_kv ? 2 * G : 0);
+  const int per_tok = H + (write_kv ? 2 * G : 0), parts = (per_tok + per_warp - 1) / per_warp;
   const long long item = (long long)blockIdx.x * PREP_WARPS + warp;
-  if (item >= (long long)n_tokens * per_tok) return;
-  const int t = (int)(item / per_tok), vec = (int)(item % per_tok);
+  if (item >= (long long)n_tokens * parts) return;
+  const int t = (int)(item / parts), vec0 = (int)(item % parts) * per_warp, vec1 = min(per_tok, vec0 + per_warp);
   const int slot = tok_slot[t];
   if (slot < 0) return;
   const int pos = tok_pos[t];
@@ -82,57 +85,174 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
     if (store_ring) ring_row[c] = row[c];
     return conv(c);
   };
-  size_t cache_row = 0;
-  if (vec >= H) {
-    const int g = (vec - H) % G;
-    const int page = page_table[(size_t)slot * max_pages + pos / page_size];
-    cache_row = ((size_t)page * G + g) * page_size + pos % page_size;
-  }
-  if (vec >= H + G) {     // a value vector: bias, cache
-    const int g = vec - H - G, src = H * D + G * D + g * DV;
-    for (int c = lane; c < DV; c += 32)
-      v_pages[cache_row * DV + c] = from_f32<T>(input(src + c) + (vb != nullptr ? vb[g * DV + c] : 0.f));
-    return;
-  }
-  const bool is_q = vec < H;
-  const int hd = is_q ? vec : vec - H;
-  const int src = is_q ? hd * D : H * D + hd * D;
-  const float* bias = is_q ? qb : kb;
-  float* s = sm[warp];
-  for (int c = lane; c < D; c += 32) s[c] = input(src + c) + (bias != nullptr ? bias[hd * D + c] : 0.f);
-  __syncwarp();
+  // the token's angles, once for all its vectors: entry c turns with its partner half a rotation away
   const int half = rot / 2;
-  const float fpos = (float)pos;
-  float o[DR];
-  float ss = 0.f;
+  float sn[DR], cs[DR];
 #pragma unroll
   for (int r = 0; r < DR; ++r) {
     const int c = lane + 32 * r;
-    float v = 0.f;
-    if (c < D) {
-      if (c < half) {
-        float sn, cs;
-        sincos_split(fpos, inv_freq[c], inv_freq_lo != nullptr ? inv_freq_lo[c] : 0.f, &sn, &cs);
-        v = s[c] * cs - s[c + half] * sn;
-      } else if (c < rot) {
-        float sn, cs;
-        sincos_split(fpos, inv_freq[c - half], inv_freq_lo != nullptr ? inv_freq_lo[c - half] : 0.f, &sn, &cs);
-        v = s[c] * cs + s[c - half] * sn;
-      } else {
-        v = s[c];
+    sn[r] = 0.f;
+    cs[r] = 1.f;
+    if (vec0 < H + G && c < rot) {
+      const int i = c < half ? c : c - half;
+      sincos_split((float)pos, inv_freq[i], inv_freq_lo != nullptr ? inv_freq_lo[i] : 0.f, &sn[r], &cs[r]);
+      if (c < half) sn[r] = -sn[r];
+    }
+  }
+  float* s = sm[warp];
+  for (int vec = vec0; vec < vec1; ++vec) {
+    size_t cache_row = 0;
+    if (vec >= H) {
+      const int g = (vec - H) % G;
+      const int page = page_table[(size_t)slot * max_pages + pos / page_size];
+      cache_row = ((size_t)page * G + g) * page_size + pos % page_size;
+    }
+    if (vec >= H + G) {     // a value vector: bias, cache
+      const int g = vec - H - G, src = H * D + G * D + g * DV;
+      for (int c = lane; c < DV; c += 32)
+        v_pages[cache_row * DV + c] = from_f32<T>(input(src + c) + (vb != nullptr ? vb[g * DV + c] : 0.f));
+      continue;
+    }
+    const bool is_q = vec < H;
+    const int hd = is_q ? vec : vec - H;
+    const int src = is_q ? hd * D : H * D + hd * D;
+    const float* bias = is_q ? qb : kb;
+    __syncwarp();           // the vector before this one has been read
+    for (int c = lane; c < D; c += 32) s[c] = input(src + c) + (bias != nullptr ? bias[hd * D + c] : 0.f);
+    __syncwarp();
+    float o[DR];
+    float ss = 0.f;
+#pragma unroll
+    for (int r = 0; r < DR; ++r) {
+      const int c = lane + 32 * r;
+      float v = 0.f;
+      if (c < D) v = c < rot ? s[c] * cs[r] + s[c < half ? c + half : c - half] * sn[r] : s[c];
+      o[r] = v;
+      ss = fmaf(v, v, ss);
+    }
+    float rinv = 1.f;                                                      // eps < 0: no unit norm
+    if (eps >= 0.f) rinv = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
+    T* dst = is_q ? q_out + ((size_t)t * H + hd) * D : k_pages + cache_row * D;
+#pragma unroll
+    for (int r = 0; r < DR; ++r) {
+      const int c = lane + 32 * r;
+      if (c < D) dst[c] = from_f32<T>(o[r] * rinv);
+    }
+  }
+}
+
+// The same behind a convolution, for steps of many tokens: a block takes RUN consecutive tokens of one sequence (part
+// blockIdx.y of tile blockIdx.x), a warp a vector of all of them, so that the weights are read once and a row's value serves
+// every token that it reaches.  The tokens' angles are formed once per block.
+constexpr int RUN = 8, RUN_WARPS = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(RUN_WARPS * 32) pool_attn_prep_run_kernel(
+    const T* __restrict__ proj, int ld, const float* __restrict__ inv_freq, const float* __restrict__ inv_freq_lo, int rot,
+    const int* __restrict__ tile_tok0, const int* __restrict__ tile_rows, const int* __restrict__ cu_q, int n_seqs,
+    const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, T* __restrict__ q_out, T* __restrict__ k_pages,
+    T* __restrict__ v_pages, const int* __restrict__ page_table, int max_pages, int page_size, int H, int G, float eps,
+    const float* __restrict__ conv_w, int taps, const T* __restrict__ ring) {
+  extern __shared__ float mem[];                  // [RUN_WARPS][RUN][D] convolved vectors, then [RUN][rot / 2][2] sines and cosines
+  const int tok0 = tile_tok0[blockIdx.x] + (int)blockIdx.y * RUN, rows = min(RUN, tile_rows[blockIdx.x] - (int)blockIdx.y * RUN);
+  if (rows <= 0) return;
+  const int slot = tok_slot[tok0];
+  if (slot < 0) return;
+  int lo = 0, hi = n_seqs - 1;                    // the sequence: the largest b with cu_q[b] <= tok0
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_q[mid] <= tok0) lo = mid; else hi = mid - 1;
+  }
+  const int t0 = cu_q[lo], n = cu_q[lo + 1] - t0, p0 = tok_pos[t0], i0 = tok0 - t0, pos0 = p0 + i0;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = rot / 2;
+  const int CH = H * D + G * (D + DV);
+  float* s = mem + (size_t)warp * RUN * D;
+  float* ang = mem + (size_t)RUN_WARPS * RUN * D;
+  for (int i = threadIdx.x; i < RUN * half; i += RUN_WARPS * 32) {
+    const int k = i / half, f = i % half;
+    float sn, cs;
+    sincos_split((float)(pos0 + k), inv_freq[f], inv_freq_lo != nullptr ? inv_freq_lo[f] : 0.f, &sn, &cs);
+    ang[2 * i] = sn;
+    ang[2 * i + 1] = cs;
+  }
+  __syncthreads();
+  const int* pages = page_table + (size_t)slot * max_pages;
+  for (int vec = warp; vec < H + 2 * G; vec += RUN_WARPS) {
+    const int g = vec < H ? 0 : (vec - H) % G;
+    if (vec >= H + G) {      // a value vector
+      for (int c = lane; c < DV; c += 32) {
+        float acc[RUN];
+        conv_run<T, RUN>(acc, conv_w, proj, ld, ring, taps, CH, slot, t0, p0, i0, n, H * D + G * D + g * DV + c);
+#pragma unroll
+        for (int k = 0; k < RUN; ++k) {
+          const int p = pos0 + k;
+          if (k < rows) v_pages[(((size_t)pages[p / page_size] * G + g) * page_size + p % page_size) * DV + c] = from_f32<T>(acc[k]);
+        }
+      }
+      continue;
+    }
+    const bool is_q = vec < H;
+    const int src = is_q ? vec * D : H * D + g * D;
+    __syncwarp();            // the vector before this one has been read
+#pragma unroll 2
+    for (int r = 0; r < DR; ++r) {
+      const int c = lane + 32 * r;
+      if (c < D) {
+        float acc[RUN];
+        conv_run<T, RUN>(acc, conv_w, proj, ld, ring, taps, CH, slot, t0, p0, i0, n, src + c);
+#pragma unroll
+        for (int k = 0; k < RUN; ++k) s[k * D + c] = acc[k];
       }
     }
-    o[r] = v;
-    ss = fmaf(v, v, ss);
-  }
-  ss = warp_sum(ss);
-  const float rinv = eps >= 0.f ? 1.f / sqrtf(ss / (float)D + eps) : 1.f;    // eps < 0: no unit norm
-  T* dst = is_q ? q_out + ((size_t)t * H + hd) * D : k_pages + cache_row * D;
+    __syncwarp();
+#pragma unroll 1
+    for (int k = 0; k < rows; ++k) {
+      float o[DR];
+      float ss = 0.f;
 #pragma unroll
-  for (int r = 0; r < DR; ++r) {
-    const int c = lane + 32 * r;
-    if (c < D) dst[c] = from_f32<T>(o[r] * rinv);
+      for (int r = 0; r < DR; ++r) {
+        const int c = lane + 32 * r;
+        float v = 0.f;
+        if (c < D) {
+          v = s[k * D + c];
+          if (c < rot) {
+            const float* a = ang + 2 * (k * half + (c < half ? c : c - half));
+            v = c < half ? v * a[1] - s[k * D + c + half] * a[0] : v * a[1] + s[k * D + c - half] * a[0];
+          }
+        }
+        o[r] = v;
+        ss = fmaf(v, v, ss);
+      }
+      float rinv = 1.f;
+      if (eps >= 0.f) rinv = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);     // eps < 0: no unit norm
+      const int p = pos0 + k;
+      T* dst = is_q ? q_out + ((size_t)(tok0 + k) * H + vec) * D
+                    : k_pages + (((size_t)pages[p / page_size] * G + g) * page_size + p % page_size) * D;
+#pragma unroll
+      for (int r = 0; r < DR; ++r) {
+        const int c = lane + 32 * r;
+        if (c < D) dst[c] = from_f32<T>(o[r] * rinv);
+      }
+    }
   }
+}
+
+template <typename T>
+int prep_run_launch(const void* proj, int ld, const float* inv_freq, const float* inv_freq_lo, int rot, const int* tile_tok0,
+                    const int* tile_rows, int n_tiles, int tile_size, const int* cu_q, int n_seqs, const int* tok_slot, const int* tok_pos,
+                    void* q_out, void* k_pages, void* v_pages, const int* page_table, int max_pages, int page_size, int H, int G, float eps,
+                    const float* conv_w, int taps, const void* ring, cudaStream_t st) {
+  const size_t smem = sizeof(float) * ((size_t)RUN_WARPS * RUN * D + (size_t)RUN * rot);
+  if (smem > 200 * 1024) return DRYFT_ERR_UNSUPPORTED;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(pool_attn_prep_run_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  dim3 grid(n_tiles, (tile_size + RUN - 1) / RUN);
+  pool_attn_prep_run_kernel<T><<<grid, RUN_WARPS * 32, smem, st>>>((const T*)proj, ld, inv_freq, inv_freq_lo, rot, tile_tok0, tile_rows, cu_q, n_seqs,
+                                                                  tok_slot, tok_pos, (T*)q_out, (T*)k_pages, (T*)v_pages, page_table, max_pages,
+                                                                  page_size, H, G, eps, conv_w, taps, (const T*)ring);
+  return launch_status();
 }
 
 // One block per token.  q_w [H * D] / k_w [G * D]: the weights of a norm over the whole projection (nullptr: no such norm).
@@ -429,12 +549,14 @@ int prep_launch(const void* proj, int ld, const float* qb, const float* kb, cons
                 const float* inv_freq_lo, int rot, const int* tok_slot, const int* tok_pos, void* q_out, void* k_pages, void* v_pages, const int* page_table,
                 int max_pages, int page_size, int n, int H, int G, float eps, int write_kv, const float* conv_w, int taps, void* ring,
                 int store_ring, cudaStream_t st) {
-  const long long items = (long long)n * (H + (write_kv ? 2 * G : 0));
+  // many tokens: a warp takes several vectors of one token, which share its angles and the rows its convolution reads
+  const int per_tok = H + (write_kv ? 2 * G : 0), per_warp = n >= 512 ? 8 : n >= 128 ? 4 : 1;
+  const long long items = (long long)n * ((per_tok + per_warp - 1) / per_warp);
   const long long blocks = (items + PREP_WARPS - 1) / PREP_WARPS;
   if (blocks > 0x7fffffffLL) return DRYFT_ERR_UNSUPPORTED;
   pool_attn_prep_kernel<T><<<(unsigned)blocks, PREP_WARPS * 32, 0, st>>>(
       (const T*)proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, (T*)q_out, (T*)k_pages, (T*)v_pages, page_table, max_pages,
-      page_size, n, H, G, eps, write_kv, conv_w, taps, (T*)ring, store_ring);
+      page_size, n, H, G, eps, write_kv, conv_w, taps, (T*)ring, store_ring, per_warp);
   return launch_status();
 }
 
@@ -472,6 +594,22 @@ DRYFT_API int dryft_pool_attn_prep(int is_bf16, const void* proj, int ld, const 
                                               max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, st)
                  : prep_launch<float>(proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, q_out, k_pages, v_pages, page_table,
                                       max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, st);
+}
+
+DRYFT_API int dryft_pool_attn_prep_run(int is_bf16, const void* proj, int ld, const float* inv_freq, const float* inv_freq_lo, int rot,
+                                       const int* tile_tok0, const int* tile_rows, int n_tiles, int tile_size, const int* cu_q, int n_seqs,
+                                       const int* tok_slot, const int* tok_pos, void* q_out, void* k_pages, void* v_pages,
+                                       const int* page_table, int max_pages, int page_size, int H, int G, float eps, const float* conv_w,
+                                       int taps, const void* ring, cudaStream_t st) {
+  if (n_tiles <= 0) return 0;
+  if (H != G * REP || rot < 0 || rot % 2 || rot > D || (rot > 0 && inv_freq == nullptr) || page_size < 1 || tile_size < 1 || taps < 1 ||
+      taps > DRYFT_CONV_MAX_TAPS || (taps > 1 && ring == nullptr))
+    return DRYFT_ERR_UNSUPPORTED;
+  return is_bf16 ? prep_run_launch<__nv_bfloat16>(proj, ld, inv_freq, inv_freq_lo, rot, tile_tok0, tile_rows, n_tiles, tile_size, cu_q, n_seqs,
+                                                  tok_slot, tok_pos, q_out, k_pages, v_pages, page_table, max_pages, page_size, H, G, eps, conv_w,
+                                                  taps, ring, st)
+                 : prep_run_launch<float>(proj, ld, inv_freq, inv_freq_lo, rot, tile_tok0, tile_rows, n_tiles, tile_size, cu_q, n_seqs, tok_slot,
+                                          tok_pos, q_out, k_pages, v_pages, page_table, max_pages, page_size, H, G, eps, conv_w, taps, ring, st);
 }
 
 DRYFT_API int dryft_pool_attn_prep_tok(int is_bf16, const void* proj, int ld, const float* q_w, const float* k_w, float norm_eps,

@@ -263,6 +263,17 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
   }
 
   // ---- divide by the sum (the sink's share is in it), store ----
+  __nv_bfloat162 z0[DT], z1[DT];      // the rows' gate logits, all requested before the first is used
+  if (gate != nullptr) {
+    const bool pairs = (gate_ld & 1) == 0 && (reinterpret_cast<uintptr_t>(gate) & 3) == 0;   // two logits a load
+    const bf16* gp0 = gate + (size_t)(tok0 + min(warp * 16 + g, rows - 1)) * gate_ld + (size_t)h * DV + 2 * t;
+    const bf16* gp1 = gate + (size_t)(tok0 + min(warp * 16 + g + 8, rows - 1)) * gate_ld + (size_t)h * DV + 2 * t;
+#pragma unroll
+    for (int j = 0; j < DT; ++j) {
+      z0[j] = pairs ? *reinterpret_cast<const __nv_bfloat162*>(gp0 + j * 8) : __halves2bfloat162(gp0[j * 8], gp0[j * 8 + 1]);
+      z1[j] = pairs ? *reinterpret_cast<const __nv_bfloat162*>(gp1 + j * 8) : __halves2bfloat162(gp1[j * 8], gp1[j * 8 + 1]);
+    }
+  }
   float l0 = l_run[0], l1 = l_run[1];
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
@@ -270,22 +281,14 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   const float f0 = l0 > 0.f ? 1.f / l0 : 0.f, f1 = l1 > 0.f ? 1.f / l1 : 0.f;
   const int r0 = warp * 16 + g, r1 = r0 + 8;
-  const bool gate_pairs = (gate_ld & 1) == 0 && (reinterpret_cast<uintptr_t>(gate) & 3) == 0;   // two logits a load
 #pragma unroll
   for (int j = 0; j < DT; ++j) {
     const int d = j * 8 + 2 * t;
     float g00 = f0, g01 = f0, g10 = f1, g11 = f1;
     if (gate != nullptr) {       // each value times the sigmoid of its own logit
-      auto factors = [&](int r, float& lo, float& hi) {
-        const bf16* gp = gate + (size_t)(tok0 + r) * gate_ld + (size_t)h * DV + d;
-        __nv_bfloat162 z;
-        if (gate_pairs) z = *reinterpret_cast<const __nv_bfloat162*>(gp);
-        else z = __halves2bfloat162(gp[0], gp[1]);
-        lo *= __fdividef(1.f, 1.f + exp2f(-1.4426950408889634f * __low2float(z)));
-        hi *= __fdividef(1.f, 1.f + exp2f(-1.4426950408889634f * __high2float(z)));
-      };
-      if (r0 < rows) factors(r0, g00, g01);
-      if (r1 < rows) factors(r1, g10, g11);
+      auto sig = [](float z) { return __fdividef(1.f, 1.f + exp2f(-1.4426950408889634f * z)); };
+      g00 *= sig(__low2float(z0[j])); g01 *= sig(__high2float(z0[j]));
+      g10 *= sig(__low2float(z1[j])); g11 *= sig(__high2float(z1[j]));
     }
     if (r0 < rows)
       *reinterpret_cast<unsigned*>(out + ((size_t)(tok0 + r0) * nH + h) * DV + d) = pack_bf16(o_acc[j][0] * g00, o_acc[j][1] * g01);

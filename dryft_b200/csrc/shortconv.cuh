@@ -10,50 +10,48 @@
 
 #define DRYFT_CONV_MAX_TAPS 16
 
-// The input of channel c at step index i of its sequence (i < 0: before this step), for a sequence whose first token of the
-// step is packed row t0 at position p0.  x points at channel 0 of packed row 0, row stride ld.
+// The input of channel c at step index i of its sequence (i < 0: before this step; n: the step's tokens of the sequence), for a
+// sequence whose first token of the step is packed row t0 at position p0.  x points at channel 0 of packed row 0, row stride ld.
+// The address is chosen without a branch, so that a run's loads are all on their way at once; what does not exist (before the
+// sequence's start, behind its end) reads the step's first row and counts as zero.
 template <typename T>
 __device__ __forceinline__ float conv_input(const T* __restrict__ x, int ld, const T* __restrict__ ring, int taps, int CH,
-                                            int slot, int t0, int p0, int i, int c) {
-  if (i >= 0) return to_f32<T>(x[(size_t)(t0 + i) * ld + c]);
+                                            int slot, int t0, int p0, int i, int n, int c) {
   const int p = p0 + i;
-  return p >= 0 ? to_f32<T>(ring[((size_t)slot * taps + p % taps) * CH + c]) : 0.f;
+  const bool here = i >= 0 && i < n, before = i < 0 && p >= 0;
+  const T* src = x + (size_t)(here ? t0 + i : t0) * ld + c;
+  if (before) src = ring + ((size_t)slot * taps + (taps == 4 ? p & 3 : p % taps)) * CH + c;
+  const float u = to_f32<T>(*src);
+  return here || before ? u : 0.f;
 }
 
-// acc[k] = the convolution's result at step indices i0 + k, k = 0..3, of channel c; tokens from index n on do not exist
-template <typename T>
-__device__ __forceinline__ void conv4(float (&acc)[4], const float* __restrict__ w, const T* __restrict__ x, int ld,
-                                      const T* __restrict__ ring, int taps, int CH, int slot, int t0, int p0, int i0, int n, int c) {
+// acc[k] = the convolution's result at step indices i0 + k, k < N, of channel c
+template <typename T, int N>
+__device__ __forceinline__ void conv_run(float (&acc)[N], const float* __restrict__ w, const T* __restrict__ x, int ld,
+                                         const T* __restrict__ ring, int taps, int CH, int slot, int t0, int p0, int i0, int n, int c) {
   const float* wc = w + (size_t)c * taps;
-  if (taps == 4) {      // the usual case, unrolled: seven inputs, four weights
+  if (taps == 4) {      // the usual case, unrolled
     const float4 ww = *reinterpret_cast<const float4*>(wc);
-    float u[7];
-    if (i0 >= 3 && i0 + 4 <= n) {      // all of them belong to this step: seven loads without a question
+    float u[N + 3];
+    if (i0 >= 3 && i0 + N <= n) {      // all inputs belong to this step
       const T* src = x + (size_t)(t0 + i0 - 3) * ld + c;
 #pragma unroll
-      for (int s = 0; s < 7; ++s) u[s] = to_f32<T>(src[(size_t)s * ld]);
+      for (int s = 0; s < N + 3; ++s) u[s] = to_f32<T>(src[(size_t)s * ld]);
     } else {
 #pragma unroll
-      for (int s = 0; s < 7; ++s) {
-        const int i = i0 - 3 + s;
-        u[s] = i < n ? conv_input<T>(x, ld, ring, taps, CH, slot, t0, p0, i, c) : 0.f;
-      }
+      for (int s = 0; s < N + 3; ++s) u[s] = conv_input<T>(x, ld, ring, 4, CH, slot, t0, p0, i0 - 3 + s, n, c);
     }
 #pragma unroll
-    for (int k = 0; k < 4; ++k) acc[k] = fmaf(ww.w, u[k + 3], fmaf(ww.z, u[k + 2], fmaf(ww.y, u[k + 1], ww.x * u[k])));
+    for (int k = 0; k < N; ++k) acc[k] = fmaf(ww.w, u[k + 3], fmaf(ww.z, u[k + 2], fmaf(ww.y, u[k + 1], ww.x * u[k])));
     return;
   }
 #pragma unroll
-  for (int k = 0; k < 4; ++k) acc[k] = 0.f;
-  for (int s = 0; s < taps + 3; ++s) {
-    const int i = i0 - (taps - 1) + s;
-    if (i >= n) break;
-    const float u = conv_input<T>(x, ld, ring, taps, CH, slot, t0, p0, i, c);
+  for (int k = 0; k < N; ++k) acc[k] = 0.f;
+#pragma unroll 1
+  for (int j = 0; j < taps; ++j) {
+    const float wj = wc[j];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const int j = s - k;
-      if (j >= 0 && j < taps) acc[k] = fmaf(wc[j], u, acc[k]);
-    }
+    for (int k = 0; k < N; ++k) acc[k] = fmaf(wj, conv_input<T>(x, ld, ring, taps, CH, slot, t0, p0, i0 + k - (taps - 1) + j, n, c), acc[k]);
   }
 }
 

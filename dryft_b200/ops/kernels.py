@@ -1770,7 +1770,9 @@ def pool_attention_lib(qk_dim: int, v_dim: int, group: int) -> ctypes.CDLL:
                                                  _i, _i, _i, _p, _i, _p]
             lib.dryft_pool_attn_prep_tok.argtypes = [_i, _p, _i, _p, _p, _f, _p, _p, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i,
                                                      _f, _i, _p]
-            for fn in ("dryft_pool_attn_prep", "dryft_pool_attn_prep_tok", "dryft_pool_attn_blocks", "dryft_pool_attn_rows"):
+            lib.dryft_pool_attn_prep_run.argtypes = [_i, _p, _i, _p, _p, _i, _p, _p, _i, _i, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _f, _p,
+                                                     _i, _p, _p]
+            for fn in ("dryft_pool_attn_prep", "dryft_pool_attn_prep_run", "dryft_pool_attn_prep_tok", "dryft_pool_attn_blocks", "dryft_pool_attn_rows"):
                 getattr(lib, fn).restype = _i
             if (lib.dryft_pool_attn_qk_dim(), lib.dryft_pool_attn_v_dim(), lib.dryft_pool_attn_group()) != (qk_dim, v_dim, group):
                 raise KernelError(f"{path} was compiled for other sizes")
@@ -1875,6 +1877,36 @@ def pool_attn_prep(proj, q_bias, k_bias, v_bias, inv_freq, inv_freq_lo, rot: int
                                  _ptr(page_table), page_table.shape[1], k_pages.shape[2], n, n_heads, n_kv, float(eps),
                                  int(write_kv), _ptr(conv_w), taps, _ptr(ring if taps > 1 else None), int(store_ring and taps > 1),
                                  _stream()), f"pool_attn_prep ({n_heads}/{n_kv} heads of {d})")
+
+
+def pool_attn_prep_run(proj, inv_freq, inv_freq_lo, rot: int, ctx, q_out, k_pages, v_pages, page_table, n_heads: int, n_kv: int, eps: float,
+                       conv_w, ring) -> None:
+    """``pool_attn_prep`` behind a convolution for a step of many tokens (``ctx``: its tiles say which tokens follow one another);
+    the ring is read, not advanced (``conv_ring_store``)."""
+    n, ld = proj.shape
+    d, dv = q_out.shape[2], v_pages.shape[-1]
+    ch = n_heads * d + n_kv * (d + dv)
+    _need(proj, "proj")
+    _need(q_out, "q_out", proj.dtype, (n, n_heads, d))
+    _need(k_pages, "k_pages", proj.dtype, (None, n_kv, None, d))
+    _need(v_pages, "v_pages", proj.dtype, (None, n_kv, k_pages.shape[2], dv))
+    _need(page_table, "page_table", torch.int32)
+    _need(conv_w, "conv_w", torch.float32, (ch, None))
+    taps = conv_w.shape[1]
+    if ld < ch:
+        raise KernelError(f"pool_attn_prep_run: a row of {ld} values is too short for {n_heads} + {n_kv} heads")
+    if taps > 1:
+        _need(ring, "ring", proj.dtype, (None, taps, ch))
+    if rot:
+        _need(inv_freq, "inv_freq", torch.float32, (rot // 2,))
+        if inv_freq_lo is not None:
+            _need(inv_freq_lo, "inv_freq_lo", torch.float32, (rot // 2,))
+    lib = pool_attention_lib(d, dv, n_heads // n_kv)
+    _ok(lib.dryft_pool_attn_prep_run(_act(proj, "proj"), _ptr(proj), ld, _ptr(inv_freq), _ptr(inv_freq_lo), int(rot), _ptr(ctx.tile_tok0),
+                                     _ptr(ctx.tile_rows), int(ctx.n_tiles), int(ctx.tile_size), _ptr(ctx.cu_q), int(ctx.n_seqs),
+                                     _ptr(ctx.tok_slot), _ptr(ctx.tok_pos), _ptr(q_out), _ptr(k_pages), _ptr(v_pages), _ptr(page_table),
+                                     page_table.shape[1], k_pages.shape[2], n_heads, n_kv, float(eps), _ptr(conv_w), taps,
+                                     _ptr(ring if taps > 1 else None), _stream()), f"pool_attn_prep_run ({n_heads}/{n_kv} heads of {d})")
 
 
 def pool_attn_prep_tok(proj, q_norm_w, k_norm_w, norm_eps: float, inv_freq, inv_freq_lo, rot: int, interleaved: bool, tok_slot, tok_pos,
@@ -2173,7 +2205,7 @@ def _delta_common(proj, x_off, b_off, dec, conv_w, ring, a_log, dt_bias, heads, 
 
 def delta_tokens(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, dt_bias, norm_w, eps: float, sigmoid_gate: bool, ctx, state,
                  out, heads: int, kv_heads: int, dim: int, vdim: int, per_channel: bool) -> None:
-    """The gated delta rule over a step of many tokens (``csrc/delta.cu``): records of four tokens each, the walk over them from
+    """The gated delta rule over a step of many tokens (``csrc/delta.cu``): records of eight tokens each, the walk over them from
     each slot's ``state [slots, H, DV, dp]``, then norm and gate into ``out [n, H*DV]``.  ``ctx``: the step's context (its
     tiles say which tokens belong together).  Three launches; the last one also advances the convolution's
     ``ring``."""
@@ -2183,9 +2215,9 @@ def delta_tokens(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, d
     _need(norm_w, "norm_w", torch.float32, (vdim,))
     _need(out, "out", proj.dtype, (n, heads * vdim))
     gate_ptr, gate_ld = _rows_of(gate, "gate", proj.dtype, n, heads * vdim)
-    if ctx.tile_size % 4:
-        raise KernelError(f"delta rule: prompt tiles of {ctx.tile_size} tokens (a multiple of 4 is needed)")
-    rec = torch.empty(((n + 3 * ctx.n_seqs) // 4 + 1, heads, 13 * delta_record_dim(dim) + 28), dtype=torch.float32, device=proj.device)
+    if ctx.tile_size % 8:
+        raise KernelError(f"delta rule: prompt tiles of {ctx.tile_size} tokens (a multiple of 8 is needed)")
+    rec = torch.empty(((n + 7 * ctx.n_seqs) // 8 + 1, heads, 25 * delta_record_dim(dim) + 100), dtype=torch.float32, device=proj.device)
     vbuf = torch.empty((n, heads, dvp), dtype=torch.float32, device=proj.device)
     o = torch.empty((n, heads * vdim), dtype=torch.float32, device=proj.device)
     lib, bf = delta_lib(), _act(proj, "proj")

@@ -203,10 +203,14 @@ class PooledWindowAttention:
                                  ctx.tok_pos, q, cache.k, cache.v, cache.page_table, self.n_heads, self.n_kv,
                                  self.eps if self.unit_norm else -1.0, owns_cache)
         else:
-            K.pool_attn_prep(proj, self.q_bias, self.k_bias, self.v_bias, pos.inv_freq if self.rot else None,
-                             getattr(pos, "inv_freq_lo", None) if self.rot else None, self.rot, ctx.tok_slot, ctx.tok_pos, q, cache.k,
-                             cache.v, cache.page_table, self.n_heads, self.n_kv, self.eps if self.unit_norm else -1.0, owns_cache,
-                             conv_w=self.conv_w, ring=state["conv"] if self.taps > 1 else None, store_ring=ctx.decode)
+            freq = (pos.inv_freq, getattr(pos, "inv_freq_lo", None), self.rot) if self.rot else (None, None, 0)
+            ring, unit_eps = state["conv"] if self.taps > 1 else None, self.eps if self.unit_norm else -1.0
+            if self.taps and not ctx.decode and self.q_bias is None and owns_cache:
+                K.pool_attn_prep_run(proj, *freq, ctx, q, cache.k, cache.v, cache.page_table, self.n_heads, self.n_kv, unit_eps, self.conv_w, ring)
+            else:
+                K.pool_attn_prep(proj, self.q_bias, self.k_bias, self.v_bias, *freq, ctx.tok_slot, ctx.tok_pos, q, cache.k, cache.v,
+                                 cache.page_table, self.n_heads, self.n_kv, unit_eps, owns_cache, conv_w=self.conv_w, ring=ring,
+                                 store_ring=ctx.decode)
             if self.taps > 1 and not ctx.decode:
                 K.conv_ring_store(proj, 0, ctx.cu_q, ctx.seq_slot, ctx.tok_pos, state["conv"], ctx.n_seqs)
         pooled = None

@@ -242,7 +242,8 @@ def test_one_key_that_stands_out_at_every_edge(size, keep, edge):
 
 @pytest.mark.parametrize("taps", [1, 2, 4, 7])
 @pytest.mark.parametrize("rot", [0, 6, 16])
-def test_convolved_rotated_queries_keys_and_values_across_cuts(taps, rot):
+@pytest.mark.parametrize("runs", [False, True])      # token by token, or runs of tokens where the step has many
+def test_convolved_rotated_queries_keys_and_values_across_cuts(taps, rot, runs):
     """The preparation of a head behind a short convolution: whole prompts, pieces shorter than the taps, single tokens; two
     sequences in a step, their slots' rings NaN before (what is not of the sequence is never read)."""
     from dryft_b200.ops import kernels as K
@@ -271,8 +272,11 @@ def test_convolved_rotated_queries_keys_and_values_across_cuts(taps, rot):
         ctx = step_context(lens, at, slots)
         q = torch.empty(sum(lens), H, d, device=DEV)
         decode = all(n == 1 for n in lens)
-        K.pool_attn_prep(x, None, None, None, freq.float().to(DEV) if rot else None, lo, rot, ctx.tok_slot, ctx.tok_pos, q, kp, vp, table, H, G, -1.0, True,
-                         conv_w=cw_d, ring=ring, store_ring=decode)
+        if runs and not decode:
+            K.pool_attn_prep_run(x, freq.float().to(DEV) if rot else None, lo, rot, ctx, q, kp, vp, table, H, G, -1.0, cw_d, ring)
+        else:
+            K.pool_attn_prep(x, None, None, None, freq.float().to(DEV) if rot else None, lo, rot, ctx.tok_slot, ctx.tok_pos, q, kp, vp, table, H, G, -1.0, True,
+                             conv_w=cw_d, ring=ring, store_ring=decode)
         if taps > 1 and not decode:
             K.conv_ring_store(x, 0, ctx.cu_q, ctx.seq_slot, ctx.tok_pos, ring, len(lens))
         o = 0
