@@ -206,7 +206,8 @@ class DusupelConfig:
             specs.append(LayerSpec(
                 block="parallel_norms", mixer=self._mixer_spec(l), ffn=ffn, norm_mixer=norm("norm1"), norm_ffn=norm("norm2") if ffn else None,
                 mixer_prefix=f"l{i}.mix.", ffn_prefix=f"l{i}.mlp.", norm_mixer_prefix=f"l{i}.", norm_ffn_prefix=f"l{i}.",
-                extra=(ExtraPart("sum", "connection", PartSpec("scaled_sum", {"mult": self.residual_mult}), f"l{i}."),)))
+                extra=(ExtraPart("sum", "connection", PartSpec("scaled_sum", {
+                    "mult": self.residual_mult, "unread": {} if ffn else {"norm2": self.width, "norm2.b": self.width}}), f"l{i}."),)))
         spec = ModelSpec(
             architecture=self.architecture,
             vocab_size=self.vocab,

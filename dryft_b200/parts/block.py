@@ -282,11 +282,13 @@ class ParallelBlock:
 
 @register_connection("scaled_sum")
 class ScaledSum:
-    """A constant ``mult`` that the sublayers' results take on their way into the stream: ``x + mult * y``."""
+    """A constant ``mult`` that the sublayers' results take on their way into the stream: ``x + mult * y``.  ``unread``: vectors
+    (name behind the prefix -> size) that a checkpoint may hold and nothing reads, such as the norm in front of a feed-forward
+    that the layer leaves out."""
 
     @staticmethod
     def tensors(params: Mapping, prefix: str) -> Dict[str, TensorInfo]:
-        return {}
+        return {prefix + name: TensorInfo((int(size),), "vector", optional=True) for name, size in (params.get("unread") or {}).items()}
 
     def __init__(self, params: Mapping, prefix: str, weights, rt: Runtime):
         self.mult = float(params.get("mult", 1.0))

@@ -47,6 +47,17 @@ def test_a_rank_is_free_but_nothing_else_is(tmp_path):
                 check()
 
 
+def test_a_layer_without_a_feed_forward_may_hold_its_norm(tmp_path):
+    cfg = M.config([M.delta(ff=None)])
+    w = M.draw_weights(cfg, 1)
+    for i, more in enumerate(({}, {"l0.norm2": torch.ones(48), "l0.norm2.b": torch.zeros(48)})):
+        d = M.write_model(cfg, dict(w, **more), str(tmp_path / str(i)))
+        Checkpoint(d).check(expected_tensors(load_config(d).model_spec()))
+    d = M.write_model(cfg, dict(w, **{"l0.norm3": torch.ones(48)}), str(tmp_path / "x"))
+    with pytest.raises(WeightsError, match="norm3"):
+        Checkpoint(d).check(expected_tensors(load_config(d).model_spec()))
+
+
 def test_errors_name_the_key():
     base = M.CONFIGS["looped"]
 
