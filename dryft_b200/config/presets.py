@@ -228,6 +228,38 @@ PRESETS.update({
 EQUAL_SIZE.update({"dusupel-1k": "kerirax-1k", "dusupel-2k": "kerirax-2k"})
 
 
+def _puturax(width: int, heads: int, kv_heads: int, dim: int, rec_heads: int, rec_dim: int, q_rank: int, kv_rank: int, rot_dim: int, experts: int,
+             ff: int, top: int, vocab: int, layers: int, groups: int = 4, keep: int = 2) -> dict:
+    """A Puturax ``config.json``: every third layer attention over latents, the others two mixers side by side.  The first layer's
+    feed-forward is dense (the size of the experts a token uses plus the always-on one), the others are routed."""
+    pair = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 30.0,
+                     "q_temp": {"coef": 0.1, "every": 512}}, "left_scale": 1.0,
+            "right": {"heads": rec_heads, "dim": rec_dim}, "right_scale": 1.0}
+    lat = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "q_rank": q_rank, "kv_rank": kv_rank,
+           "scale": (dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": 10000.0}}
+    out = []
+    for i in range(layers):
+        mlp = {"kind": "dense", "ff": ff * (top + 1)} if i == 0 else \
+            {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": ff},
+             "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
+        out.append({"type": "latent_attention", "mixer": lat, "mlp": mlp} if i % 3 == 1 else {"type": "parallel", "mixer": pair, "mlp": mlp})
+    return {"architecture": "Puturax", "vocab": vocab, "width": width, "embedding": {"scale": width ** 0.5}, "norm": {"eps": 1e-5}, "layers": out}
+
+
+# Puturax shapes with layers the size of a real model's, and beside each the closest design at equal size: the Kerirax shape of
+# the same width, number of layer runs, head counts and size, latent sizes, expert count and size, experts a token uses and
+# vocabulary (its scan keeps a vector per channel where time mixing keeps a matrix per head).
+PRESETS.update({
+    "puturax-tiny": _puturax(width=64, heads=4, kv_heads=2, dim=16, rec_heads=4, rec_dim=16, q_rank=24, kv_rank=32, rot_dim=8, experts=8, ff=32,
+                             top=2, vocab=256, layers=4),
+    "puturax-1k": _puturax(width=1024, heads=8, kv_heads=2, dim=128, rec_heads=16, rec_dim=64, q_rank=384, kv_rank=256, rot_dim=64, experts=32,
+                           ff=512, top=4, vocab=32768, layers=8),
+    "puturax-2k": _puturax(width=2048, heads=16, kv_heads=4, dim=128, rec_heads=32, rec_dim=64, q_rank=768, kv_rank=512, rot_dim=64, experts=64,
+                           ff=768, top=8, vocab=65536, layers=12),
+})
+EQUAL_SIZE.update({"puturax-1k": "kerirax-1k", "puturax-2k": "kerirax-2k"})
+
+
 def preset(name: str) -> dict:
     if name not in PRESETS:
         raise KeyError(f"unknown preset {name!r}; known: " + ", ".join(sorted(PRESETS)))

@@ -30,6 +30,10 @@
 // inv * sum_k T(x*w) W in place of sum_k T(T(x*inv)*w) W -- one rounding of the activations fewer than the
 // reference makes (model.py:28-32), the statistics still in 32-bit.
 //
+// Several products of the same number of rows whose activations differ may share a launch (plain activations only): the
+// weights of group j are rows j * grp_rows .. of W (the last group takes what is left), its activations the M rows that start
+// j * grp_stride elements further on.  grp_rows is a multiple of 16, so that a tile belongs to one group.
+//
 // The kernel may be launched as a programmatic dependent of the launch before it: it requests its
 // first weights, which depend on nothing, and only then waits for the earlier grid.
 // No block waits on another block of its grid; there is no spin in this file.
@@ -118,7 +122,8 @@ template <int MB, int MODE, int PRO, int GROUPS, int GW>
 __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) gemm_decode_kernel(
     const bf16* __restrict__ A, int lda, const bf16* __restrict__ W, void* C, int ldc, int M, int N,
     const float* __restrict__ norm_w, const float* __restrict__ ss_in, int ss_parts, float eps, float* __restrict__ ss_out,
-    const float* __restrict__ next_w, bf16* __restrict__ xw_out, int rs) {
+    const float* __restrict__ next_w, bf16* __restrict__ xw_out, int rs, int grp_rows, int grp_last,
+    long long grp_stride) {
   constexpr bool NORM = PRO == NORMED;
   constexpr int MP = 8 * MB;
   constexpr int WARPS = GW, THREADS = GW * 32, SPW = K / 32 / GW;   // of a group; SPW: 32-wide k steps a warp
@@ -285,20 +290,25 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
   constexpr bool STAGED = PRO != PLAIN;   // the block's activations are in shared memory
   const bf16* a_frag = A + (size_t)g * lda + k_warp;
   const size_t a_mb = (size_t)8 * lda;
+  // where the activations of a tile's group of products start (one group: at A)
+  auto group_of = [&](int tl) {
+    return grp_rows > 0 ? a_frag + (size_t)min(tl * TILE_N / grp_rows, grp_last) * grp_stride : a_frag;
+  };
   const bf16* a_row[MB];   // STAGED: where batch row mb * 8 + g lies (the row of zeros from rs on)
 #pragma unroll
   for (int mb = 0; mb < MB; ++mb) a_row[mb] = a_res + (size_t)(mb * 8 + g < rs ? mb * 8 + g : rs) * KA + k_warp;
   // plain activations come from L2 AD steps ahead, in a ring of registers of their own
   constexpr int AD = STAGED ? 1 : pick_ahead(CHUNK, MB == 1 ? 5 : 4);
   uint4 ar[MB][AD];
-  auto plain_a = [&](int mb, int step) {
-    return mb * 8 + g < M ? ld_prev(reinterpret_cast<const uint4*>(a_frag + mb * a_mb + step * 32)) : zero;
+  const bf16* a_cur = PRO == PLAIN ? group_of(tile) : a_frag;
+  auto plain_a = [&](const bf16* from, int mb, int step) {
+    return mb * 8 + g < M ? ld_prev(reinterpret_cast<const uint4*>(from + mb * a_mb + step * 32)) : zero;
   };
   if (!STAGED && tile < n_tiles) {
 #pragma unroll
     for (int mb = 0; mb < MB; ++mb)
 #pragma unroll
-      for (int u = 0; u < AD; ++u) ar[mb][u] = plain_a(mb, u);
+      for (int u = 0; u < AD; ++u) ar[mb][u] = plain_a(a_cur, mb, u);
   }
   for (; tile < n_tiles; tile += gridDim.x * GROUPS) {
     float acc[MB][4];
@@ -310,6 +320,7 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
     const bool has_next = next < n_tiles;
     const bf16 *nw0 = nullptr, *nw1 = nullptr;
     if (has_next) rows_of(next, nw0, nw1);
+    const bf16* a_next = PRO == PLAIN && has_next ? group_of(next) : a_cur;
 
 #pragma unroll
     for (int s = 0; s < SPWP; ++s) {
@@ -321,9 +332,9 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
           mma16816(acc[mb], wa[u].x, wb[u].x, wa[u].y, wb[u].y, a.x, a.y);
           mma16816(acc[mb], wa[u].z, wb[u].z, wa[u].w, wb[u].w, a.z, a.w);
         }
-        if (!STAGED) {   // the slot takes the step AD further on; the activations are the same for every tile
+        if (!STAGED) {   // the slot takes the step AD further on; the activations are the same for every tile of a group
           const int ta = s + AD < SPWP ? s + AD : s + AD - SPWP;
-          if (ta < SPW && (s + AD < SPWP || has_next)) ar[mb][s % AD] = plain_a(mb, ta);
+          if (ta < SPW && (s + AD < SPWP || has_next)) ar[mb][s % AD] = plain_a(s + AD < SPWP ? a_cur : a_next, mb, ta);
         }
       }
       // these registers take the step CHUNK further on: of this tile, or of the block's next one, whose
@@ -340,6 +351,7 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
     }
     w0 = nw0;
     w1 = nw1;
+    a_cur = a_next;
 
     if (PRO == SCALED && !inv_done) {
       inv_done = true;
@@ -428,7 +440,7 @@ template <int MB, int PRO, int GROUPS, int GW> size_t smem_of(int staged) {
 template <int MB, int MODE, int PRO, int GROUPS, int GW>
 int launch4(const void* A, int lda, const void* W, void* C, int ldc, int M, int N, const float* norm_w,
             const float* ss_in, int ss_parts, float eps, float* ss_out, const float* next_w, void* xw_out, int pdl,
-            int rs, int staged, int blocks_per_sm, cudaStream_t st) {
+            int rs, int staged, int blocks_per_sm, int grp_rows, int grp_last, long long grp_stride, cudaStream_t st) {
   constexpr int MP = 8 * MB;
   const size_t smem = smem_of<MB, PRO, GROUPS, GW>(staged);
   const size_t smem_max = smem_of<MB, PRO, GROUPS, GW>(PRO == PLAIN ? 0 : MP);
@@ -460,7 +472,7 @@ int launch4(const void* A, int lda, const void* W, void* C, int ldc, int M, int 
   cfg.attrs = attr;
   cfg.numAttrs = pdl ? 1 : 0;
   cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_decode_kernel<MB, MODE, PRO, GROUPS, GW>, (const bf16*)A, lda, (const bf16*)W, C, ldc,
-                                     M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, (bf16*)xw_out, rs);
+                                     M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, (bf16*)xw_out, rs, grp_rows, grp_last, grp_stride);
   if (e != cudaSuccess) return (int)e;
   return launch_status();
 }
@@ -472,12 +484,12 @@ int launch4(const void* A, int lda, const void* W, void* C, int ldc, int M, int 
 template <int MB, int MODE, int PRO>
 int launch3(const void* A, int lda, const void* W, void* C, int ldc, int M, int N, const float* norm_w,
             const float* ss_in, int ss_parts, float eps, float* ss_out, const float* next_w, void* xw_out, int pdl,
-            cudaStream_t st) {
+            int grp_rows, int grp_last, long long grp_stride, cudaStream_t st) {
   constexpr int MP = 8 * MB;
   const int rs = M < MP ? M : MP;                                  // activation rows there are
   const int staged = PRO == PLAIN ? 0 : (rs < MP ? rs + 1 : MP);   // and the row of zeros behind them
 #define DRYFT_GO(GROUPS, GW, PER_SM) \
-  launch4<MB, MODE, PRO, GROUPS, GW>(A, lda, W, C, ldc, M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, xw_out, pdl, rs, staged, PER_SM, st)
+  launch4<MB, MODE, PRO, GROUPS, GW>(A, lda, W, C, ldc, M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, xw_out, pdl, rs, staged, PER_SM, grp_rows, grp_last, grp_stride, st)
   constexpr int WIDE = (K % 512 == 0 && K / 512 >= 8 && PRO != SCALED) ? 16 : 8;   // 16 warps on one tile where a warp keeps 8 steps
   const int n_tiles = MODE == SILU ? (N + 7) / 8 : (N + ROWS - 1) / ROWS;
   // (decided by what 8 / 16 rows would need, not by M: the split of K, and with it the order of the sums,
@@ -492,12 +504,12 @@ int launch3(const void* A, int lda, const void* W, void* C, int ldc, int M, int 
 struct Args {
   const void* A; int lda; const void* W; void* C; int ldc; int M; int N;
   const float* norm_w; const float* ss_in; int ss_parts; float eps; float* ss_out; const float* next_w; void* xw_out;
-  int pdl; cudaStream_t st;
+  int pdl; int grp_rows, grp_last; long long grp_stride; cudaStream_t st;
 };
 template <int MB, int MODE, int PRO>
 int launch_a(const Args& a) {
   return launch3<MB, MODE, PRO>(a.A, a.lda, a.W, a.C, a.ldc, a.M, a.N, a.norm_w, a.ss_in, a.ss_parts, a.eps, a.ss_out, a.next_w,
-                                a.xw_out, a.pdl, a.st);
+                                a.xw_out, a.pdl, a.grp_rows, a.grp_last, a.grp_stride, a.st);
 }
 template <int MB, int MODE>
 int launch2(int pro, const Args& a) {
@@ -522,9 +534,11 @@ DRYFT_API int dryft_gemm_decode_k() { return K; }
 // next_w [N] and xw_out [M, ldc], the weighted activations T(x * next_w) for the product after it.
 // scaled != 0: A holds such weighted activations; the sums are scaled by rsqrt(mean(x^2) + eps) from
 // ss_in (norm_w is not read).
+// grp_rows > 0 (a multiple of 16): products of several activations in one launch, see the top of this file; grp_count groups.
 DRYFT_API int dryft_gemm_decode(const void* A, int lda, const void* W, void* C, int ldc, int mode, int M, int N,
                                 const float* norm_w, const float* ss_in, int ss_parts, float eps, float* ss_out, int pdl,
-                                int scaled, const float* next_w, void* xw_out, cudaStream_t st) {
+                                int scaled, const float* next_w, void* xw_out, int grp_rows, int grp_count, long long grp_stride,
+                                cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
   if ((lda & 7) || M > 16) return DRYFT_ERR_UNSUPPORTED;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return DRYFT_ERR_UNSUPPORTED;
@@ -532,6 +546,9 @@ DRYFT_API int dryft_gemm_decode(const void* A, int lda, const void* W, void* C, 
   if (pro != PLAIN && (!ss_in || ss_parts <= 0)) return DRYFT_ERR_UNSUPPORTED;
   if (pro == NORMED && ((uintptr_t)norm_w & 15)) return DRYFT_ERR_UNSUPPORTED;
   if ((xw_out != nullptr) != (next_w != nullptr) || (xw_out && mode != RESIDUAL)) return DRYFT_ERR_UNSUPPORTED;
-  Args a = {A, lda, W, C, ldc, M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, xw_out, pdl, st};
+  if (grp_rows < 0 || (grp_rows > 0 && (grp_rows % ROWS || grp_count < 1 || (grp_stride & 7) || pro != PLAIN || mode == SILU)))
+    return DRYFT_ERR_UNSUPPORTED;
+  Args a = {A, lda, W, C, ldc, M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, xw_out, pdl, grp_rows, grp_count - 1,
+            grp_stride, st};
   return M <= 8 ? launch1<1>(mode, pro, a) : launch1<2>(mode, pro, a);
 }

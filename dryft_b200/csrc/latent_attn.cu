@@ -15,7 +15,7 @@
 //                    tokens splits each token's keys over several blocks, joined by latent_combine.  The query's rotated part is rotated here.  Heads-major input and output:
 //                    q_lat [H, N, kv_rank] (32-bit), q [N, H, q_stride] with the rotated part at q_rot_off,
 //                    o_lat [H, N, kv_rank].
-// head_gate          out[n, h, :] = T( o[h, n, :] * sigmoid(gate_logit[n, h]) )
+// head_gate          out[n, h, :] = T( o[h, n, :] * sigmoid(gate_logit[n, h]) )      (`per_value`: gate_logit[n, h * V + v], here and below)
 //
 // Rotation: pairs (2i, 2i+1) when `interleaved`, else (i, i + R/2); angle = position * inv_freq[i] (sincos_split below).
 // Norms, angles, scores, softmax and the weighted sum are 32-bit whatever the cache type T.  Sizes are runtime arguments
@@ -343,7 +343,7 @@ __global__ void latent_combine_kernel(const float* __restrict__ part, const int*
 
 template <typename T>
 __global__ void head_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_ld, T* __restrict__ out,
-                                 int n_tokens, int H, int vdim) {
+                                 int n_tokens, int H, int vdim, int per_value) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (size_t)n_tokens * H * vdim) return;
   const int v = (int)(i % vdim);
@@ -351,7 +351,7 @@ __global__ void head_gate_kernel(const float* __restrict__ o, const T* __restric
   const size_t n = i / ((size_t)vdim * H);
   float val = o[((size_t)hd * n_tokens + n) * vdim + v];
   if (gate) {
-    const float g = to_f32<T>(gate[n * gate_ld + hd]);
+    const float g = to_f32<T>(gate[n * gate_ld + (per_value ? hd * vdim + v : hd)]);
     val *= 1.f / (1.f + expf(-g));
   }
   out[i] = from_f32<T>(val);
@@ -364,7 +364,7 @@ __global__ void head_gate_kernel(const float* __restrict__ o, const T* __restric
 //
 // latent_scratch_table   table[slot_b][p] = (pages of the sequences before b) + p   for the step's sequences
 // latent_expand_store    per token: q_out[n, h] = [q_plain | rotate(q_rot)], key page row = [k_plain,h | rotate(k_rot)],
-//                        value page row = [v_h | zeros]  (all of the head size `hd` >= the value size)
+//                        value page row = [v_h | zeros]  (`vw` entries: the head size `hd`, or any width from the value size up)
 // head_gate_rows         out[n, h*V + v] = T( o[n, h, v] * sigmoid(gate_logit[n, h]) )   for o [n, H, hd]
 __global__ void latent_scratch_table_kernel(const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int n_seqs,
                                             int* __restrict__ table, int max_pages, int page_size) {
@@ -383,7 +383,7 @@ __global__ void __launch_bounds__(PREP_THREADS) latent_expand_store_kernel(
     const T* __restrict__ q, const T* __restrict__ kv, int kv_ld, int v_off, const T* __restrict__ proj, int ld, int krot_off,
     const float* __restrict__ inv_freq, const float* __restrict__ inv_freq_lo, int interleaved,
     const int* __restrict__ tok_slot, const int* __restrict__ tok_pos, const int* __restrict__ table, int max_pages,
-    int page_size, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, int H, int dim, int rot, int vdim) {
+    int page_size, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, int H, int dim, int rot, int vdim, int vw) {
   extern __shared__ __align__(16) float buf[];   // [rot] the shared key part, rotated; then [H][rot] raw query parts
   const int n = blockIdx.x;
   const int slot = tok_slot[n];
@@ -409,20 +409,25 @@ __global__ void __launch_bounds__(PREP_THREADS) latent_expand_store_kernel(
     }
     q_out[((size_t)n * H + h) * hd + d] = qv;
     k_pages[at] = kvv;
-    v_pages[at] = d < vdim ? kv[(size_t)n * kv_ld + v_off + h * vdim + d] : from_f32<T>(0.f);
+    if (vw == hd) v_pages[at] = d < vdim ? kv[(size_t)n * kv_ld + v_off + h * vdim + d] : from_f32<T>(0.f);
   }
+  if (vw != hd)
+    for (int i = threadIdx.x; i < H * vw; i += PREP_THREADS) {
+      const int h = i / vw, d = i % vw;
+      v_pages[((page * H + h) * page_size + pos % page_size) * vw + d] = d < vdim ? kv[(size_t)n * kv_ld + v_off + h * vdim + d] : from_f32<T>(0.f);
+    }
 }
 
 template <typename T>
 __global__ void head_gate_rows_kernel(const T* __restrict__ o, int hd, const T* __restrict__ gate, int gate_ld,
-                                      T* __restrict__ out, int n_tokens, int H, int vdim) {
+                                      T* __restrict__ out, int n_tokens, int H, int vdim, int per_value) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= (size_t)n_tokens * H * vdim) return;
   const int v = (int)(i % vdim);
   const int h = (int)((i / vdim) % H);
   const size_t n = i / ((size_t)vdim * H);
   float val = to_f32<T>(o[(n * H + h) * hd + v]);
-  if (gate) val *= 1.f / (1.f + expf(-to_f32<T>(gate[n * gate_ld + h])));
+  if (gate) val *= 1.f / (1.f + expf(-to_f32<T>(gate[n * gate_ld + (per_value ? h * vdim + v : h)])));
   out[i] = from_f32<T>(val);
 }
 
@@ -449,18 +454,18 @@ __global__ void latent_fold_q_kernel(const T* __restrict__ q, int q_stride, cons
 
 template <typename T>
 __global__ void latent_unfold_o_kernel(const T* __restrict__ o_lat, const T* __restrict__ w, const T* __restrict__ gate,
-                                       int gate_ld, T* __restrict__ out, int n_tokens, int H, int kv_rank, int vdim) {
+                                       int gate_ld, T* __restrict__ out, int n_tokens, int H, int kv_rank, int vdim, int per_value) {
   extern __shared__ __align__(16) float vin[];
   const int n = blockIdx.x, h = blockIdx.y;
   for (int r = threadIdx.x; r < kv_rank; r += blockDim.x) vin[r] = to_f32<T>(o_lat[((size_t)h * n_tokens + n) * kv_rank + r]);
   __syncthreads();
-  const float g = gate ? 1.f / (1.f + expf(-to_f32<T>(gate[(size_t)n * gate_ld + h]))) : 1.f;
+  auto gate_of = [&](int v) { return gate ? 1.f / (1.f + expf(-to_f32<T>(gate[(size_t)n * gate_ld + (per_value ? h * vdim + v : h)]))) : 1.f; };
   const T* wh = w + (size_t)h * kv_rank * vdim;
   for (int v = threadIdx.x; v < vdim; v += blockDim.x) {
     float acc = 0.f;
 #pragma unroll 8
     for (int r = 0; r < kv_rank; ++r) acc = fmaf(vin[r], to_f32<T>(wh[(size_t)r * vdim + v]), acc);
-    out[((size_t)n * H + h) * vdim + v] = from_f32<T>(acc * g);
+    out[((size_t)n * H + h) * vdim + v] = from_f32<T>(acc * gate_of(v));
   }
 }
 
@@ -553,7 +558,7 @@ DRYFT_API int dryft_latent_fold_q(int is_bf16, const void* q, int q_stride, cons
 }
 
 DRYFT_API int dryft_latent_unfold_o(int is_bf16, const void* o_lat, const void* w, const void* gate, int gate_ld, void* out, int n_tokens,
-                                    int H, int kv_rank, int vdim, cudaStream_t st) {
+                                    int H, int kv_rank, int vdim, int per_value, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
   if (H <= 0 || H > 65535 || vdim <= 0 || kv_rank <= 0 || kv_rank > 12000) return DRYFT_ERR_UNSUPPORTED;
   typedef __nv_bfloat16 bf;
@@ -562,10 +567,10 @@ DRYFT_API int dryft_latent_unfold_o(int is_bf16, const void* o_lat, const void* 
   dim3 grid(n_tokens, H);
   if (is_bf16)
     latent_unfold_o_kernel<bf><<<grid, threads, smem, st>>>((const bf*)o_lat, (const bf*)w, (const bf*)gate, gate_ld, (bf*)out, n_tokens, H,
-                                                            kv_rank, vdim);
+                                                            kv_rank, vdim, per_value);
   else
     latent_unfold_o_kernel<float><<<grid, threads, smem, st>>>((const float*)o_lat, (const float*)w, (const float*)gate, gate_ld, (float*)out,
-                                                               n_tokens, H, kv_rank, vdim);
+                                                               n_tokens, H, kv_rank, vdim, per_value);
   return launch_status();
 }
 
@@ -580,42 +585,42 @@ DRYFT_API int dryft_latent_expand_store(int is_bf16, const void* q, const void* 
                                         int krot_off, const float* inv_freq, const float* inv_freq_lo, int interleaved,
                                         const int* tok_slot, const int* tok_pos, const int* table, int max_pages, int page_size,
                                         void* q_out, void* k_pages, void* v_pages, int n, int H, int dim, int rot, int vdim,
-                                        cudaStream_t st) {
+                                        int vw, cudaStream_t st) {
   if (n <= 0) return 0;
-  if (H <= 0 || dim <= 0 || rot < 0 || (rot & 1) || vdim > dim + rot) return DRYFT_ERR_UNSUPPORTED;
+  if (H <= 0 || dim <= 0 || rot < 0 || (rot & 1) || vw < vdim) return DRYFT_ERR_UNSUPPORTED;
   typedef __nv_bfloat16 bf;
   const size_t smem = sizeof(float) * ((size_t)rot * (H + 1) + 1);
   if (smem > 48 * 1024) return DRYFT_ERR_UNSUPPORTED;
   if (is_bf16)
     latent_expand_store_kernel<bf><<<n, PREP_THREADS, smem, st>>>((const bf*)q, (const bf*)kv, kv_ld, v_off, (const bf*)proj, ld, krot_off,
                                                                   inv_freq, inv_freq_lo, interleaved, tok_slot, tok_pos, table, max_pages,
-                                                                  page_size, (bf*)q_out, (bf*)k_pages, (bf*)v_pages, H, dim, rot, vdim);
+                                                                  page_size, (bf*)q_out, (bf*)k_pages, (bf*)v_pages, H, dim, rot, vdim, vw);
   else
     latent_expand_store_kernel<float><<<n, PREP_THREADS, smem, st>>>((const float*)q, (const float*)kv, kv_ld, v_off, (const float*)proj,
                                                                      ld, krot_off, inv_freq, inv_freq_lo, interleaved, tok_slot, tok_pos,
                                                                      table, max_pages, page_size, (float*)q_out, (float*)k_pages,
-                                                                     (float*)v_pages, H, dim, rot, vdim);
+                                                                     (float*)v_pages, H, dim, rot, vdim, vw);
   return launch_status();
 }
 
 DRYFT_API int dryft_head_gate_rows(int is_bf16, const void* o, int hd, const void* gate, int gate_ld, void* out, int n_tokens, int H,
-                                   int vdim, cudaStream_t st) {
+                                   int vdim, int per_value, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
   typedef __nv_bfloat16 bf;
   const size_t total = (size_t)n_tokens * H * vdim;
   const unsigned blocks = (unsigned)((total + 255) / 256);
-  if (is_bf16) head_gate_rows_kernel<bf><<<blocks, 256, 0, st>>>((const bf*)o, hd, (const bf*)gate, gate_ld, (bf*)out, n_tokens, H, vdim);
-  else head_gate_rows_kernel<float><<<blocks, 256, 0, st>>>((const float*)o, hd, (const float*)gate, gate_ld, (float*)out, n_tokens, H, vdim);
+  if (is_bf16) head_gate_rows_kernel<bf><<<blocks, 256, 0, st>>>((const bf*)o, hd, (const bf*)gate, gate_ld, (bf*)out, n_tokens, H, vdim, per_value);
+  else head_gate_rows_kernel<float><<<blocks, 256, 0, st>>>((const float*)o, hd, (const float*)gate, gate_ld, (float*)out, n_tokens, H, vdim, per_value);
   return launch_status();
 }
 
 DRYFT_API int dryft_head_gate(int is_bf16, const float* o, const void* gate, int gate_ld, void* out, int n_tokens, int H, int vdim,
-                              cudaStream_t st) {
+                              int per_value, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
   typedef __nv_bfloat16 bf;
   const size_t total = (size_t)n_tokens * H * vdim;
   const unsigned blocks = (unsigned)((total + 255) / 256);
-  if (is_bf16) head_gate_kernel<bf><<<blocks, 256, 0, st>>>(o, (const bf*)gate, gate_ld, (bf*)out, n_tokens, H, vdim);
-  else head_gate_kernel<float><<<blocks, 256, 0, st>>>(o, (const float*)gate, gate_ld, (float*)out, n_tokens, H, vdim);
+  if (is_bf16) head_gate_kernel<bf><<<blocks, 256, 0, st>>>(o, (const bf*)gate, gate_ld, (bf*)out, n_tokens, H, vdim, per_value);
+  else head_gate_kernel<float><<<blocks, 256, 0, st>>>(o, (const float*)gate, gate_ld, (float*)out, n_tokens, H, vdim, per_value);
   return launch_status();
 }

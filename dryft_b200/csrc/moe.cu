@@ -5,7 +5,9 @@
 //                 is restricted to the `keep` highest-ranked groups
 //                 (n_groups = keep = 1: no groups).  The `top` allowed experts with the largest scores are chosen;
 //                 their weights are the scores themselves, or the scores divided by their sum (`renorm`: the softmax
-//                 over the chosen logits only).  `bias` (optional, [E]) is added to the logits first.
+//                 over the chosen logits only; `renorm_eps` joins that sum).  `corr` (optional, [E]) is added to the scores that experts and
+//                 groups are chosen by, never to the weights, and bit 2 of `renorm` ranks a group by the sum of its two largest.
+//                 `bias` (optional, [E]) is added to the logits first.
 //                 Ties go to the lower index.  One warp per token.  moe_route_rows is the same for few tokens with the
 //                 router's product inside (one block per token, one launch instead of two).
 //   moe_rows      an assignment a = (token, k) multiplies its token's activation row by its expert's matrices, every
@@ -36,13 +38,14 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
-// One warp's choice for one token: z holds the E logits (global or shared memory), s and gs are the warp's scratch
-// ([E] scores, [n_groups] group scores) in shared memory.
-__device__ __forceinline__ void route_one(const float* z, const float* __restrict__ bias, float* s, float* gs, int lane, int n, int E,
-                                          int n_groups, int keep, int top, int renorm, int* __restrict__ idx_out,
-                                          float* __restrict__ w_out) {
-  const bool sigmoid_scores = renorm >= 2;      // bit 1 of `renorm`: every expert's score is the sigmoid of its own logit
-  renorm &= 1;
+constexpr float SHUT_OUT = -3.402823466e38f;   // choice score of an expert outside the kept groups: below every score there is
+
+// One warp's choice for one token: z holds the E logits (global or shared memory); s, ch and gs are the warp's scratch
+// ([E] scores, [E] scores the choice goes by, [n_groups] group scores) in shared memory.  A score taken becomes -inf.
+__device__ __forceinline__ void route_one(const float* z, const float* __restrict__ bias, const float* __restrict__ corr, float* s, float* ch,
+                                          float* gs, int lane, int n, int E, int n_groups, int keep, int top, int flags, float renorm_eps,
+                                          int* __restrict__ idx_out, float* __restrict__ w_out) {
+  const bool renorm = flags & 1, sigmoid_scores = flags & 2, by_two = flags & 4;
   if (sigmoid_scores) {
     for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-(z[e] + (bias != nullptr ? bias[e] : 0.f))));
   } else {
@@ -59,59 +62,65 @@ __device__ __forceinline__ void route_one(const float* z, const float* __restric
     __syncwarp();
     for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
   }
+  for (int e = lane; e < E; e += 32) ch[e] = s[e] + (corr != nullptr ? corr[e] : 0.f);     // the lane's own entries
   __syncwarp();
   if (n_groups > 1) {
     const int gsz = E / n_groups;
     for (int g = lane; g < n_groups; g += 32) {
-      float m = -1.f;
-      for (int j = 0; j < gsz; ++j) m = fmaxf(m, s[g * gsz + j]);
-      gs[g] = m;
+      float m = SHUT_OUT, m2 = SHUT_OUT;      // the largest and the second
+      for (int j = 0; j < gsz; ++j) {
+        const float c = ch[g * gsz + j];
+        if (c > m) { m2 = m; m = c; } else if (c > m2) m2 = c;
+      }
+      gs[g] = by_two && gsz > 1 ? m + m2 : m;
     }
     __syncwarp();
-    // take the `keep` best groups away one by one (marking them -2); what is left at the end is shut out
+    // take the `keep` best groups away one by one (marking them -inf); what is left at the end is shut out
     for (int r = 0; r < keep; ++r) {
-      float bv = -1.5f;
+      float bv = -INFINITY;
       int bi = 0x7fffffff;
       for (int g = lane; g < n_groups; g += 32)
         if (gs[g] > bv) { bv = gs[g]; bi = g; }
       warp_argmax(bv, bi);
-      if (lane == 0 && bi < n_groups) gs[bi] = -2.f;
+      if (lane == 0 && bi < n_groups) gs[bi] = -INFINITY;
       __syncwarp();
     }
     for (int e = lane; e < E; e += 32)
-      if (gs[e / gsz] != -2.f) s[e] = -1.f;
+      if (gs[e / gsz] != -INFINITY) ch[e] = SHUT_OUT;
     __syncwarp();
   }
   float wsum = 0.f;
   for (int r = 0; r < top; ++r) {
-    float bv = -2.f;
+    float bv = -INFINITY;
     int bi = 0x7fffffff;
     for (int e = lane; e < E; e += 32)
-      if (s[e] > bv) { bv = s[e]; bi = e; }
+      if (ch[e] > bv) { bv = ch[e]; bi = e; }
     warp_argmax(bv, bi);
-    if (bi >= E) { bi = 0; bv = 0.f; }   // nothing comparable left (a NaN row): a defined choice of weight zero
-    if (bv < 0.f) bv = 0.f;              // fewer allowed experts than `top`
+    float w = 0.f;
+    if (bi >= E) bi = 0;                           // nothing comparable left (a NaN row): a defined choice of weight zero
+    else if (bv > SHUT_OUT) w = s[bi];             // else fewer allowed experts than `top`: weight zero
     if (lane == 0) {
       idx_out[(size_t)n * top + r] = bi;
-      w_out[(size_t)n * top + r] = bv;
-      s[bi] = -2.f;
+      w_out[(size_t)n * top + r] = w;
+      ch[bi] = -INFINITY;
     }
-    wsum += bv;
+    wsum += w;
     __syncwarp();
   }
+  wsum += renorm_eps;
   if (renorm && lane == 0 && wsum > 0.f)
     for (int r = 0; r < top; ++r) w_out[(size_t)n * top + r] /= wsum;
 }
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(
-    const float* __restrict__ logits, const float* __restrict__ bias, int n_tokens, int E, int n_groups, int keep, int top, int renorm,
-    int* __restrict__ idx_out, float* __restrict__ w_out) {
+    const float* __restrict__ logits, const float* __restrict__ bias, const float* __restrict__ corr, int n_tokens, int E, int n_groups, int keep,
+    int top, int renorm, float renorm_eps, int* __restrict__ idx_out, float* __restrict__ w_out) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = blockIdx.x * ROUTE_WARPS + warp;
   if (n >= n_tokens) return;
-  float* s = sm + (size_t)warp * (E + n_groups);
-  route_one(logits + (size_t)n * E, bias, s, s + E, lane, n, E, n_groups, keep, top, renorm, idx_out, w_out);
+  float* s = sm + (size_t)warp * (2 * E + n_groups);
+  route_one(logits + (size_t)n * E, bias, corr, s, s + E, s + 2 * E, lane, n, E, n_groups, keep, top, renorm, renorm_eps, idx_out, w_out);
 }
 
 // Few tokens (decode): the router's product and its choice in one launch.  One block per token: the token's row is staged
@@ -119,11 +128,11 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(
 constexpr int ROUTE_ROW_THREADS = 1024;   // 32 warps: one or two experts a warp keeps the block one or two trips to memory long
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_ROW_THREADS) moe_route_rows_kernel(
-    const T* __restrict__ h, const T* __restrict__ w_router, const float* __restrict__ bias, int K, int E, int n_groups, int keep, int top,
-    int renorm, int* __restrict__ idx_out, float* __restrict__ w_out) {
+    const T* __restrict__ h, const T* __restrict__ w_router, const float* __restrict__ bias, const float* __restrict__ corr, int K, int E,
+    int n_groups, int keep, int top, int renorm, float renorm_eps, int* __restrict__ idx_out, float* __restrict__ w_out) {
   extern __shared__ __align__(16) unsigned char smraw[];
   T* xs = reinterpret_cast<T*>(smraw);                  // the token's row
-  float* z = reinterpret_cast<float*>(smraw + (sizeof(T) * (size_t)K + 15) / 16 * 16);   // [E] logits, [E] scores, [n_groups]
+  float* z = reinterpret_cast<float*>(smraw + (sizeof(T) * (size_t)K + 15) / 16 * 16);   // [E] logits, [E] scores, [E] choice scores, [n_groups]
   const int n = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   for (int c = threadIdx.x; c < K; c += ROUTE_ROW_THREADS) xs[c] = h[(size_t)n * K + c];
   __syncthreads();
@@ -147,7 +156,7 @@ __global__ void __launch_bounds__(ROUTE_ROW_THREADS) moe_route_rows_kernel(
     if (lane == 0) z[e] = d;
   }
   __syncthreads();
-  if (warp == 0) route_one(z, bias, z + E, z + 2 * E, lane, n, E, n_groups, keep, top, renorm, idx_out, w_out);
+  if (warp == 0) route_one(z, bias, corr, z + E, z + 2 * E, z + 3 * E, lane, n, E, n_groups, keep, top, renorm, renorm_eps, idx_out, w_out);
 }
 
 constexpr int ROWS_THREADS = 128;
@@ -261,14 +270,14 @@ int rows_launch(const void* a_in, int a_div, const void* w, const int* idx, int 
 }
 }  // namespace
 
-DRYFT_API int dryft_moe_route(const float* logits, const float* bias, int n_tokens, int E, int n_groups, int keep, int top, int renorm,
-                              int* idx_out, float* w_out, cudaStream_t st) {
+DRYFT_API int dryft_moe_route(const float* logits, const float* bias, const float* corr, int n_tokens, int E, int n_groups, int keep, int top,
+                              int renorm, float renorm_eps, int* idx_out, float* w_out, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
   if (E < 1 || top < 1 || top > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups) return DRYFT_ERR_UNSUPPORTED;
-  const size_t smem = sizeof(float) * (size_t)ROUTE_WARPS * (E + n_groups);
+  const size_t smem = sizeof(float) * (size_t)ROUTE_WARPS * (2 * E + n_groups);
   if (smem > 48 * 1024) return DRYFT_ERR_UNSUPPORTED;
-  moe_route_kernel<<<(n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS, ROUTE_WARPS * 32, smem, st>>>(logits, bias, n_tokens, E, n_groups, keep,
-                                                                                               top, renorm, idx_out, w_out);
+  moe_route_kernel<<<(n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS, ROUTE_WARPS * 32, smem, st>>>(logits, bias, corr, n_tokens, E, n_groups,
+                                                                                               keep, top, renorm, renorm_eps, idx_out, w_out);
   return launch_status();
 }
 
@@ -288,17 +297,17 @@ DRYFT_API int dryft_moe_combine(int is_bf16, const void* y, const float* wts, in
   return launch_status();
 }
 
-DRYFT_API int dryft_moe_route_rows(int is_bf16, const void* h, const void* w_router, const float* bias, int n_tokens, int K, int E, int n_groups,
-                                   int keep, int top, int renorm, int* idx_out, float* w_out, cudaStream_t st) {
+DRYFT_API int dryft_moe_route_rows(int is_bf16, const void* h, const void* w_router, const float* bias, const float* corr, int n_tokens, int K, int E,
+                                   int n_groups, int keep, int top, int renorm, float renorm_eps, int* idx_out, float* w_out, cudaStream_t st) {
   if (n_tokens <= 0) return 0;
   if (E < 1 || top < 1 || top > E || n_groups < 1 || E % n_groups || keep < 1 || keep > n_groups || K < 1) return DRYFT_ERR_UNSUPPORTED;
-  const size_t smem = sizeof(float) * (size_t)(2 * E + n_groups) + ((is_bf16 ? 2 : 4) * (size_t)K + 15) / 16 * 16;
+  const size_t smem = sizeof(float) * (size_t)(3 * E + n_groups) + ((is_bf16 ? 2 : 4) * (size_t)K + 15) / 16 * 16;
   if (smem > 48 * 1024) return DRYFT_ERR_UNSUPPORTED;
   if (is_bf16)
     moe_route_rows_kernel<__nv_bfloat16><<<n_tokens, ROUTE_ROW_THREADS, smem, st>>>((const __nv_bfloat16*)h, (const __nv_bfloat16*)w_router,
-                                                                                    bias, K, E, n_groups, keep, top, renorm, idx_out, w_out);
+                                                                                    bias, corr, K, E, n_groups, keep, top, renorm, renorm_eps, idx_out, w_out);
   else
-    moe_route_rows_kernel<float><<<n_tokens, ROUTE_ROW_THREADS, smem, st>>>((const float*)h, (const float*)w_router, bias, K, E, n_groups, keep,
-                                                                            top, renorm, idx_out, w_out);
+    moe_route_rows_kernel<float><<<n_tokens, ROUTE_ROW_THREADS, smem, st>>>((const float*)h, (const float*)w_router, bias, corr, K, E, n_groups,
+                                                                            keep, top, renorm, renorm_eps, idx_out, w_out);
   return launch_status();
 }

@@ -13,6 +13,8 @@
 //                     the angle pos * inv_freq[i], evaluated in 32-bit), THEN divided by their root mean square over D
 //                     (no weight; skipped when eps < 0); v (+ bias); k and v written into the cache at the token's position.  A warp a vector, or several of
 //                     one token in a step of many tokens.
+//                     `v_eps` >= 0: each value head is divided by its root mean square too, and cached so.  `qt_every` > 0: the
+//                     query of position p is multiplied by 1 + qt_coef * ln((p + 1) / qt_every + 1), whole quotient.
 //                     With convolution weights (shortconv.cuh) q, k and v first pass a short causal convolution per channel
 //                     of [q | k | v], and a decode step stores its own projected values in the convolution's ring.
 //   pool_attn_prep_run  the same behind a convolution for steps of many tokens: a block a run of eight tokens, a warp a vector of
@@ -62,7 +64,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
     const float* __restrict__ inv_freq, const float* __restrict__ inv_freq_lo, int rot, const int* __restrict__ tok_slot,
     const int* __restrict__ tok_pos, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, const int* __restrict__ page_table, int max_pages,
     int page_size, int n_tokens, int H, int G, float eps, int write_kv, const float* __restrict__ conv_w, int taps, T* __restrict__ ring,
-    int store_ring, int per_warp) {
+    int store_ring, int per_warp, float v_eps, float qt_coef, int qt_every) {
   __shared__ float sm[PREP_WARPS][D > DV ? D : DV];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int per_tok = H + (write_kv ? 2 * G : 0), parts = (per_tok + per_warp - 1) / per_warp;
@@ -109,6 +111,23 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
     }
     if (vec >= H + G) {     // a value vector: bias, cache
       const int g = vec - H - G, src = H * D + G * D + g * DV;
+      if (v_eps >= 0.f) {   // divided by its root mean square
+        float vv[DVR];
+        float ss = 0.f;
+#pragma unroll
+        for (int r = 0; r < DVR; ++r) {
+          const int c = lane + 32 * r;
+          vv[r] = c < DV ? input(src + c) + (vb != nullptr ? vb[g * DV + c] : 0.f) : 0.f;
+          ss = fmaf(vv[r], vv[r], ss);
+        }
+        const float vinv = 1.f / sqrtf(warp_sum(ss) / (float)DV + v_eps);
+#pragma unroll
+        for (int r = 0; r < DVR; ++r) {
+          const int c = lane + 32 * r;
+          if (c < DV) v_pages[cache_row * DV + c] = from_f32<T>(vv[r] * vinv);
+        }
+        continue;
+      }
       for (int c = lane; c < DV; c += 32)
         v_pages[cache_row * DV + c] = from_f32<T>(input(src + c) + (vb != nullptr ? vb[g * DV + c] : 0.f));
       continue;
@@ -132,6 +151,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) pool_attn_prep_kernel(
     }
     float rinv = 1.f;                                                      // eps < 0: no unit norm
     if (eps >= 0.f) rinv = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
+    if (is_q && qt_every > 0) rinv *= fmaf(qt_coef, logf((float)((pos + 1) / qt_every + 1)), 1.f);
     T* dst = is_q ? q_out + ((size_t)t * H + hd) * D : k_pages + cache_row * D;
 #pragma unroll
     for (int r = 0; r < DR; ++r) {
@@ -392,13 +412,26 @@ template <typename T> __device__ __forceinline__ float gate_at(const T* __restri
   return gate == nullptr ? 1.f : 1.f / (1.f + expf(-to_f32<T>(gate[(size_t)t * gate_ld + (size_t)head * DV + c])));
 }
 
-template <typename T>
+// How a score is changed before the softmax: squashed to cap * tanh(s / cap) (cap > 0), then r1_h * ln(1 + r2_h * distance) taken off
+// (r1 given; distances in tokens, so not together with pooled rows).  32-bit path: CUDA's tanhf and log1pf; bfloat16 path: the
+// same functions from one exponential and one logarithm, absolute errors below 1e-6 of the cap or of r1.
+struct ScoreMods { float cap; const float* r1; const float* r2; };
+template <typename T> __device__ __forceinline__ float mod_score(float s, float cap, float r1, float r2, float dist) {
+  if (sizeof(T) == 4) {
+    if (cap > 0.f) s = cap * tanhf(s / cap);
+    return s - r1 * log1pf(r2 * dist);
+  }
+  if (cap > 0.f) s = cap - __fdividef(2.f * cap, 1.f + __expf(2.f * s / cap));      // cap * (1 - 2 / (1 + e^(2 s / cap)))
+  return s - r1 * __logf(fmaf(r2, dist, 1.f));
+}
+
+template <typename T, bool MODS>
 __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
     const T* __restrict__ q, const T* __restrict__ k_pages, const T* __restrict__ v_pages, const int* __restrict__ page_table,
     int max_pages, int page_size, const T* __restrict__ pk_pages, const T* __restrict__ pv_pages, const int* __restrict__ pool_table,
     int pool_max_pages, const float* __restrict__ sink, const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     T* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int G, int n_splits, float scale, int size, int P, int keep, const T* __restrict__ gate,
-    int gate_ld) {
+    int gate_ld, ScoreMods mods) {
   __shared__ float qs[REP][D];
   __shared__ float wo[ROWS_WARPS][REP][DV];
   __shared__ float wml[ROWS_WARPS][REP][2];
@@ -419,8 +452,13 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
   __syncthreads();
 
   float m[REP], l[REP], o[REP][DVR];
+  float mr1[MODS ? REP : 1], mr2[MODS ? REP : 1];
 #pragma unroll
   for (int h = 0; h < REP; ++h) {
+    if (MODS) {
+      mr1[h] = mods.r1 != nullptr ? mods.r1[g * REP + h] : 0.f;
+      mr2[h] = mods.r1 != nullptr ? mods.r2[g * REP + h] : 0.f;
+    }
     m[h] = -INFINITY;
     l[h] = 0.f;
 #pragma unroll
@@ -431,6 +469,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
     const bool valid = u < u1;
     const T* kr = k_pages;
     const T* vr = v_pages;
+    float dist = 0.f;
     if (valid) {
       if (u < nb) {
         const int page = pool_table[(size_t)slot * pool_max_pages + u / page_size];
@@ -439,6 +478,7 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
         vr = pv_pages + r * DV;
       } else {
         const int j = u - nb < nk ? u - nb : lo + (u - nb - nk);
+        dist = (float)(i - j);
         const int page = page_table[(size_t)slot * max_pages + j / page_size];
         const size_t r = ((size_t)page * G + g) * page_size + j % page_size;
         kr = k_pages + r * D;
@@ -452,7 +492,8 @@ __global__ void __launch_bounds__(ROWS_WARPS * 32) pool_attn_rows_kernel(
     float pr[REP];
 #pragma unroll
     for (int h = 0; h < REP; ++h) {
-      const float sc = valid ? dots[h] * scale : -INFINITY;
+      float sc = valid ? dots[h] * scale : -INFINITY;
+      if (MODS && valid) sc = mod_score<T>(sc, mods.cap, mr1[h], mr2[h], dist);
       const float mn = fmaxf(m[h], warp_max(sc));          // finite: the tile holds at least one key
       const float corr = expf(m[h] - mn);                  // exp(-inf) = 0 for the first tile
       const float pv = valid ? expf(sc - mn) : 0.f;
@@ -548,7 +589,7 @@ template <typename T>
 int prep_launch(const void* proj, int ld, const float* qb, const float* kb, const float* vb, const float* inv_freq,
                 const float* inv_freq_lo, int rot, const int* tok_slot, const int* tok_pos, void* q_out, void* k_pages, void* v_pages, const int* page_table,
                 int max_pages, int page_size, int n, int H, int G, float eps, int write_kv, const float* conv_w, int taps, void* ring,
-                int store_ring, cudaStream_t st) {
+                int store_ring, float v_eps, float qt_coef, int qt_every, cudaStream_t st) {
   // many tokens: a warp takes several vectors of one token, which share its angles and the rows its convolution reads
   const int per_tok = H + (write_kv ? 2 * G : 0), per_warp = n >= 512 ? 8 : n >= 128 ? 4 : 1;
   const long long items = (long long)n * ((per_tok + per_warp - 1) / per_warp);
@@ -556,7 +597,7 @@ int prep_launch(const void* proj, int ld, const float* qb, const float* kb, cons
   if (blocks > 0x7fffffffLL) return DRYFT_ERR_UNSUPPORTED;
   pool_attn_prep_kernel<T><<<(unsigned)blocks, PREP_WARPS * 32, 0, st>>>(
       (const T*)proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, (T*)q_out, (T*)k_pages, (T*)v_pages, page_table, max_pages,
-      page_size, n, H, G, eps, write_kv, conv_w, taps, (T*)ring, store_ring, per_warp);
+      page_size, n, H, G, eps, write_kv, conv_w, taps, (T*)ring, store_ring, per_warp, v_eps, qt_coef, qt_every);
   return launch_status();
 }
 
@@ -564,11 +605,12 @@ template <typename T>
 int rows_launch(const void* q, const void* k_pages, const void* v_pages, const int* page_table, int max_pages, int page_size,
                 const void* pk, const void* pv, const int* pool_table, int pool_max_pages, const float* sink, const int* tok_slot,
                 const int* tok_pos, void* out, float* part_o, float* part_ml, int n, int G, int n_splits, float scale, int size, int P,
-                int keep, const void* gate, int gate_ld, cudaStream_t st) {
+                int keep, const void* gate, int gate_ld, ScoreMods mods, cudaStream_t st) {
   dim3 grid(n, G, n_splits);
-  pool_attn_rows_kernel<T><<<grid, ROWS_WARPS * 32, 0, st>>>((const T*)q, (const T*)k_pages, (const T*)v_pages, page_table, max_pages,
-                                                            page_size, (const T*)pk, (const T*)pv, pool_table, pool_max_pages, sink,
-                                                            tok_slot, tok_pos, (T*)out, part_o, part_ml, G, n_splits, scale, size, P, keep, (const T*)gate, gate_ld);
+  auto kernel = mods.cap > 0.f || mods.r1 != nullptr ? pool_attn_rows_kernel<T, true> : pool_attn_rows_kernel<T, false>;
+  kernel<<<grid, ROWS_WARPS * 32, 0, st>>>((const T*)q, (const T*)k_pages, (const T*)v_pages, page_table, max_pages, page_size, (const T*)pk,
+                                           (const T*)pv, pool_table, pool_max_pages, sink, tok_slot, tok_pos, (T*)out, part_o, part_ml, G,
+                                           n_splits, scale, size, P, keep, (const T*)gate, gate_ld, mods);
   int rc = launch_status();
   if (rc || n_splits == 1) return rc;
   dim3 cgrid(n, G * REP);
@@ -584,16 +626,17 @@ DRYFT_API int dryft_pool_attn_group() { return REP; }
 DRYFT_API int dryft_pool_attn_prep(int is_bf16, const void* proj, int ld, const float* qb, const float* kb, const float* vb,
                                    const float* inv_freq, const float* inv_freq_lo, int rot, const int* tok_slot, const int* tok_pos,
                                    void* q_out, void* k_pages, void* v_pages, const int* page_table, int max_pages, int page_size, int n, int H, int G, float eps,
-                                   int write_kv, const float* conv_w, int taps, void* ring, int store_ring, cudaStream_t st) {
+                                   int write_kv, const float* conv_w, int taps, void* ring, int store_ring, float v_eps, float qt_coef,
+                                   int qt_every, cudaStream_t st) {
   if (n <= 0) return 0;
   if (H != G * REP || rot < 0 || rot % 2 || rot > D || (rot > 0 && inv_freq == nullptr) || (write_kv && page_size < 1))
     return DRYFT_ERR_UNSUPPORTED;
   if (conv_w != nullptr && (taps < 1 || taps > DRYFT_CONV_MAX_TAPS || !write_kv || ((taps > 1 || store_ring) && ring == nullptr)))
     return DRYFT_ERR_UNSUPPORTED;
   return is_bf16 ? prep_launch<__nv_bfloat16>(proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, q_out, k_pages, v_pages, page_table,
-                                              max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, st)
+                                              max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, v_eps, qt_coef, qt_every, st)
                  : prep_launch<float>(proj, ld, qb, kb, vb, inv_freq, inv_freq_lo, rot, tok_slot, tok_pos, q_out, k_pages, v_pages, page_table,
-                                      max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, st);
+                                      max_pages, page_size, n, H, G, eps, write_kv, conv_w, taps, ring, store_ring, v_eps, qt_coef, qt_every, st);
 }
 
 DRYFT_API int dryft_pool_attn_prep_run(int is_bf16, const void* proj, int ld, const float* inv_freq, const float* inv_freq_lo, int rot,
@@ -651,13 +694,15 @@ DRYFT_API int dryft_pool_attn_rows(int is_bf16, const void* q, const void* k_pag
                                    int max_pages, int page_size, const void* pk, const void* pv, const int* pool_table,
                                    int pool_max_pages, const float* sink, const int* tok_slot, const int* tok_pos, void* out,
                                    float* part_o, float* part_ml, int n, int G, int n_splits, float scale, int size, int P, int keep,
-                                   const void* gate, int gate_ld, cudaStream_t st) {
+                                   const void* gate, int gate_ld, float softcap, const float* r1, const float* r2, cudaStream_t st) {
   if (n <= 0) return 0;
+  if (!(softcap >= 0.f) || (r1 != nullptr) != (r2 != nullptr) || ((softcap > 0.f || r1 != nullptr) && P > 0)) return DRYFT_ERR_UNSUPPORTED;
+  const ScoreMods mods{softcap, r1, r2};
   if (G < 1 || G > 65535 || n_splits < 1 || n_splits > 65535 || size < 1 || keep < 0 || page_size < 1 || (P > 0 && pk == nullptr) ||
       (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return DRYFT_ERR_UNSUPPORTED;
   return is_bf16 ? rows_launch<__nv_bfloat16>(q, k_pages, v_pages, page_table, max_pages, page_size, pk, pv, pool_table, pool_max_pages,
-                                              sink, tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, gate, gate_ld, st)
+                                              sink, tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, gate, gate_ld, mods, st)
                  : rows_launch<float>(q, k_pages, v_pages, page_table, max_pages, page_size, pk, pv, pool_table, pool_max_pages, sink,
-                                      tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, gate, gate_ld, st);
+                                      tok_slot, tok_pos, out, part_o, part_ml, n, G, n_splits, scale, size, P, keep, gate, gate_ld, mods, st);
 }

@@ -16,6 +16,10 @@
 // (P = 0: no blocks).  The softmax's denominator also holds exp(sink_head): the running maximum starts at the sink and
 // the running sum at one (no sink: -inf and zero).
 //
+// MODS: a score is squashed to cap * tanh(s / cap) (cap > 0) and r1_h * ln(1 + r2_h * (p - j)) is taken off (r1 given), both in
+// 32-bit before the softmax; not together with pooled rows.  The logarithms of a (query tile, key tile) pair depend on the
+// distance only, so the block's threads make the 128 there can be once and every score reads its own from shared memory.
+//
 // No block waits on another block; the only waits are cp.async.wait_group and __syncthreads.
 #include "common.cuh"
 #include <math.h>
@@ -69,7 +73,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   return *reinterpret_cast<unsigned*>(&v);
 }
 
-constexpr size_t smem_bytes() { return sizeof(bf16) * ((size_t)KS * (BM + 2 * BN) + (size_t)VS * 2 * BN); }
+template <bool MODS> constexpr size_t smem_bytes() { return (MODS ? sizeof(float) * 2 * (BM + BN) : 0) + sizeof(bf16) * ((size_t)KS * (BM + 2 * BN) + (size_t)VS * 2 * BN); }
 
 // rows of V whose key position is >= v_end are zero-filled
 __device__ __forceinline__ void load_page(bf16* ks, bf16* vs, const bf16* kp, const bf16* vp, int tid, int key0, int v_end) {
@@ -84,6 +88,10 @@ __device__ __forceinline__ void load_page(bf16* ks, bf16* vs, const bf16* kp, co
   }
 }
 
+// exp2 / reciprocal / log2 of the hardware (errors of 2 ulp, 1 ulp and 2^-22)
+__device__ __forceinline__ float ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
+
+template <bool MODS>
 __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     const bf16* __restrict__ q,                                          // [N, nH, DQ]
     const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,  // [pages, nKV, BN, DQ], [pages, nKV, BN, DV]
@@ -95,11 +103,13 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
     bf16* __restrict__ out,                                              // [N, nH * DV]
     int nH, int nKV, float scale_log2, int size, int P, int keep,
-    const bf16* __restrict__ gate, int gate_ld) {                        // gate logits [N, nH * DV] of row stride gate_ld, or null
+    const bf16* __restrict__ gate, int gate_ld,                          // gate logits [N, nH * DV] of row stride gate_ld, or null
+    float cap, const float* __restrict__ bias_r1, const float* __restrict__ bias_r2) {   // MODS
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);   // [BM][KS]
   bf16* ks = qs + BM * KS;                        // [2][BN][KS]
   bf16* vs = ks + 2 * BN * KS;                    // [2][BN][VS]
+  float* dl = reinterpret_cast<float*>(vs + 2 * BN * VS);   // MODS: [2][BM + BN] logarithms of a key tile's distances
 
   // heads run fastest: the host lists the tiles with the most keys first
   const int tile = blockIdx.x / nH, h = blockIdx.x % nH, kvh = h / G;
@@ -146,8 +156,18 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     }
   };
 
+  // MODS, in log2 units: entry i of a key tile's table belongs to the distance pos0 - key0 + i - (BN - 1)
+  const float r1h = MODS && bias_r1 != nullptr ? bias_r1[h] : 0.f, r2h = MODS && bias_r1 != nullptr ? bias_r2[h] : 0.f;
+  const float cap2 = cap * 1.4426950408889634f;          // the cap in log2 units, and what turns a dot product into 2 s / cap
+  const float to_arg = MODS && cap > 0.f ? 2.f * scale_log2 / cap : 0.f;
+  auto fill_logs = [&](int it, int stage) {
+    const int base = pos0 - token_page(it) * BN - (BN - 1);
+    for (int i = tid; i < BM + BN; i += THREADS)
+      dl[stage * (BM + BN) + i] = r1h * __log2f(fmaf(r2h, (float)max(base + i, 0), 1.f));
+  };
   load_tile(0, 0);
   cp_async_commit();
+  if (MODS) fill_logs(0, 0);
 
   float o_acc[DT][4];
 #pragma unroll
@@ -171,6 +191,7 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     if (it + 1 < n_tiles) {
       load_tile(it + 1, stage ^ 1);
       cp_async_commit();
+      if (MODS) fill_logs(it + 1, stage ^ 1);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
@@ -205,13 +226,20 @@ __global__ void __launch_bounds__(THREADS) pool_attn_prefill_kernel(
     }
     // ---- mask, online softmax (log2 domain) ----
     float mx0 = -INFINITY, mx1 = -INFINITY;
+    // MODS: this thread's first entry of the distances' logarithms (row g, key 2t of the tile); row g + 8 lies 8 further on
+    const float* dlt = dl + stage * (BM + BN) + warp * 16 + g + (BN - 1) - 2 * t;
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int kp = key0 + j * 8 + 2 * t + (i & 1);
         const bool vis = (i < 2) ? ((kp >= vlo0 || kp < vkeep) && kp < vhi0) : ((kp >= vlo1 || kp < vkeep) && kp < vhi1);
-        const float v = vis ? s[j][i] * scale_log2 : -INFINITY;
+        float raw = s[j][i] * scale_log2;
+        if (MODS) {
+          if (cap > 0.f) raw = cap2 - __fdividef(2.f * cap2, 1.f + ex2(s[j][i] * to_arg));     // cap * tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap))
+          raw -= dlt[(i >> 1) * 8 - j * 8 - (i & 1)];
+        }
+        const float v = vis ? raw : -INFINITY;
         s[j][i] = v;
         if (i < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
       }
@@ -305,23 +333,26 @@ DRYFT_API int dryft_pool_attn_prefill(const void* q, const void* k_pages, const 
                                       int page_size, const void* pk_pages, const void* pv_pages, const int* pool_table,
                                       int pool_max_pages, const float* sink, const int* tile_tok0, const int* tile_rows,
                                       const int* tok_slot, const int* tok_pos, void* out, int n_tiles, int nH, int nKV, float scale,
-                                      int size, int P, int keep, const void* gate, int gate_ld, cudaStream_t st) {
+                                      int size, int P, int keep, const void* gate, int gate_ld, float softcap, const float* r1,
+                                      const float* r2, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
   if (nH != nKV * G || nH > 65535 || page_size != BN || size < 1 || P < 0 || keep < 0) return DRYFT_ERR_UNSUPPORTED;
   if (P > 0 && (pk_pages == nullptr || pv_pages == nullptr || pool_table == nullptr)) return DRYFT_ERR_UNSUPPORTED;
-  const size_t smem = smem_bytes();
+  const bool mods = softcap > 0.f || r1 != nullptr;
+  if (!(softcap >= 0.f) || (r1 != nullptr) != (r2 != nullptr) || (mods && P > 0)) return DRYFT_ERR_UNSUPPORTED;
+  const size_t smem = mods ? smem_bytes<true>() : smem_bytes<false>();
   if (smem > 227 * 1024) return DRYFT_ERR_UNSUPPORTED;
-  static bool attr_set = false;  // set by the first (eager) launch, outside any stream capture
-  if (smem > 48 * 1024 && !attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(pool_attn_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  auto kernel = mods ? pool_attn_prefill_kernel<true> : pool_attn_prefill_kernel<false>;
+  static bool attr_set[2] = {false, false};  // set by the first (eager) launch, outside any stream capture
+  if (smem > 48 * 1024 && !attr_set[mods]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    attr_set = true;
+    attr_set[mods] = true;
   }
   if ((long long)n_tiles * nH > 2147483647LL) return DRYFT_ERR_UNSUPPORTED;
   dim3 grid((unsigned)(n_tiles * nH));
-  pool_attn_prefill_kernel<<<grid, THREADS, smem, st>>>((const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, page_table,
-                                                       max_pages, (const bf16*)pk_pages, (const bf16*)pv_pages, pool_table,
-                                                       pool_max_pages, sink, tile_tok0, tile_rows, tok_slot, tok_pos, (bf16*)out, nH,
-                                                       nKV, scale * 1.4426950408889634f, size, P, keep, (const bf16*)gate, gate_ld);
+  kernel<<<grid, THREADS, smem, st>>>((const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, page_table, max_pages, (const bf16*)pk_pages,
+                                      (const bf16*)pv_pages, pool_table, pool_max_pages, sink, tile_tok0, tile_rows, tok_slot, tok_pos, (bf16*)out,
+                                      nH, nKV, scale * 1.4426950408889634f, size, P, keep, (const bf16*)gate, gate_ld, softcap, r1, r2);
   return launch_status();
 }

@@ -10,6 +10,9 @@
 //                 h_i[n] = T( (x32[n] - mean) / sqrt(mean((x32[n] - mean)^2) + eps) * w_i + b_i ); the row stays in shared memory
 //                 (4 * width bytes), the mean is formed before the deviations are squared.  `rows` (optional): output row r
 //                 reads stream row rows[r] (no terms then: nothing is written to the stream).
+//   stream_norm_join  y = s0 * y0[n] + s1 * y1[n] + s2 * y2[n] + sum_k wts[n, k] * yr[n * top + k] ;  x32[n] += y / sqrt(mean(y^2) + eps) * factor :
+//                 the norm on a sublayer's OUTPUT; and, when a norm weight is given, h[n] = T( norm of the new row ), the norm in
+//                 front of the sublayer that comes next, in the same launch.  The row stays in shared memory (4 * width bytes).
 //   pack_pair     out[n] = T([a32[n] | b32[n]]): two 32-bit rows side by side as one operand row of a product
 //   softcap       z <- cap * tanh(z / cap) over 32-bit logits, in place
 //
@@ -154,6 +157,92 @@ int sum_ln_launch(float* x32, const int* rows, const void* y0, float s0, const v
   return launch_status();
 }
 
+template <typename T, int VEC>
+__global__ void __launch_bounds__(THREADS) stream_norm_join_kernel(
+    float* __restrict__ x32, const T* __restrict__ y0, float s0, const T* __restrict__ y1, float s1, const T* __restrict__ y2, float s2,
+    const T* __restrict__ yr, const float* __restrict__ wts, int top, const float* __restrict__ factor, float eps,
+    const float* __restrict__ norm_w, float norm_eps, T* __restrict__ h, int width) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float scratch[33];
+  const size_t n = blockIdx.x;
+  float* x = x32 + n * width;
+  const float* wt = wts + n * top;
+  float ss = 0.f;
+  // a thread reads and writes the same entries of the row in every pass
+  if (VEC == 4) {
+    for (int c = threadIdx.x * 4; c < width; c += THREADS * 4) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      auto term = [&](const T* y, float s) {
+        const float4 t = load4<T>(y + c);
+        v.x = fmaf(s, t.x, v.x); v.y = fmaf(s, t.y, v.y); v.z = fmaf(s, t.z, v.z); v.w = fmaf(s, t.w, v.w);
+      };
+      if (y0 != nullptr) term(y0 + n * width, s0);
+      if (y1 != nullptr) term(y1 + n * width, s1);
+      if (y2 != nullptr) term(y2 + n * width, s2);
+      if (yr != nullptr) {
+#pragma unroll 4
+        for (int k = 0; k < top; ++k) term(yr + (n * top + k) * width, wt[k]);      // in the order of the choices
+      }
+      *reinterpret_cast<float4*>(row + c) = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += THREADS) {
+      float v = 0.f;
+      if (y0 != nullptr) v = fmaf(s0, to_f32<T>(y0[n * width + c]), v);
+      if (y1 != nullptr) v = fmaf(s1, to_f32<T>(y1[n * width + c]), v);
+      if (y2 != nullptr) v = fmaf(s2, to_f32<T>(y2[n * width + c]), v);
+      if (yr != nullptr)
+        for (int k = 0; k < top; ++k) v = fmaf(wt[k], to_f32<T>(yr[(n * top + k) * width + c]), v);
+      row[c] = v;
+      ss = fmaf(v, v, ss);
+    }
+  }
+  float rinv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  ss = 0.f;
+  if (VEC == 4) {
+    for (int c = threadIdx.x * 4; c < width; c += THREADS * 4) {
+      const float4 y = *reinterpret_cast<const float4*>(row + c), f = *reinterpret_cast<const float4*>(factor + c);
+      float4 v = *reinterpret_cast<const float4*>(x + c);
+      v.x = fmaf(y.x * rinv, f.x, v.x); v.y = fmaf(y.y * rinv, f.y, v.y); v.z = fmaf(y.z * rinv, f.z, v.z); v.w = fmaf(y.w * rinv, f.w, v.w);
+      *reinterpret_cast<float4*>(x + c) = v;
+      *reinterpret_cast<float4*>(row + c) = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += THREADS) {
+      const float v = fmaf(row[c] * rinv, factor[c], x[c]);
+      x[c] = v;
+      row[c] = v;
+      ss = fmaf(v, v, ss);
+    }
+  }
+  if (norm_w == nullptr) return;
+  rinv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + norm_eps);
+  if (VEC == 4) {
+    for (int c = threadIdx.x * 4; c < width; c += THREADS * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(row + c), w = *reinterpret_cast<const float4*>(norm_w + c);
+      store4<T>(h + n * width + c, make_float4(v.x * rinv * w.x, v.y * rinv * w.y, v.z * rinv * w.z, v.w * rinv * w.w));
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += THREADS) h[n * width + c] = from_f32<T>(row[c] * rinv * norm_w[c]);
+  }
+}
+
+template <typename T, int VEC>
+int norm_join_launch(float* x32, const void* y0, float s0, const void* y1, float s1, const void* y2, float s2, const void* yr, const float* wts,
+                     int top, const float* factor, float eps, const float* norm_w, float norm_eps, void* h, int n, int width, cudaStream_t st) {
+  const size_t smem = sizeof(float) * (size_t)width;
+  if (smem > 200 * 1024) return DRYFT_ERR_UNSUPPORTED;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(stream_norm_join_kernel<T, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  stream_norm_join_kernel<T, VEC><<<n, THREADS, smem, st>>>(x32, (const T*)y0, s0, (const T*)y1, s1, (const T*)y2, s2, (const T*)yr, wts, top, factor,
+                                                          eps, norm_w, norm_eps, (T*)h, width);
+  return launch_status();
+}
+
 template <typename T>
 __global__ void __launch_bounds__(THREADS) pack_pair_kernel(const float* __restrict__ a, const float* __restrict__ b,
                                                            T* __restrict__ out, int width) {
@@ -196,6 +285,20 @@ DRYFT_API int dryft_stream_sum_ln(int is_bf16, float* x32, const int* rows, cons
                : sum_ln_launch<__nv_bfloat16, 1>(x32, rows, y0, s0, y1, s1, y2, s2, w0, b0, h0, w1, b1, h1, eps, n, width, st);
   return vec ? sum_ln_launch<float, 4>(x32, rows, y0, s0, y1, s1, y2, s2, w0, b0, h0, w1, b1, h1, eps, n, width, st)
              : sum_ln_launch<float, 1>(x32, rows, y0, s0, y1, s1, y2, s2, w0, b0, h0, w1, b1, h1, eps, n, width, st);
+}
+
+DRYFT_API int dryft_stream_norm_join(int is_bf16, float* x32, const void* y0, float s0, const void* y1, float s1, const void* y2, float s2,
+                                     const void* yr, const float* wts, int top, const float* factor, float eps, const float* norm_w,
+                                     float norm_eps, void* h, int n, int width, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if (width <= 0 || factor == nullptr || (yr != nullptr && (top < 1 || wts == nullptr)) || (norm_w != nullptr && h == nullptr)) return DRYFT_ERR_UNSUPPORTED;
+  typedef __nv_bfloat16 bf;
+  const bool vec = width % 4 == 0;
+  if (is_bf16)
+    return vec ? norm_join_launch<bf, 4>(x32, y0, s0, y1, s1, y2, s2, yr, wts, top, factor, eps, norm_w, norm_eps, h, n, width, st)
+               : norm_join_launch<bf, 1>(x32, y0, s0, y1, s1, y2, s2, yr, wts, top, factor, eps, norm_w, norm_eps, h, n, width, st);
+  return vec ? norm_join_launch<float, 4>(x32, y0, s0, y1, s1, y2, s2, yr, wts, top, factor, eps, norm_w, norm_eps, h, n, width, st)
+             : norm_join_launch<float, 1>(x32, y0, s0, y1, s1, y2, s2, yr, wts, top, factor, eps, norm_w, norm_eps, h, n, width, st);
 }
 
 DRYFT_API int dryft_pack_pair(int is_bf16, const float* a, const float* b, void* out, int n, int width, cudaStream_t st) {

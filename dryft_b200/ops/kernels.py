@@ -68,10 +68,10 @@ def core() -> ctypes.CDLL:
             lib.dryft_stream_norm_add.argtypes = [_i, _p, _p, _i, _p, _f, _f, _p, _p, _i, _i, _p]
             lib.dryft_stream_norm_rows.argtypes = [_i, _i, _p, _p, _p, _f, _f, _p, _i, _i, _p]
             lib.dryft_kv_maps_store.argtypes = [_i, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _p]
-            lib.dryft_moe_route.argtypes = [_p, _p, _i, _i, _i, _i, _i, _i, _p, _p, _p]
+            lib.dryft_moe_route.argtypes = [_p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _p]
             lib.dryft_moe_rows.argtypes = [_i, _p, _i, _p, _p, _i, _i, _i, _i, _p, _i, _p, _f, _f, _f, _p]
             lib.dryft_moe_combine.argtypes = [_i, _p, _p, _i, _i, _p, _i, _p]
-            lib.dryft_moe_route_rows.argtypes = [_i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _p, _p]
+            lib.dryft_moe_route_rows.argtypes = [_i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _p]
             for name in ("dryft_step_meta", "dryft_step_advance", "dryft_tokens_from_state", "dryft_embed",
                          "dryft_rmsnorm", "dryft_residual_add", "dryft_silu_mul", "dryft_qk_norm_rope_store", "dryft_rope_table",
                          "dryft_gemm_nt_f32", "dryft_argmax_rows", "dryft_sample_rows", "dryft_gemm_small_m", "dryft_row_sumsq",
@@ -137,7 +137,7 @@ def gemm_decode_lib(k: int) -> ctypes.CDLL:
         lib = _variants.get(key)
         if lib is None:
             lib = _load(build.build_library("gemm_decode", ("gemm_decode.cu",), {"DRYFT_K": k}))
-            lib.dryft_gemm_decode.argtypes = [_p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _i, _f, _p, _i, _i, _p, _p, _p]
+            lib.dryft_gemm_decode.argtypes = [_p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _i, _f, _p, _i, _i, _p, _p, _i, _i, _ll, _p]
             lib.dryft_gemm_decode.restype = _i
             if lib.dryft_gemm_decode_k() != k:
                 raise KernelError("the compiled decode product is for another inner size")
@@ -760,33 +760,40 @@ def diff_attn_rows(q, k_pages, v_pages, page_table, tok_slot, tok_pos, out, scal
 
 
 # ----------------------------------------------------------------------------- mixture of experts
-def _route_flags(renorm: bool, score: str) -> int:
+def _route_flags(renorm: bool, score: str, group_rank: str = "max") -> int:
     if score not in ("softmax", "sigmoid"):
         raise KernelError(f"moe_route: scores are 'softmax' or 'sigmoid', got {score!r}")
-    return int(bool(renorm)) | (2 if score == "sigmoid" else 0)
+    if group_rank not in ("max", "top2"):
+        raise KernelError(f"moe_route: groups are ranked by 'max' or 'top2', got {group_rank!r}")
+    return int(bool(renorm)) | (2 if score == "sigmoid" else 0) | (4 if group_rank == "top2" else 0)
 
 
-def moe_route(logits, n_groups: int, keep: int, top: int, idx_out, w_out, renorm: bool = False, bias=None, score: str = "softmax") -> None:
+def moe_route(logits, n_groups: int, keep: int, top: int, idx_out, w_out, renorm: bool = False, bias=None, score: str = "softmax",
+              correction=None, group_rank: str = "max", renorm_eps: float = 0.0) -> None:
     """The router's choice per token from 32-bit ``logits [n, experts]`` (plus ``bias [experts]``, if given): ``idx_out [n, top]``
     int32, ``w_out [n, top]`` float32.  ``renorm``: the chosen scores divided by their sum (a softmax over the chosen logits).
-    ``score="sigmoid"``: an expert's score is the sigmoid of its own logit instead of the softmax over all of them."""
+    ``score="sigmoid"``: an expert's score is the sigmoid of its own logit instead of the softmax over all of them.
+    ``correction [experts]``: added to the scores that experts and groups are chosen by, not to the weights; ``group_rank="top2"``: a
+    group is ranked by the sum of its two largest instead of its largest; ``renorm_eps`` joins the sum that ``renorm`` divides by."""
     n, e = logits.shape
     _need(logits, "router logits", torch.float32)
     if bias is not None:
         _need(bias, "router bias", torch.float32, (e,))
+    if correction is not None:
+        _need(correction, "router correction", torch.float32, (e,))
     _need(idx_out, "idx_out", torch.int32, (n, top))
     _need(w_out, "w_out", torch.float32, (n, top))
-    _ok(core().dryft_moe_route(_ptr(logits), _ptr(bias), n, e, int(n_groups), int(keep), int(top), _route_flags(renorm, score), _ptr(idx_out), _ptr(w_out),
-                               _stream()), f"moe_route ({e} experts, {n_groups} groups, keep {keep}, top {top})")
+    _ok(core().dryft_moe_route(_ptr(logits), _ptr(bias), _ptr(correction), n, e, int(n_groups), int(keep), int(top),
+                               _route_flags(renorm, score, group_rank), float(renorm_eps), _ptr(idx_out), _ptr(w_out), _stream()), f"moe_route ({e} experts, {n_groups} groups, keep {keep}, top {top})")
 
 
 def moe_route_rows_supported(hidden: int, experts: int, groups: int, itemsize: int) -> bool:
     """Whether the one-launch router (product and choice) takes these sizes: its row and scores fit 48 KB of shared memory."""
-    return 4 * (2 * experts + groups) + (itemsize * hidden + 15) // 16 * 16 <= 48 * 1024
+    return 4 * (3 * experts + groups) + (itemsize * hidden + 15) // 16 * 16 <= 48 * 1024
 
 
 def moe_route_rows(h, w_router, n_groups: int, keep: int, top: int, idx_out, w_out, renorm: bool = False, bias=None,
-                   score: str = "softmax") -> None:
+                   score: str = "softmax", correction=None, group_rank: str = "max", renorm_eps: float = 0.0) -> None:
     """``moe_route`` of ``logits = h @ w_router.T`` (32-bit sums) in one launch, for few tokens: one block per token."""
     n, k = h.shape
     e = w_router.shape[0]
@@ -796,8 +803,10 @@ def moe_route_rows(h, w_router, n_groups: int, keep: int, top: int, idx_out, w_o
     _need(w_out, "w_out", torch.float32, (n, top))
     if bias is not None:
         _need(bias, "router bias", torch.float32, (e,))
-    _ok(core().dryft_moe_route_rows(_act(h, "h"), _ptr(h), _ptr(w_router), _ptr(bias), n, k, e, int(n_groups), int(keep), int(top), _route_flags(renorm, score),
-                                    _ptr(idx_out), _ptr(w_out), _stream()), f"moe_route_rows ({e} experts over {k})")
+    if correction is not None:
+        _need(correction, "router correction", torch.float32, (e,))
+    _ok(core().dryft_moe_route_rows(_act(h, "h"), _ptr(h), _ptr(w_router), _ptr(bias), _ptr(correction), n, k, e, int(n_groups), int(keep), int(top),
+                                    _route_flags(renorm, score, group_rank), float(renorm_eps), _ptr(idx_out), _ptr(w_out), _stream()), f"moe_route_rows ({e} experts over {k})")
 
 
 def moe_rows(a, w, idx, out, mode: str, in_w=None, limit: Optional[float] = None, alpha: float = 1.0, up_offset: float = 0.0) -> None:
@@ -1054,14 +1063,14 @@ def gemm_small_m(a, w, out, *, mode: str = "store", norm_w=None, ss_in=None, ss_
         lib = gemm_decode_lib(k)
         if xw_in is not None:
             rc = lib.dryft_gemm_decode(_ptr(xw_in), k, _ptr(w), _ptr(out), n, code, m, n, None, _ptr(ss_in), int(ss_parts),
-                                       float(eps), _ptr(ss_out), int(pdl), 1, _ptr(next_w), _ptr(xw_out), _stream())
+                                       float(eps), _ptr(ss_out), int(pdl), 1, _ptr(next_w), _ptr(xw_out), 0, 0, 0, _stream())
             if rc != UNSUPPORTED:
                 _ok(rc, f"gemm_decode (M={m}, N={n}, K={k}, mode={mode}, activations weighted ahead)")
                 return
             if norm_w is None:  # it refuses what does not fit its shared memory; with norm_w the plain form takes over
                 _ok(rc, f"gemm_decode (M={m}, N={n}, K={k}, mode={mode}, activations weighted ahead; give norm_w for the other form)")
         rc = lib.dryft_gemm_decode(_ptr(a), k, _ptr(w), _ptr(out), n, code, m, n, _ptr(norm_w), _ptr(ss_in), int(ss_parts),
-                                   float(eps), _ptr(ss_out), int(pdl), 0, _ptr(next_w), _ptr(xw_out), _stream())
+                                   float(eps), _ptr(ss_out), int(pdl), 0, _ptr(next_w), _ptr(xw_out), 0, 0, 0, _stream())
         if rc != UNSUPPORTED or xw_out is not None or ss_out is not None:
             # the general form below cannot leave xw_out, and leaves another number of blocks of sums of squares
             _ok(rc, f"gemm_decode (M={m}, N={n}, K={k}, mode={mode})")
@@ -1069,6 +1078,26 @@ def gemm_small_m(a, w, out, *, mode: str = "store", norm_w=None, ss_in=None, ss_
     _ok(core().dryft_gemm_small_m(_ptr(a), k, _ptr(w), _ptr(out), n, code, m, n, k, _ptr(norm_w), _ptr(ss_in),
                                   int(ss_parts), float(eps), _ptr(ss_out), int(pdl), _stream()),
         f"gemm_small_m (M={m}, N={n}, K={k}, mode={mode})")
+
+
+def gemm_decode_groups_supported(m: int, k: int, grp_rows: int) -> bool:
+    """Whether ``gemm_decode_groups`` takes these sizes: few rows, an inner size with a library of its own, whole tiles a group."""
+    return 0 < m <= SMALL_M_LIMIT and k > 0 and k % 256 == 0 and grp_rows > 0 and grp_rows % 16 == 0
+
+
+def gemm_decode_groups(a, w, out, grp_rows: int, pdl: bool = False) -> None:
+    """Several products in one launch, for few rows: ``a [J, M, K]`` bfloat16, ``w [N, K]``; columns ``j * grp_rows ..`` of
+    ``out [M, N]`` (float32) are ``a[j] @ w[j * grp_rows : (j + 1) * grp_rows].T``, the last group taking the rows that are left."""
+    j, m, k = a.shape
+    n = w.shape[0]
+    _need(a, "a", torch.bfloat16)
+    _need(w, "w", torch.bfloat16, (n, k))
+    _need(out, "out", torch.float32, (m, n))
+    if not gemm_decode_groups_supported(m, k, grp_rows) or n <= (j - 1) * grp_rows:
+        raise KernelError(f"gemm_decode_groups: {j} groups of {grp_rows} of {n} outputs, {m} rows over {k} inputs")
+    rc = gemm_decode_lib(k).dryft_gemm_decode(_ptr(a), k, _ptr(w), _ptr(out), n, 1, m, n, None, None, 0, 0.0, None, int(pdl), 0, None, None,
+                                              int(grp_rows), j, m * k, _stream())
+    _ok(rc, f"gemm_decode_groups ({j} x {grp_rows} outputs, M={m}, K={k})")
 
 
 STREAM_M_LIMIT = 64
@@ -1264,12 +1293,12 @@ def latent_attn_lib() -> ctypes.CDLL:
     return _single_lib("latent_attn", {
         "dryft_latent_prep": [_i, _p, _i, _i, _i, _p, _i, _i, _i, _p, _f, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _p, _i, _p],
         "dryft_latent_scratch_table": [_p, _p, _i, _p, _i, _i, _p],
-        "dryft_latent_expand_store": [_i, _p, _p, _i, _i, _p, _i, _i, _p, _p, _i, _p, _p, _p, _i, _i, _p, _p, _p, _i, _i, _i, _i, _i, _p],
-        "dryft_head_gate_rows": [_i, _p, _i, _p, _i, _p, _i, _i, _i, _p],
+        "dryft_latent_expand_store": [_i, _p, _p, _i, _i, _p, _i, _i, _p, _p, _i, _p, _p, _p, _i, _i, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p],
+        "dryft_head_gate_rows": [_i, _p, _i, _p, _i, _p, _i, _i, _i, _i, _p],
         "dryft_latent_fold_q": [_i, _p, _i, _p, _p, _i, _i, _i, _i, _p],
-        "dryft_latent_unfold_o": [_i, _p, _p, _p, _i, _p, _i, _i, _i, _i, _p],
+        "dryft_latent_unfold_o": [_i, _p, _p, _p, _i, _p, _i, _i, _i, _i, _i, _p],
         "dryft_latent_attn_rows": [_i, _p, _p, _i, _i, _p, _p, _i, _i, _p, _p, _p, _p, _i, _p, _p, _i, _i, _i, _i, _i, _f, _i, _p, _p],
-        "dryft_head_gate": [_i, _p, _p, _i, _p, _i, _i, _i, _p],
+        "dryft_head_gate": [_i, _p, _p, _i, _p, _i, _i, _i, _i, _p],
     })
 
 
@@ -1507,13 +1536,14 @@ def latent_attn_rows(q_lat, q, q_rot_off: int, k_pages, page_table, tok_slot, to
 def latent_expand_store(q, kv, v_off: int, proj, krot_off: int, inv_freq, interleaved: bool, cu_q, seq_slot, n_seqs: int, tok_slot,
                         tok_pos, table, q_out, k_pages, v_pages, dim: int, rot: int, vdim: int, inv_freq_lo=None) -> None:
     """For a step whose sequences all start at position 0: pages of the step's own (``table [slots, pages]`` is filled
-    here) receive per-head keys ``[k_plain | rotated shared part]`` and values ``[v | zeros]`` of head size ``dim + rot``;
+    here) receive per-head keys ``[k_plain | rotated shared part]`` of size ``dim + rot`` and values ``[v | zeros]`` of ``v_pages``' own width;
     ``q_out [n, H, dim + rot]`` receives the queries with their rotated part rotated.  ``q [n, H, dim + rot]``,
     ``kv [n, >= H*dim + H*vdim]`` (keys' unrotated parts at column 0, values at ``v_off``), ``proj`` holds the shared key part
     at ``krot_off``.  Two launches."""
     n, n_heads, hd = q.shape
     _need(q, "q")
-    if hd != dim + rot or vdim > hd:
+    vw = v_pages.shape[-1]
+    if hd != dim + rot or vdim > vw:
         raise KernelError(f"latent_expand_store: head size {hd} against {dim} + {rot}, values of {vdim}")
     _need(kv, "kv", q.dtype)
     _need(proj, "proj", q.dtype)
@@ -1522,7 +1552,7 @@ def latent_expand_store(q, kv, v_off: int, proj, krot_off: int, inv_freq, interl
     page = k_pages.shape[2]
     _need(q_out, "q_out", q.dtype, (n, n_heads, hd))
     _need(k_pages, "k_pages", q.dtype, (None, n_heads, page, hd))
-    _need(v_pages, "v_pages", q.dtype, tuple(k_pages.shape))
+    _need(v_pages, "v_pages", q.dtype, (k_pages.shape[0], n_heads, page, vw))
     for t, nm in ((cu_q, "cu_q"), (seq_slot, "seq_slot"), (tok_slot, "tok_slot"), (tok_pos, "tok_pos"), (table, "table")):
         _need(t, nm, torch.int32)
     if rot:
@@ -1535,11 +1565,12 @@ def latent_expand_store(q, kv, v_off: int, proj, krot_off: int, inv_freq, interl
     _ok(lib.dryft_latent_expand_store(_act(q, "q"), _ptr(q), _ptr(kv), kv.shape[1], int(v_off), _ptr(proj), proj.shape[1], int(krot_off),
                                       _ptr(inv_freq), _ptr(_freq_lo(inv_freq_lo, rot)), int(interleaved), _ptr(tok_slot), _ptr(tok_pos),
                                       _ptr(table), table.shape[1], page, _ptr(q_out), _ptr(k_pages), _ptr(v_pages), n, n_heads, dim, rot,
-                                      vdim, _stream()), "latent_expand_store")
+                                      vdim, vw, _stream()), "latent_expand_store")
 
 
-def head_gate_rows(o, gate, gate_col: int, out, n_heads: int, vdim: int) -> None:
-    """``out[n, h*V + v] = T(o[n, h*hd + v] * sigmoid(gate[n, gate_col + h]))`` for ``o [n, H*hd]`` (``gate`` None: no gate)."""
+def head_gate_rows(o, gate, gate_col: int, out, n_heads: int, vdim: int, per_value: bool = False) -> None:
+    """``out[n, h*V + v] = T(o[n, h*hd + v] * sigmoid(gate[n, gate_col + h]))`` for ``o [n, H*hd]`` (``gate`` None: no gate;
+    ``per_value``: the logit of value ``v`` is ``gate[n, gate_col + h*V + v]``)."""
     n = o.shape[0]
     hd = o.shape[1] // n_heads
     _need(o, "o", None, (n, n_heads * hd))
@@ -1547,25 +1578,26 @@ def head_gate_rows(o, gate, gate_col: int, out, n_heads: int, vdim: int) -> None
     gate_ptr, gate_ld = None, 0
     if gate is not None:
         _need(gate, "gate", out.dtype)
-        if gate.dim() != 2 or gate.shape[0] < n or gate.shape[1] < gate_col + n_heads:
+        if gate.dim() != 2 or gate.shape[0] < n or gate.shape[1] < gate_col + n_heads * (vdim if per_value else 1):
             raise KernelError("head_gate_rows: gate columns outside the gate tensor")
         gate_ptr, gate_ld = ctypes.c_void_p(gate.data_ptr() + gate_col * gate.element_size()), gate.shape[1]
-    _ok(latent_attn_lib().dryft_head_gate_rows(_act(out, "out"), _ptr(o), hd, gate_ptr, gate_ld, _ptr(out), n, n_heads, vdim, _stream()),
+    _ok(latent_attn_lib().dryft_head_gate_rows(_act(out, "out"), _ptr(o), hd, gate_ptr, gate_ld, _ptr(out), n, n_heads, vdim, int(per_value), _stream()),
         "head_gate_rows")
 
 
-def head_gate(o, gate, gate_col: int, out) -> None:
-    """``out[n, h*V + v] = T(o[h, n, v] * sigmoid(gate[n, gate_col + h]))`` (``gate`` None: no gate); ``o`` float32."""
+def head_gate(o, gate, gate_col: int, out, per_value: bool = False) -> None:
+    """``out[n, h*V + v] = T(o[h, n, v] * sigmoid(gate[n, gate_col + h]))`` (``gate`` None: no gate;
+    ``per_value``: the logit of value ``v`` is ``gate[n, gate_col + h*V + v]``); ``o`` float32."""
     n_heads, n, vdim = o.shape
     _need(o, "o", torch.float32)
     _need(out, "out", None, (n, n_heads * vdim))
     gate_ptr, gate_ld = None, 0
     if gate is not None:
         _need(gate, "gate", out.dtype)
-        if gate.dim() != 2 or gate.shape[0] < n or gate.shape[1] < gate_col + n_heads:
+        if gate.dim() != 2 or gate.shape[0] < n or gate.shape[1] < gate_col + n_heads * (vdim if per_value else 1):
             raise KernelError("head_gate: gate columns outside the gate tensor")
         gate_ptr, gate_ld = ctypes.c_void_p(gate.data_ptr() + gate_col * gate.element_size()), gate.shape[1]
-    _ok(latent_attn_lib().dryft_head_gate(_act(out, "out"), _ptr(o), gate_ptr, gate_ld, _ptr(out), n, n_heads, vdim, _stream()),
+    _ok(latent_attn_lib().dryft_head_gate(_act(out, "out"), _ptr(o), gate_ptr, gate_ld, _ptr(out), n, n_heads, vdim, int(per_value), _stream()),
         "head_gate")
 
 
@@ -1582,9 +1614,10 @@ def latent_fold_q(q, w_k, q_lat, dim: int) -> None:
         "latent_fold_q")
 
 
-def latent_unfold_o(o_lat, w_v, gate, gate_col: int, out) -> None:
+def latent_unfold_o(o_lat, w_v, gate, gate_col: int, out, per_value: bool = False) -> None:
     """``out[n, h*V:(h+1)*V] = T(sigmoid(gate[n, gate_col + h]) * (o_lat[h, n] @ w_v[h]))`` with ``w_v [H, kv_rank, V]``
-    (``gate`` None: no gate)."""
+    (``gate`` None: no gate;
+    ``per_value``: the logit of value ``v`` is ``gate[n, gate_col + h*V + v]``)."""
     n_heads, n, kv_rank = o_lat.shape
     vdim = w_v.shape[2]
     _need(o_lat, "o_lat")
@@ -1593,11 +1626,11 @@ def latent_unfold_o(o_lat, w_v, gate, gate_col: int, out) -> None:
     gate_ptr, gate_ld = None, 0
     if gate is not None:
         _need(gate, "gate", out.dtype)
-        if gate.dim() != 2 or gate.shape[0] < n or gate.shape[1] < gate_col + n_heads:
+        if gate.dim() != 2 or gate.shape[0] < n or gate.shape[1] < gate_col + n_heads * (vdim if per_value else 1):
             raise KernelError("latent_unfold_o: gate columns outside the gate tensor")
         gate_ptr, gate_ld = ctypes.c_void_p(gate.data_ptr() + gate_col * gate.element_size()), gate.shape[1]
     _ok(latent_attn_lib().dryft_latent_unfold_o(_act(out, "out"), _ptr(o_lat), _ptr(w_v), gate_ptr, gate_ld, _ptr(out), n, n_heads, kv_rank,
-                                                vdim, _stream()), "latent_unfold_o")
+                                                vdim, int(per_value), _stream()), "latent_unfold_o")
 
 
 # ----------------------------------------------------------------------------- a stream whose norm follows the sum
@@ -1764,10 +1797,10 @@ def pool_attention_lib(qk_dim: int, v_dim: int, group: int) -> ctypes.CDLL:
                                        {"DRYFT_QK_DIM": qk_dim, "DRYFT_V_DIM": v_dim, "DRYFT_GROUP": group})
             lib = _load(path)
             lib.dryft_pool_attn_prep.argtypes = [_i, _p, _i, _p, _p, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _f,
-                                                 _i, _p, _i, _p, _i, _p]
+                                                 _i, _p, _i, _p, _i, _f, _f, _i, _p]
             lib.dryft_pool_attn_blocks.argtypes = [_i, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _i, _i, _i, _p]
             lib.dryft_pool_attn_rows.argtypes = [_i, _p, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f,
-                                                 _i, _i, _i, _p, _i, _p]
+                                                 _i, _i, _i, _p, _i, _f, _p, _p, _p]
             lib.dryft_pool_attn_prep_tok.argtypes = [_i, _p, _i, _p, _p, _f, _p, _p, _i, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i,
                                                      _f, _i, _p]
             lib.dryft_pool_attn_prep_run.argtypes = [_i, _p, _i, _p, _p, _i, _p, _p, _i, _i, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _f, _p,
@@ -1799,7 +1832,7 @@ def pool_attention_prefill_lib(qk_dim: int, v_dim: int, group: int, page: int = 
                                        {"DRYFT_QK_DIM": qk_dim, "DRYFT_V_DIM": v_dim, "DRYFT_GROUP": group, "DRYFT_PAGE": page})
             lib = _load(path)
             lib.dryft_pool_attn_prefill.argtypes = [_p, _p, _p, _p, _i, _i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f,
-                                                    _i, _i, _i, _p, _i, _p]
+                                                    _i, _i, _i, _p, _i, _f, _p, _p, _p]
             lib.dryft_pool_attn_prefill.restype = _i
             if (lib.dryft_pool_attn_prefill_qk_dim(), lib.dryft_pool_attn_prefill_v_dim()) != (qk_dim, v_dim):
                 raise KernelError("pooled-window prompt attention: the library was built for another head shape")
@@ -1812,12 +1845,27 @@ def _gate_of(gate, dtype, n: int, cols: int):
     return (ctypes.c_void_p(0), 0) if gate is None else _rows_of(gate, "gate", dtype, n, cols)
 
 
+def _score_mods(softcap, dist_bias, n_heads: int, pool: int):
+    """``cap, r1, r2`` of the changes to a score: ``cap * tanh(s / cap)`` (None: not squashed), then ``r1[h] * ln(1 + r2[h] * distance)``
+    taken off (``dist_bias = (r1, r2)``, None: nothing)."""
+    if softcap is not None and not softcap > 0.0:
+        raise KernelError(f"attention scores are squashed by a positive cap, got {softcap}")
+    r1, r2 = dist_bias if dist_bias is not None else (None, None)
+    for t, nm in ((r1, "r1"), (r2, "r2")):
+        if t is not None:
+            _need(t, nm, torch.float32, (n_heads,))
+    if (softcap is not None or r1 is not None) and pool:
+        raise KernelError("squashed or biased scores do not go with pooled rows")
+    return float(softcap or 0.0), _ptr(r1), _ptr(r2)
+
+
 def pool_attn_prefill(q, k_pages, v_pages, page_table, pooled, sink, tile_tok0, tile_rows, tok_slot, tok_pos, out, n_tiles: int,
-                      scale: float, size: int, pool: int, keep: int = 0, gate=None) -> None:
+                      scale: float, size: int, pool: int, keep: int = 0, gate=None, softcap: Optional[float] = None, dist_bias=None) -> None:
     """Prompt attention (bfloat16) of ``q [n, H, D]``, tile by tile of up to 64 tokens of one sequence, over the last ``size``
     cached tokens, the sequence's first ``keep`` tokens and the pooled rows of the blocks of ``pool`` positions wholly before them (``pooled = (pk_pages, pv_pages,
     pool_table)``; ``pool = 0``: none); the softmax's denominator also holds ``exp(sink[head])`` (if given).
-    ``gate [n, H * DV]`` (a column slice is fine): logits whose sigmoids multiply the output value by value."""
+    ``gate [n, H * DV]`` (a column slice is fine): logits whose sigmoids multiply the output value by value.
+    ``softcap``, ``dist_bias``: see ``_score_mods``."""
     n, n_heads, d = q.shape
     n_kv, page = k_pages.shape[1], k_pages.shape[2]
     dv = v_pages.shape[-1]
@@ -1838,16 +1886,18 @@ def pool_attn_prefill(q, k_pages, v_pages, page_table, pooled, sink, tile_tok0, 
     _ok(lib.dryft_pool_attn_prefill(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1], page, _ptr(pk),
                                     _ptr(pv), _ptr(pt), pt.shape[1] if pt is not None else 0, _ptr(sink), _ptr(tile_tok0),
                                     _ptr(tile_rows), _ptr(tok_slot), _ptr(tok_pos), _ptr(out), int(n_tiles), n_heads, n_kv,
-                                    float(scale), int(size), int(pool), int(keep), *_gate_of(gate, q.dtype, n, n_heads * dv), _stream()),
+                                    float(scale), int(size), int(pool), int(keep), *_gate_of(gate, q.dtype, n, n_heads * dv),
+                                    *_score_mods(softcap, dist_bias, n_heads, pool), _stream()),
         f"pool_attn_prefill (window {size}, blocks of {pool})")
 
 
 def pool_attn_prep(proj, q_bias, k_bias, v_bias, inv_freq, inv_freq_lo, rot: int, tok_slot, tok_pos, q_out, k_pages, v_pages,
-                   page_table, n_heads: int, n_kv: int, eps: float, write_kv: bool, conv_w=None, ring=None, store_ring: bool = False) -> None:
+                   page_table, n_heads: int, n_kv: int, eps: float, write_kv: bool, conv_w=None, ring=None, store_ring: bool = False,
+                   v_eps: float = -1.0, q_temp: Optional[Tuple[float, int]] = None) -> None:
     """Per token of ``proj [n, H*D (+ G*D + G*DV)]``: (with ``conv_w [H*D + G*(D+DV), taps]``: a short causal convolution per
     channel, earlier steps' values from ``ring [slots, taps, channels]``; ``store_ring``: a decode step stores its own there), bias, rotation of the first ``rot`` dims (rotate-half), division by the
-    root mean square over the head (no weight; ``eps < 0``: not divided) for q and k; v plus its bias; k and v into the cache
-    pages."""
+    root mean square over the head (no weight; ``eps < 0``: not divided) for q and k; v plus its bias (``v_eps >= 0``: divided by its root mean square over the head too); k and v into the
+    cache pages.  ``q_temp = (coef, every)``: the query of position p times ``1 + coef * ln((p + 1) // every + 1)``."""
     n, ld = proj.shape
     d, dv = q_out.shape[2], v_pages.shape[-1]
     _need(proj, "proj")
@@ -1876,6 +1926,7 @@ def pool_attn_prep(proj, q_bias, k_bias, v_bias, inv_freq, inv_freq_lo, rot: int
                                  _ptr(inv_freq_lo), int(rot), _ptr(tok_slot), _ptr(tok_pos), _ptr(q_out), _ptr(k_pages), _ptr(v_pages),
                                  _ptr(page_table), page_table.shape[1], k_pages.shape[2], n, n_heads, n_kv, float(eps),
                                  int(write_kv), _ptr(conv_w), taps, _ptr(ring if taps > 1 else None), int(store_ring and taps > 1),
+                                 float(v_eps), float(q_temp[0]) if q_temp else 0.0, int(q_temp[1]) if q_temp else 0,
                                  _stream()), f"pool_attn_prep ({n_heads}/{n_kv} heads of {d})")
 
 
@@ -1957,10 +2008,10 @@ def pool_attn_blocks(k_pages, v_pages, page_table, pk_pages, pv_pages, pool_tabl
 
 
 def pool_attn_rows(q, k_pages, v_pages, page_table, pooled, sink, tok_slot, tok_pos, out, scale: float, size: int, pool: int,
-                   n_splits: int = 1, part_o=None, part_ml=None, keep: int = 0, gate=None) -> None:
+                   n_splits: int = 1, part_o=None, part_ml=None, keep: int = 0, gate=None, softcap: Optional[float] = None, dist_bias=None) -> None:
     """Row-wise attention of ``q [n, H, D]`` over the last ``size`` cached tokens, the sequence's first ``keep`` tokens and, beside them, the pooled row of every block
     of ``pool`` positions that lies wholly before them (``pooled = (pk_pages, pv_pages, pool_table)``; ``pool = 0``: none), one
-    softmax whose denominator also holds ``exp(sink[head])`` (if given).  ``out [n, H, DV]``; ``gate`` as in ``pool_attn_prefill``."""
+    softmax whose denominator also holds ``exp(sink[head])`` (if given).  ``out [n, H, DV]``; ``gate``, ``softcap`` and ``dist_bias`` as in ``pool_attn_prefill``."""
     n, n_heads, d = q.shape
     n_kv, page = k_pages.shape[1], k_pages.shape[2]
     dv = v_pages.shape[-1]
@@ -1983,7 +2034,8 @@ def pool_attn_rows(q, k_pages, v_pages, page_table, pooled, sink, tok_slot, tok_
     _ok(lib.dryft_pool_attn_rows(_act(q, "q"), _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(page_table), page_table.shape[1], page,
                                  _ptr(pk), _ptr(pv), _ptr(pt), pt.shape[1] if pt is not None else 0, _ptr(sink), _ptr(tok_slot),
                                  _ptr(tok_pos), _ptr(out), _ptr(part_o), _ptr(part_ml), n, n_kv, int(n_splits), float(scale), int(size),
-                                 int(pool), int(keep), *_gate_of(gate, q.dtype, n, n_heads * dv), _stream()), f"pool_attn_rows (window {size}, blocks of {pool})",
+                                 int(pool), int(keep), *_gate_of(gate, q.dtype, n, n_heads * dv),
+                                 *_score_mods(softcap, dist_bias, n_heads, pool), _stream()), f"pool_attn_rows (window {size}, blocks of {pool})",
         n_kernels=2 if n_splits > 1 else 1)
 
 
@@ -1992,6 +2044,7 @@ def stream_par_lib() -> ctypes.CDLL:
     return _single_lib("stream_par", {
         "dryft_stream_sum": [_i, _p, _p, _p, _f, _p, _f, _p, _f, _p, _i, _f, _p, _p, _f, _p, _i, _i, _p],
         "dryft_stream_sum_ln": [_i, _p, _p, _p, _f, _p, _f, _p, _f, _p, _p, _p, _p, _p, _p, _f, _i, _i, _p],
+        "dryft_stream_norm_join": [_i, _p, _p, _f, _p, _f, _p, _f, _p, _p, _i, _p, _f, _p, _f, _p, _i, _i, _p],
         "dryft_pack_pair": [_i, _p, _p, _p, _i, _i, _p],
         "dryft_softcap": [_p, _ll, _f, _p],
     })
@@ -2070,6 +2123,36 @@ def stream_sum_ln(x32, terms=(), *, norms=(), eps: float = 0.0, rows=None, n_row
     _ok(stream_par_lib().dryft_stream_sum_ln(int(act == torch.bfloat16), _ptr(x32), _ptr(rows), _ptr(terms[0][0]), terms[0][1], _ptr(terms[1][0]),
                                              terms[1][1], _ptr(terms[2][0]), terms[2][1], _ptr(w0), _ptr(b0), _ptr(h0), _ptr(w1), _ptr(b1), _ptr(h1),
                                              float(eps), n, width, _stream()), "stream_sum_ln")
+
+
+def stream_norm_join(x32, terms=(), *, factor, eps: float, rows=None, wts=None, norm_w=None, norm_eps: float = 0.0, h=None) -> None:
+    """``x32[n] += y / sqrt(mean(y^2) + eps) * factor`` in place with ``y = sum_i scale_i * y_i[n] + sum_k wts[n, k] * rows[n * top + k]``, all of it
+    32-bit, for up to three ``terms`` ``(y_i, scale_i)`` of the activation type and a routed feed-forward's ``rows [n * top, width]`` with
+    their ``wts [n, top]`` (float32); with ``norm_w`` also ``h[n] = T(x32[n] / sqrt(mean(x32[n]^2) + norm_eps) * norm_w)`` of the new stream."""
+    n, width = x32.shape
+    _need(x32, "x32", torch.float32)
+    _need(factor, "factor", torch.float32, (width,))
+    terms = [(y, float(sc)) for y, sc in terms if y is not None]
+    if len(terms) > 3:
+        raise KernelError("stream_norm_join: at most three terms beside the routed rows")
+    act, top = None, 0
+    for y, _ in terms:
+        _need(y, "term", act, (n, width))
+        act = y.dtype
+    if rows is not None:
+        _need(wts, "wts", torch.float32, (n, None))
+        top = wts.shape[1]
+        _need(rows, "rows", act, (n * top, width))
+        act = rows.dtype
+    if act not in (torch.float32, torch.bfloat16):
+        raise KernelError(f"stream_norm_join: what joins the stream is float32 or bfloat16, got {act}")
+    if norm_w is not None:
+        _need(norm_w, "norm_w", torch.float32, (width,))
+        _need(h, "h", act, (n, width))
+    terms += [(None, 0.0)] * (3 - len(terms))
+    _ok(stream_par_lib().dryft_stream_norm_join(int(act == torch.bfloat16), _ptr(x32), _ptr(terms[0][0]), terms[0][1], _ptr(terms[1][0]), terms[1][1],
+                                                _ptr(terms[2][0]), terms[2][1], _ptr(rows), _ptr(wts), top, _ptr(factor), float(eps), _ptr(norm_w),
+                                                float(norm_eps), _ptr(h if norm_w is not None else None), n, width, _stream()), "stream_norm_join")
 
 
 def pack_pair(a32, b32, out) -> None:
@@ -2246,3 +2329,94 @@ def delta_decode(proj, x_off: int, b_off: int, dec, gate, conv_w, ring, a_log, d
                                        gate_ld, _ptr(conv_w), taps, _ptr(ring if taps > 1 else None), _ptr(a_log), _ptr(dt_bias),
                                        _ptr(norm_w), float(eps), int(sigmoid_gate), _ptr(tok_slot), _ptr(tok_pos), n, heads, kv_heads, dim,
                                        vdim, _ptr(state), _ptr(out), _stream()), f"delta_decode ({heads}/{kv_heads} heads of {dim} x {vdim})")
+
+
+# ----------------------------------------------------------------------------- time mixing: decayed outer products (csrc/wkv.cu)
+WKV_MAX_DIM = 256
+WKV_CHUNK_TOKENS = 64     # tokens a chunk of a many-token step walks in order (more for steps of more than 8,192 tokens)
+
+
+def wkv_lib() -> ctypes.CDLL:
+    return _single_lib("wkv", {
+        "dryft_wkv_mix": [_i, _p, _p, _p, _p, _p, _i, _i, _p],
+        "dryft_wkv_tanh": [_i, _p, _p, _ll, _p],
+        "dryft_wkv_walk": [_i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _p, _p, _p, _p],
+        "dryft_wkv_norm": [_i, _p, _p, _i, _p, _f, _p, _i, _p, _p, _i, _i, _i, _p, _p],
+        "dryft_wkv_decode": [_i, _p, _p, _p, _p, _i, _p, _i, _i, _p, _p, _p, _p, _f, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _p],
+    })
+
+
+def wkv_mix(h, last, mu, tok_slot, out) -> None:
+    """``out[j, t] = T(h[t] + (h[t-1] - h[t]) * mu[j])`` for the five mixtures ``j``; the token before a sequence's first one of the
+    step is ``last[slot]``."""
+    n, width = h.shape
+    _need(h, "h")
+    _need(last, "last", h.dtype, (None, width))
+    _need(mu, "mu", torch.float32, (5, width))
+    _need(tok_slot, "tok_slot", torch.int32)
+    _need(out, "out", h.dtype, (5, n, width))
+    _ok(wkv_lib().dryft_wkv_mix(_act(h, "h"), _ptr(h), _ptr(last), _ptr(mu), _ptr(tok_slot), _ptr(out), n, width, _stream()), "wkv_mix")
+
+
+def wkv_tanh(low, out) -> None:
+    """``out = T(tanh(low))`` of 32-bit values."""
+    _need(low, "low", torch.float32)
+    _need(out, "out", None, tuple(low.shape))
+    _ok(wkv_lib().dryft_wkv_tanh(_act(out, "out"), _ptr(low), _ptr(out), low.numel(), _stream()), "wkv_tanh")
+
+
+def wkv_tokens(r, k, v, g, z, w0, u, norm_w, eps: float, h, last, ctx, state, out, chunked: bool = False) -> None:
+    """A step of several tokens a sequence: ``o_t = S^T r_t + (r_t . (u * k_t)) v_t``, ``S <- diag(w_t) S + k_t v_t^T`` with ``w = exp(-exp(z +
+    w0))``, then ``out = T(o / rms(o) * norm_w * silu(g))`` per head; ``last[slot]`` receives the step's last row of ``h``.  ``r, k [n, H*d]``,
+    ``v, g [n, H*dv]`` of the activation type (``d = dv``), ``z [n, H*d]`` float32; ``state [slots, H, d, dv]`` float32 is left advanced.
+    ``chunked``: chunks of the step run side by side (three launches in place of one)."""
+    n, width = h.shape
+    heads, d, dv = state.shape[1:]
+    for t, nm, cols in ((r, "r", heads * d), (k, "k", heads * d), (v, "v", heads * dv), (g, "g", heads * dv)):
+        _need(t, nm, h.dtype, (n, cols))
+    if d != dv:
+        raise KernelError(f"wkv: keys of {d} and values of {dv} share one row stride and must have one size")
+    _need(z, "z", torch.float32, (n, heads * d))
+    for t, nm, cnt in ((w0, "w0", heads * d), (u, "u", heads * d), (norm_w, "norm_w", heads * dv)):
+        _need(t, nm, torch.float32, (cnt,))
+    _need(state, "state", torch.float32)
+    _need(last, "last", h.dtype, (None, width))
+    _need(out, "out", h.dtype, (n, heads * dv))
+    dev = h.device
+    o = torch.empty((n, heads * dv), dtype=torch.float32, device=dev)
+    cht = n_chunks = 0
+    cstate = cdecay = None
+    if chunked:
+        cht = max(WKV_CHUNK_TOKENS, -(-n // 128 // 32) * 32)
+        n_chunks = n // cht + int(ctx.n_seqs)
+        cstate = torch.empty((n_chunks, heads, d, dv), dtype=torch.float32, device=dev)
+        cdecay = torch.empty((n_chunks, heads, d), dtype=torch.float32, device=dev)
+    what = f"({heads} heads of {d})"
+    _ok(wkv_lib().dryft_wkv_walk(_act(h, "h"), _ptr(r), _ptr(k), _ptr(v), heads * d, _ptr(z), _ptr(w0), _ptr(u), _ptr(ctx.cu_q), _ptr(ctx.seq_slot),
+                                 int(ctx.n_seqs), cht, n_chunks, heads, d, dv, _ptr(state), _ptr(cstate), _ptr(cdecay), _ptr(o), _stream()),
+        "wkv_walk " + what, n_kernels=3 if chunked else 1)
+    _ok(wkv_lib().dryft_wkv_norm(_act(h, "h"), _ptr(o), _ptr(g), heads * dv, _ptr(norm_w), float(eps), _ptr(h), width, _ptr(last), _ptr(ctx.tok_slot),
+                                 n, heads, dv, _ptr(out), _stream()), "wkv_norm " + what)
+
+
+def wkv_decode(r, k, v, g, low, w2, w0, u, norm_w, eps: float, h, last, tok_slot, state, out) -> None:
+    """``wkv_tokens`` for one token a sequence in one launch behind the products, the decay's second product (``tanh(low) @ w2.T``) inside:
+    ``r, k, v, g`` and ``low [n, R]`` are float32 column ranges (row slices of one tensor are fine; the first four share a row stride)."""
+    n, width = h.shape
+    heads, d, dv = state.shape[1:]
+    ptrs, lds = zip(*[_rows_of(t, nm, torch.float32, n, cols) for t, nm, cols in
+                      ((r, "r", heads * d), (k, "k", heads * d), (v, "v", heads * dv), (g, "g", heads * dv), (low, "low", low.shape[1]))])
+    if len(set(lds[:4])) != 1:
+        raise KernelError("wkv_decode: r, k, v and g have different row strides")
+    rank = low.shape[1]
+    _need(w2, "w2", h.dtype, (heads * d, rank))
+    for t, nm, cnt in ((w0, "w0", heads * d), (u, "u", heads * d), (norm_w, "norm_w", heads * dv)):
+        _need(t, nm, torch.float32, (cnt,))
+    _need(h, "h")
+    _need(last, "last", h.dtype, (None, width))
+    _need(state, "state", torch.float32)
+    _need(out, "out", h.dtype, (n, heads * dv))
+    _need(tok_slot, "tok_slot", torch.int32)
+    _ok(wkv_lib().dryft_wkv_decode(_act(h, "h"), *ptrs[:4], lds[0], ptrs[4], lds[4], rank, _ptr(w2), _ptr(w0), _ptr(u), _ptr(norm_w), float(eps),
+                                   _ptr(h), width, _ptr(last), _ptr(tok_slot), n, heads, d, dv, _ptr(state), _ptr(out), _stream()),
+        f"wkv_decode ({heads} heads of {d})")

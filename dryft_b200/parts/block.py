@@ -358,6 +358,67 @@ class ParallelNormsBlock:
                         hn2=outs[1], hn2_norm=next_norms[1] if outs[1] is not None else None)
 
 
+@register_block("sandwich")
+class SandwichBlock:
+    """A norm in front of and behind each sublayer, around a 32-bit stream:
+
+        x <- x + norm_out(mixer(norm_mixer(x))) ;   x <- x + norm_ffn_out(ffn(norm_ffn(x)))
+
+    ``extra`` holds the two norms behind the sublayers (``mixer_out``, ``ffn_out``).  All four must offer ``plain_params``
+    (``rmsnorm_offset`` does).  The norm of a sublayer's output, its addition and the norm in front of whatever reads the stream
+    next are one kernel (``csrc/stream_par.cu:stream_norm_join``), which also forms what the output is made of: a mixer that offers
+    ``forward_terms`` hands over its results unsummed with their factors, a routed feed-forward its ``top`` rows per token with
+    their weights (``forward_parts``) and its always-on expert's row (``forward_shared``).  In a step of few rows the always-on
+    expert runs beside the routed ones on a stream of its own.  A layer without a feed-forward stops after the mixer."""
+
+    takes_next_norm = True
+
+    def __init__(self, norm_mixer, mixer, norm_ffn, ffn, extra: Optional[Mapping] = None):
+        self.extra = dict(extra or {})
+        self.norm_mixer, self.mixer, self.norm_ffn, self.ffn = norm_mixer, mixer, norm_ffn, ffn
+        self.mixer_out, self.ffn_out = self.extra.get("mixer_out"), self.extra.get("ffn_out")
+        for nm in (norm_mixer, self.mixer_out) + ((norm_ffn, self.ffn_out) if ffn is not None else ()):
+            if nm is None or not hasattr(nm, "plain_params"):
+                raise ValueError("the 'sandwich' arrangement needs a norm in front of and behind each sublayer (extra parts mixer_out, "
+                                 "ffn_out), all of them offering plain_params")
+        K.stream_par_lib()
+
+    def _join(self, x, terms, norm_out, next_norm, rows=None, wts=None):
+        """The stream plus the norm of the sum, in place; the new stream normed for ``next_norm`` (None: not known)."""
+        factor, eps = norm_out.plain_params()
+        plain = ParallelBlock._plain(next_norm) if next_norm is not None else None
+        if plain is None:
+            K.stream_norm_join(x, terms, factor=factor, eps=eps, rows=rows, wts=wts)
+            return None
+        hn = torch.empty(x.shape, dtype=self.mixer.rt.dtype, device=x.device)
+        K.stream_norm_join(x, terms, factor=factor, eps=eps, rows=rows, wts=wts, norm_w=plain[0], norm_eps=plain[1], h=hn)
+        return hn
+
+    def forward(self, res: Residual, ctx: StepContext, cache, state, owns_cache: bool = True, next_norm=None) -> Residual:
+        x, rt = res.x, self.mixer.rt
+        if x.dtype != torch.float32:
+            raise ValueError("the 'sandwich' arrangement keeps its stream in float32; the embedding must start one")
+        if res.delta is not None:
+            x.add_(res.delta)
+        n = res.hn if (res.hn is not None and res.hn_norm is self.norm_mixer) else self.norm_mixer.forward(x)
+        terms = getattr(self.mixer, "forward_terms", None)
+        terms = terms(n, ctx, cache, state, owns_cache) if terms is not None else [(self.mixer.forward(n, ctx, cache, state, owns_cache), 1.0)]
+        if self.ffn is None:
+            hn = self._join(x, terms, self.mixer_out, next_norm)
+            return Residual(x, hn=hn, hn_norm=next_norm if hn is not None else None)
+        n = self._join(x, terms, self.mixer_out, self.norm_ffn)
+        parts = getattr(self.ffn, "forward_parts", None)
+        if parts is None:
+            hn = self._join(x, [(self.ffn.forward(n, ctx), 1.0)], self.ffn_out, next_norm)
+        else:
+            jobs = [lambda: parts(n, ctx), lambda: self.ffn.forward_shared(n) if hasattr(self.ffn, "forward_shared") else None]
+            (y, wts, _), shared = rt.run_branches(jobs, first_stream=0) if rt.branches(x.shape[0]) else [j() for j in jobs]
+            if shared is not None and shared[1] is not None:
+                raise ValueError("the 'sandwich' arrangement adds the always-on expert as it is: it has no gate here")
+            hn = self._join(x, [(shared[0], 1.0)] if shared is not None else [], self.ffn_out, next_norm, rows=y, wts=wts)
+        return Residual(x, hn=hn, hn_norm=next_norm if hn is not None else None)
+
+
 @register_connection("loop_mix")
 class LoopMix:
     """How a stretch of layers that runs several times is entered: ``x <- W [x | x0] + step[t]`` with ``x0`` the embedding's

@@ -173,3 +173,45 @@ class PolyNormMLP:
         for r0 in range(0, n, chunk):
             out[r0:r0 + chunk] = self._rows(h[r0:r0 + chunk])
         return out
+
+
+@register_ffn("relu2_mlp")
+class Relu2MLP:
+    """``down(max(up(h), 0)^2)`` without a gate branch.  ``params["names"]`` maps ``up``, ``down`` to the tensors' names behind the
+    prefix."""
+
+    @staticmethod
+    def _names(params: Mapping, prefix: str) -> Dict[str, str]:
+        given = params.get("names") or {}
+        return {r: prefix + given.get(r, r + "_proj.weight") for r in ("up", "down")}
+
+    @staticmethod
+    def tensors(params: Mapping, prefix: str) -> Dict[str, TensorInfo]:
+        h, i = params["hidden_size"], params["intermediate_size"]
+        nm = Relu2MLP._names(params, prefix)
+        return {nm["up"]: TensorInfo((i, h), "matrix"), nm["down"]: TensorInfo((h, i), "matrix")}
+
+    def __init__(self, params: Mapping, prefix: str, weights, rt: Runtime):
+        self.rt = rt
+        self.hidden = int(params["hidden_size"])
+        self.inter = int(params["intermediate_size"])
+        nm = self._names(params, prefix)
+        self.w_up = weights.load(nm["up"], "matrix")
+        self.w_down = weights.load(nm["down"], "matrix")
+        K.rowops_lib()
+
+    def _rows(self, h: torch.Tensor) -> torch.Tensor:
+        z = linear(h, self.w_up, self.rt)
+        act = torch.empty_like(z)
+        K.relu2(z, act)
+        return linear(act, self.w_down, self.rt)
+
+    def forward(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        n = h.shape[0]
+        chunk = self.rt.ffn_chunk_rows
+        if n <= chunk:
+            return self._rows(h)
+        out = torch.empty((n, self.hidden), dtype=h.dtype, device=h.device)
+        for r0 in range(0, n, chunk):
+            out[r0:r0 + chunk] = self._rows(h[r0:r0 + chunk])
+        return out

@@ -7,6 +7,7 @@ With ``H`` heads, per head ``d`` unrotated and ``r`` rotated query/key dims, val
     [c_raw | k_rot] = W_dkv h ;  c = rmsnorm(c_raw) ;  k_rot rotated at the token's position, one vector for all heads
     per head:  k = W_uk c ,  v = W_uv c ;  score(i, j) = (q_plain . k + q_rot . k_rot) * scale ,  0 <= i - j < window
     o = softmax(score) v ;  o <- o * sigmoid(W_g h)_head  ->  @ W_o.T
+    (``gate="value"``: a gate per value, ``W_g [H * dv, hidden]``: o <- o * sigmoid(W_g h) element by element; ``gate`` False: none)
     (``sink``: the softmax's denominator of head ``h`` also holds ``exp(sink_h)``, a learned number without key or value)
 
 Only ``[c | k_rot]`` is cached, one row per token for all heads (a keys-only cache group).  The per-head key and value
@@ -53,7 +54,7 @@ class LatentAttention:
              nm["dkv_norm"]: TensorInfo((kr,), "vector"), nm["uk"]: TensorInfo((h * d, kr), "matrix"),
              nm["uv"]: TensorInfo((h * dv, kr), "matrix"), nm["o"]: TensorInfo((w, h * dv), "matrix")}
         if params.get("gate", True):
-            t[nm["gate"]] = TensorInfo((h, w), "matrix")
+            t[nm["gate"]] = TensorInfo((h * dv if params.get("gate") == "value" else h, w), "matrix")
         if params.get("sink", False):
             t[nm["sink"]] = TensorInfo((h,), "vector", False, 0.0)
         return t
@@ -71,6 +72,7 @@ class LatentAttention:
         self.eps = float(params["eps"])
         self.window: Optional[int] = params.get("window")
         self.has_gate = bool(params.get("gate", True))
+        self.value_gate = params.get("gate", True) == "value"
         if self.kv_rank > 512:
             raise ValueError(f"latent_attention: latents of up to 512 are served, got kv_rank={self.kv_rank}")
         pos: PartSpec = params.get("position") or PartSpec("none")
@@ -81,7 +83,7 @@ class LatentAttention:
         names, rows = [nm["dq"], nm["dkv"]], [self.q_rank, self.kv_rank + self.rot_dim]
         if self.has_gate:
             names.append(nm["gate"])
-            rows.append(self.n_heads)
+            rows.append(self.n_heads * self.v_dim if self.value_gate else self.n_heads)
         self.w_in = weights.load_fused(names, rows, self.hidden)    # one product for everything that reads the mixer's input
         self.dkv_off = self.q_rank
         self.gate_col = self.q_rank + self.kv_rank + self.rot_dim
@@ -100,15 +102,20 @@ class LatentAttention:
         # prompts whose sequences all start at position 0 (bfloat16): keys and values per head from the step's own latents
         # (one product), then the library's tensor-core prompt attention over pages of the step's own
         hd = d + self.rot_dim
-        self.use_prompt_tc = rt.is_bf16 and hd % 16 == 0 and hd <= 256 and dv <= hd and rt.page_size == 64
+        self.use_prompt_tc = rt.is_bf16 and hd % 16 == 0 and hd <= 256 and (dv <= hd or self.value_gate) and rt.page_size == 64
         self.uses_fresh_steps = self.use_prompt_tc
-        if self.use_prompt_tc and self.sink is not None:
+        # a gate per value is applied inside the prompt kernel that knows one, whose values have a size of their own
+        self.prompt_vw = hd
+        if self.use_prompt_tc and self.value_gate:
+            self.prompt_vw = self.v_dim
+            self.use_prompt_tc = self.uses_fresh_steps = K.pool_attention_prefill_supported(hd, self.v_dim, 1, rt.page_size)
+        elif self.use_prompt_tc and self.sink is not None:
             # with a sink the prompt kernel is the one that opens its softmax with it (values padded to the key size)
             self.use_prompt_tc = self.uses_fresh_steps = K.pool_attention_prefill_supported(hd, hd, 1, rt.page_size)
         if self.use_prompt_tc:
             self.w_ukv = torch.cat([w_uk, w_uv], dim=0).contiguous()      # [H*d + H*dv, kr]
-            if self.sink is not None:
-                K.pool_attention_prefill_lib(hd, hd, 1, rt.page_size)
+            if self.sink is not None or self.value_gate:
+                K.pool_attention_prefill_lib(hd, self.prompt_vw, 1, rt.page_size)
             else:
                 K.attention_prefill_lib(hd, 1, rt.page_size)
 
@@ -136,11 +143,16 @@ class LatentAttention:
             kv = linear(c_rows, self.w_ukv, self.rt)                      # [n, H*d | H*dv]
             n_pages = n // page + ctx.n_seqs + 1
             k_s = torch.zeros((n_pages, H, page, hd), dtype=h.dtype, device=dev)
-            v_s = torch.zeros((n_pages, H, page, hd), dtype=h.dtype, device=dev)
+            v_s = torch.zeros((n_pages, H, page, self.prompt_vw), dtype=h.dtype, device=dev)
             table = torch.zeros((cache.page_table.shape[0], (n + page - 1) // page + 1), dtype=torch.int32, device=dev)
             q_full = torch.empty((n, H, hd), dtype=h.dtype, device=dev)
             K.latent_expand_store(q, kv, H * d, proj, self.dkv_off + kr, self.position.inv_freq, self.position.interleaved, ctx.cu_q,
                                   ctx.seq_slot, ctx.n_seqs, ctx.tok_slot, ctx.tok_pos, table, q_full, k_s, v_s, d, r, dv, inv_freq_lo=lo)
+            if self.value_gate:
+                out = torch.empty((n, H, dv), dtype=h.dtype, device=dev)
+                K.pool_attn_prefill(q_full, k_s, v_s, table, None, self.sink, ctx.tile_tok0, ctx.tile_rows, ctx.tok_slot, ctx.tok_pos, out,
+                                    ctx.n_tiles, self.scale, self.window or (1 << 30), 0, gate=proj[:, self.gate_col:])
+                return linear(out.view(n, H * dv), self.w_o, self.rt)
             o_pad = torch.empty((n, H * hd), dtype=h.dtype, device=dev)
             if self.sink is not None:
                 K.pool_attn_prefill(q_full, k_s, v_s, table, None, self.sink, ctx.tile_tok0, ctx.tile_rows, ctx.tok_slot, ctx.tok_pos,
@@ -166,9 +178,10 @@ class LatentAttention:
                            inv_freq_lo=lo, n_splits=self._n_splits(n, ctx.max_kv), sink=self.sink)
         out = torch.empty((n, H * dv), dtype=h.dtype, device=dev)
         if own:
-            K.latent_unfold_o(o_lat, self.w_uv_t, proj if self.has_gate else None, self.gate_col, out)
+            K.latent_unfold_o(o_lat, self.w_uv_t, proj if self.has_gate else None, self.gate_col, out, per_value=self.value_gate)
         else:
-            K.head_gate(torch.bmm(o_lat, self.w_uv_t, out_dtype=torch.float32), proj if self.has_gate else None, self.gate_col, out)
+            K.head_gate(torch.bmm(o_lat, self.w_uv_t, out_dtype=torch.float32), proj if self.has_gate else None, self.gate_col, out,
+                        per_value=self.value_gate)
         return linear(out, self.w_o, self.rt)
 
     HEADS_PER_BLOCK, KEYS_PER_TILE = 16, 32     # csrc/latent_attn.cu

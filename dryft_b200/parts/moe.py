@@ -3,7 +3,7 @@
 ``E`` small experts without biases -- SwiGLU (``down(silu(gate(h)) * up(h))``) or, with ``activation="relu2"``, ungated
 (``down(max(up(h), 0)^2)``) -- of which a token uses ``top``.  The router may have a bias on its logits (``router_bias``: a
 tensor name), and ``renormalize`` divides the chosen scores by their sum, which is the softmax over the chosen logits only.
-An always-on expert of the same form (``shared``: ``{"intermediate_size", "gate"}``) may run for every token beside them; its
+An always-on expert of the same form, gated or not (``shared``: ``{"intermediate_size", "gate"}``) may run for every token beside them; its
 output is weighted by ``sigmoid(w_gate . h)``, one number per token, when it has a gate.  Router:
 ``z = W_router h`` and ``s = softmax(z)`` over all experts in 32-bit; expert ``e`` belongs to group ``e // (E / groups)`` (contiguous and equally
 sized), a group is ranked by the maximum of its members' scores, and selection is restricted to the ``keep`` highest-ranked
@@ -22,6 +22,10 @@ chosen expert's weight multiplies its INPUT, ``out = sum_k expert_k(w_k h)``, no
 linear, the weight is applied to their 32-bit sums, before the activation.  ``activation="clamped"`` (with ``limit``,
 ``alpha``, ``up_offset``): ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, ``down(g * sigmoid(alpha g) * (u +
 up_offset))``.
+
+``correction``: a vector (tensor role ``correction``) added to the scores that experts and groups are chosen by; the weights stay the
+scores themselves.  ``group_rank="top2"``: a group is ranked by the sum of its two largest choice scores.  ``renorm_eps`` joins
+the sum that ``renormalize`` divides by.
 """
 
 from __future__ import annotations
@@ -35,7 +39,7 @@ from .base import Runtime, StepContext, TensorInfo, register_ffn
 from .linear import linear
 
 _ROLES = {"router": "router.weight", "router_bias": "router.bias", "expert": "experts.{}.", "gate": "gate_proj.weight",
-          "up": "up_proj.weight", "down": "down_proj.weight", "shared": "shared.", "shared_gate": "shared.gate.weight"}
+          "up": "up_proj.weight", "down": "down_proj.weight", "shared": "shared.", "shared_gate": "shared.gate.weight", "correction": "router.correction"}
 SHARED_PAD = 8   # the always-on expert's first product carries its gate logit as one more column, padded to this many
 
 
@@ -54,6 +58,8 @@ class MoE:
         t = {prefix + nm["router"]: TensorInfo((e, w), "matrix")}
         if params.get("router_bias"):
             t[prefix + nm["router_bias"]] = TensorInfo((e,), "vector", False, 0.0)
+        if params.get("correction"):
+            t[prefix + nm["correction"]] = TensorInfo((e,), "vector", False, 0.0)
         for i in range(e):
             ep = prefix + nm["expert"].format(i)
             if gated:
@@ -80,6 +86,10 @@ class MoE:
         self.groups = int(params.get("groups", 1))
         self.keep = int(params.get("keep", self.groups))
         self.renorm = bool(params.get("renormalize", False))
+        self.renorm_eps = float(params.get("renorm_eps", 0.0))
+        self.group_rank = params.get("group_rank", "max")
+        if self.group_rank not in ("max", "top2"):
+            raise ValueError(f"moe: group_rank must be 'max' or 'top2', got {self.group_rank!r}")
         if self.experts % self.groups or not 1 <= self.keep <= self.groups or not 1 <= self.top <= self.experts:
             raise ValueError(f"moe: {self.experts} experts, {self.groups} groups, keep {self.keep}, top {self.top} do not go together")
         act = params.get("activation", "swiglu")
@@ -107,6 +117,7 @@ class MoE:
         # accumulation and a 32-bit result; in the 32-bit path everything is float32.
         self.w_router = weights.load(prefix + nm["router"], "matrix")
         self.router_bias = weights.load(prefix + nm["router_bias"], "vector") if params.get("router_bias") else None
+        self.correction = weights.load(prefix + nm["correction"], "vector") if params.get("correction") else None
         gu, dn = [], []
         for i in range(self.experts):
             ep = prefix + nm["expert"].format(i)
@@ -125,17 +136,18 @@ class MoE:
         self.side, self.side_out = None, None      # (first column, columns) of rows that ride with the always-on expert's product
         sh = params.get("shared")
         if sh is not None:
-            if self.gated:
-                raise ValueError("moe: an always-on expert is served for ungated experts (activation 'relu2') only")
+            if self.clamped:
+                raise ValueError("moe: an always-on expert is served for the activations 'swiglu' and 'relu2'")
             self.shared_inter = fs = int(sh["intermediate_size"])
             self.shared_gate = bool(sh.get("gate", True))
             sp = prefix + nm["shared"]
-            names, rows = [sp + nm["up"]], [fs]
+            names, rows = ([sp + nm["gate"], sp + nm["up"]], [fs, fs]) if self.gated else ([sp + nm["up"]], [fs])
+            self.shared_cols = sum(rows)       # gate | up (or up alone); its gate logit is the column behind them
             if self.shared_gate:
                 names.append(prefix + nm["shared_gate"])
                 rows.append(1)
             w = weights.load_fused(names, rows, self.hidden)
-            pad = (-w.shape[0]) % SHARED_PAD
+            pad = (-w.shape[0]) % SHARED_PAD if self.shared_gate or not self.gated else 0
             self.w_shared_up = torch.cat([w, torch.zeros((pad, self.hidden), dtype=w.dtype, device=w.device)]) if pad else w
             self.w_shared_down = weights.load(sp + nm["down"], "matrix")
 
@@ -152,10 +164,12 @@ class MoE:
         if (n <= self.ROUTE_ROWS_MAX and self.w_router.dtype == h.dtype and self.w_router.numel() <= self.ROUTE_ROWS_MAX_WEIGHTS
                 and K.moe_route_rows_supported(self.hidden, self.experts, self.groups, h.element_size())):
             K.moe_route_rows(h, self.w_router, self.groups, self.keep, self.top, idx, wts, renorm=self.renorm,
-                             bias=self.router_bias, score=self.score)   # one launch
+                             bias=self.router_bias, score=self.score, correction=self.correction, group_rank=self.group_rank,
+                             renorm_eps=self.renorm_eps)   # one launch
             return idx, wts
         logits = linear(h, self.w_router, self.rt, out_dtype=torch.float32)
-        K.moe_route(logits, self.groups, self.keep, self.top, idx, wts, renorm=self.renorm, bias=self.router_bias, score=self.score)
+        K.moe_route(logits, self.groups, self.keep, self.top, idx, wts, renorm=self.renorm, bias=self.router_bias, score=self.score,
+                    correction=self.correction, group_rank=self.group_rank, renorm_eps=self.renorm_eps)
         return idx, wts
 
     def absorb_rows(self, w: torch.Tensor) -> bool:
@@ -178,9 +192,12 @@ class MoE:
         if self.side is not None:
             self.side_out = z[:, self.side[0]:self.side[0] + self.side[1]]
         act = torch.empty((h.shape[0], self.shared_inter), dtype=h.dtype, device=h.device)
-        K.relu2(z[:, :self.shared_inter], act)
+        if self.gated:
+            K.glu_clamp(z if z.shape[1] == self.shared_cols else z[:, :self.shared_cols].contiguous(), act, None, 1.0, 0.0)
+        else:
+            K.relu2(z[:, :self.shared_inter], act)
         ys = linear(act, self.w_shared_down, self.rt)
-        return ys, (z[:, self.shared_inter:self.shared_inter + 1] if self.shared_gate else None)
+        return ys, (z[:, self.shared_cols:self.shared_cols + 1] if self.shared_gate else None)
 
     def forward_parts(self, h: torch.Tensor, ctx: StepContext) -> Tuple[torch.Tensor, torch.Tensor, int]:
         """``(y [n*top, hidden], wts [n, top], top)``: row ``n*top + k`` is the output of token ``n``'s k-th expert, not yet

@@ -26,6 +26,11 @@ per-sequence state.  ``value_gate``: the concatenated heads are multiplied eleme
 and ``k_norm [kv_heads * qk_dim]``, ``eps`` inside the root) before the rotation.  The rotation's layout is the position
 part's (``half``: dims ``i`` and ``i + R/2``; ``interleaved``: dims ``2i`` and ``2i + 1``).
 
+``value_norm``: each head's value is divided by its root mean square over ``v_dim`` and cached so.  ``q_temp`` (``coef``, ``every``): the
+query of position p is multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``softcap``: a scaled score becomes ``cap *
+tanh(score / cap)``.  ``distance_bias``: then ``r1_h * ln(1 + r2_h * (i - j))`` is taken off, two numbers per head (roles ``r1``,
+``r2``).  ``unit_sink``: the denominator holds one more exponential of score 0, without key, value or tensor.
+
 Without a ``window`` every earlier token is seen and there are no pooled rows.  A run step that borrows another's cache uses
 its own queries, window, pool, scale and sink over the owner's rows; when it summarises the same blocks as the owner it
 reads the owner's pooled rows, else it keeps pooled rows of its own (``CacheEntry.fills_pooled``).
@@ -48,7 +53,7 @@ from .linear import linear
 
 _ROLES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight", "q_bias": "q_proj.bias",
           "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "sink": "sink", "q_norm": "q_norm.weight", "k_norm": "k_norm.weight",
-          "gate": "g_proj.weight", "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight"}
+          "gate": "g_proj.weight", "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight", "r1": "distance.r1", "r2": "distance.r2"}
 NO_WINDOW = 1 << 30   # "every earlier token" as a window size
 
 
@@ -84,6 +89,8 @@ class PooledWindowAttention:
             t[nm["gate"]] = TensorInfo((nh, w), "matrix")
         if params.get("value_gate", False):
             t[nm["gate"]] = TensorInfo((nh * dv, w), "matrix")
+        if params.get("distance_bias", False):
+            t[nm["r1"]], t[nm["r2"]] = TensorInfo((nh,), "vector", False, 0.5), TensorInfo((nh,), "vector", False, 0.25)
         taps = params.get("conv_taps")
         if taps:
             for role, ch in (("q_conv", nh * d), ("k_conv", nkv * d), ("v_conv", nkv * dv)):
@@ -141,6 +148,21 @@ class PooledWindowAttention:
         self.k_bias = weights.load(nm["k_bias"], "vector") if bias and self.own_kv else None
         self.v_bias = weights.load(nm["v_bias"], "vector") if bias and self.own_kv else None
         self.sink = weights.load(nm["sink"], "vector") if params.get("sink", False) else None
+        if params.get("unit_sink", False):
+            if self.sink is not None:
+                raise ValueError("pooled_window_attention: a sink with a tensor or one of score 0, not both")
+            self.sink = torch.zeros(self.n_heads, dtype=torch.float32, device=rt.device)
+        self.value_norm = bool(params.get("value_norm", False))
+        qt = params.get("q_temp")
+        self.q_temp = (float(qt["coef"]), int(qt["every"])) if qt else None
+        self.softcap = float(params["softcap"]) if params.get("softcap") is not None else None
+        self.dist_bias = None
+        if params.get("distance_bias", False):
+            self.dist_bias = tuple(weights.load(nm[r], "vector").to(torch.float32).contiguous() for r in ("r1", "r2"))
+        if (self.softcap is not None and not self.softcap > 0.0) or (self.q_temp is not None and self.q_temp[1] < 1):
+            raise ValueError(f"pooled_window_attention: softcap {self.softcap}, query temperature {self.q_temp}")
+        if self.pool and (self.softcap is not None or self.dist_bias is not None):
+            raise ValueError("pooled_window_attention: squashed or biased scores do not go with pooled blocks")
         self.side, self.side_out = None, None      # (first column, columns) of rows that ride with the input product
         pos: PartSpec = params.get("position") or PartSpec("none")
         self.position = POSITIONS.get(pos.kind)(pos.params, self.qk_dim, rt)
@@ -151,6 +173,9 @@ class PooledWindowAttention:
             raise ValueError("pooled_window_attention: the convolution does not go with a norm over the whole projection or the interleaved layout")
         if self.prep_by_token and bias:
             raise ValueError("pooled_window_attention: biases do not go with a norm over the whole projection or the interleaved layout")
+        if (self.prep_by_token or self.taps) and (self.value_norm or self.q_temp is not None):
+            raise ValueError("pooled_window_attention: a value norm or a query temperature does not go with a convolution, a norm over the "
+                             "whole projection or the interleaved layout")
         if self.head_gate:
             K.latent_attn_lib()            # the per-head gate kernel lives beside the other gated attention
         self.rot = int(getattr(self.position, "rotary_dim", 0) or 0) if getattr(self.position, "inv_freq", None) is not None else 0
@@ -210,7 +235,7 @@ class PooledWindowAttention:
             else:
                 K.pool_attn_prep(proj, self.q_bias, self.k_bias, self.v_bias, *freq, ctx.tok_slot, ctx.tok_pos, q, cache.k, cache.v,
                                  cache.page_table, self.n_heads, self.n_kv, unit_eps, owns_cache, conv_w=self.conv_w, ring=ring,
-                                 store_ring=ctx.decode)
+                                 store_ring=ctx.decode, v_eps=self.eps if self.value_norm else -1.0, q_temp=self.q_temp)
             if self.taps > 1 and not ctx.decode:
                 K.conv_ring_store(proj, 0, ctx.cu_q, ctx.seq_slot, ctx.tok_pos, state["conv"], ctx.n_seqs)
         pooled = None
@@ -226,7 +251,8 @@ class PooledWindowAttention:
         gate = proj[:, self.gate_col:self.gate_col + self.o_dim] if self.value_gate else None     # applied inside the attention
         if self.use_prefill_kernel and not ctx.decode and ctx.n_tiles > 0 and cache.k.shape[2] == 64:
             K.pool_attn_prefill(q, cache.k, cache.v, cache.page_table, pooled, self.sink, ctx.tile_tok0, ctx.tile_rows, ctx.tok_slot,
-                                ctx.tok_pos, o, ctx.n_tiles, self.scale, self.size, self.pool, keep=self.keep, gate=gate)
+                                ctx.tok_pos, o, ctx.n_tiles, self.scale, self.size, self.pool, keep=self.keep, gate=gate,
+                                softcap=self.softcap, dist_bias=self.dist_bias)
         else:
             s = self._n_splits(n, ctx.max_kv)
             part_o = part_ml = None
@@ -234,7 +260,8 @@ class PooledWindowAttention:
                 part_o = torch.empty((n, self.n_heads, s, self.v_dim), dtype=torch.float32, device=dev)
                 part_ml = torch.empty((n, self.n_heads, s, 2), dtype=torch.float32, device=dev)
             K.pool_attn_rows(q, cache.k, cache.v, cache.page_table, pooled, self.sink, ctx.tok_slot, ctx.tok_pos, o, self.scale,
-                             self.size, self.pool, s, part_o, part_ml, keep=self.keep, gate=gate)
+                             self.size, self.pool, s, part_o, part_ml, keep=self.keep, gate=gate, softcap=self.softcap,
+                             dist_bias=self.dist_bias)
         o = o.view(n, self.o_dim)
         if self.head_gate:
             K.head_gate_rows(o, proj, self.gate_col, o, self.n_heads, self.v_dim)     # in place: an entry reads only itself
