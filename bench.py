@@ -194,10 +194,10 @@ def prefill_time(eng, tokens, iters, seed):
 
 # ----------------------------------------------------------------------------- two designs at equal size
 def compare_arm(args, warmup) -> int:
-    """Prefill and decode throughput of Tevovik, Vobusun, Mogelix, Kerirax or Dusupel shapes, each beside the shape of equal size (same
+    """Prefill and decode throughput of Tevovik, Vobusun, Mogelix, Kerirax, Dusupel or Puturax shapes, each beside the shape of equal size (same
     width, layers, heads, vocabulary; the dense intermediate size is the expert size times the experts a token uses, or the
     Vobusun feed-forward's own size; a Mogelix shape stands beside the Tevovik shape of its sizes, a Kerirax shape beside
-    the Mogelix shape of its sizes, a Dusupel shape beside the Kerirax shape of its sizes).  One JSON line."""
+    the Mogelix shape of its sizes, a Dusupel or Puturax shape beside the Kerirax shape of its sizes).  One JSON line."""
     import torch
 
     from dryft_b200.config import config_from_dict, preset
@@ -388,9 +388,9 @@ def main() -> int:
     ap.add_argument("--seed", type=int, default=0)
     ap.add_argument("--compare", default=None, metavar="SHAPE[,SHAPE]",
                     help="instead of the default workload: prefill (2,048 tokens) and decode (batch 1 and 8) of these Tevovik, "
-                         "Vobusun, Mogelix, Kerirax or Dusupel presets, each beside the preset of equal size (tevovik-1k, tevovik-2k, vobusun-1k, "
+                         "Vobusun, Mogelix, Kerirax, Dusupel or Puturax presets, each beside the preset of equal size (tevovik-1k, tevovik-2k, vobusun-1k, "
                          "vobusun-2k beside dense Qwen3 shapes; mogelix-1k, mogelix-2k beside the Tevovik shapes; kerirax-1k, "
-                         "kerirax-2k beside the Mogelix shapes; dusupel-1k, dusupel-2k beside the Kerirax shapes)")
+                         "kerirax-2k beside the Mogelix shapes; dusupel-1k, dusupel-2k, puturax-1k, puturax-2k beside the Kerirax shapes)")
     ap.add_argument("--small-m-max", type=int, default=None,
                     help="rows up to which decode products stream weights themselves (the engine's default if not given)")
     ap.add_argument("--engine-opt", action="append", default=[], metavar="NAME=VALUE",

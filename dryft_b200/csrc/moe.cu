@@ -89,7 +89,9 @@ __device__ __forceinline__ void route_one(const float* z, const float* __restric
       if (gs[e / gsz] != -INFINITY) ch[e] = SHUT_OUT;
     __syncwarp();
   }
-  float wsum = 0.f;
+  // lane r keeps choice r (and r + 32, ...: written as they come, scaled in a second pass), so that one store a lane leaves the token
+  float wsum = 0.f, my_w = 0.f;
+  int my_i = 0;
   for (int r = 0; r < top; ++r) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -99,17 +101,19 @@ __device__ __forceinline__ void route_one(const float* z, const float* __restric
     float w = 0.f;
     if (bi >= E) bi = 0;                           // nothing comparable left (a NaN row): a defined choice of weight zero
     else if (bv > SHUT_OUT) w = s[bi];             // else fewer allowed experts than `top`: weight zero
-    if (lane == 0) {
-      idx_out[(size_t)n * top + r] = bi;
-      w_out[(size_t)n * top + r] = w;
-      ch[bi] = -INFINITY;
-    }
+    if (lane == (r & 31)) { my_w = w; my_i = bi; ch[bi] = -INFINITY; }
+    if (top > 32 && lane == (r & 31)) { idx_out[(size_t)n * top + r] = my_i; w_out[(size_t)n * top + r] = my_w; }
     wsum += w;
     __syncwarp();
   }
   wsum += renorm_eps;
-  if (renorm && lane == 0 && wsum > 0.f)
-    for (int r = 0; r < top; ++r) w_out[(size_t)n * top + r] /= wsum;
+  const bool scale = renorm && wsum > 0.f;
+  if (top > 32) {
+    for (int r = lane; scale && r < top; r += 32) w_out[(size_t)n * top + r] /= wsum;      // the lane's own entries
+  } else if (lane < top) {
+    idx_out[(size_t)n * top + lane] = my_i;
+    w_out[(size_t)n * top + lane] = scale ? my_w / wsum : my_w;
+  }
 }
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(

@@ -12,8 +12,10 @@
 //               chunk from a ZERO state, leaving its own state and the product of its decays per key channel; wkv_prefix, per
 //               sequence, start(k+1) = decays_k * start(k) + own(k), which turns the chunks' own states into their start states
 //               and leaves the final state in the slot; MODE 2, every chunk again from its start state, writing o.
-//   wkv_norm    out = T( o / sqrt(mean(o^2) + eps) * norm_w * silu(g) ), the mean over a head's values; and the step's last
-//               inputs into `last`
+//               Where a block holds all of a head's value columns it also norms and gates a tile's read-outs before they leave it:
+//                   out = T( o / sqrt(mean(o^2) + eps) * norm_w * silu(g) )      (the mean over a head's values)
+//               and leaves the step's last inputs in `last`; else
+//   wkv_norm    does both behind the walk
 //   wkv_decode  one token per sequence: tanh, the decay's second product, decay, bonus, read-out, state update, norm, gate and
 //               `last` in ONE launch behind the products; a block per (sequence, head)
 //
@@ -73,7 +75,10 @@ template <typename T, int V> __device__ __forceinline__ void store_piece(T* p, c
 #pragma unroll
     for (int j = 0; j < V; ++j) e[j] = from_f32<T>(f[j]);
 #pragma unroll
-    for (int i = 0; i < V; i += 16 / (int)sizeof(T)) *reinterpret_cast<uint4*>(p + i) = *reinterpret_cast<const uint4*>(e + i);
+    for (int i = 0; i < V; i += 16 / (int)sizeof(T)) {
+      if constexpr (V * sizeof(T) == 8) *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(e);
+      else *reinterpret_cast<uint4*>(p + i) = *reinterpret_cast<const uint4*>(e + i);
+    }
   }
 }
 
@@ -126,11 +131,14 @@ constexpr int COLS = 4;      // value columns a thread's piece of the state has
 
 // RS: threads that share a group of value columns (RS * 16 >= d); blockDim = RS * CG, CG groups of four columns.
 // V: elements a vector load of the operands takes (4, or 1 where sizes are no multiple of four).  TT: tokens staged at once.
+struct Finish { const void* g; const float* norm_w; float eps; const void* h; int width; void *last, *out; };   // out null: the read-outs leave as they are
+
 template <typename T, int RS, int MODE, int V, int TT>
 __global__ void __launch_bounds__(256) wkv_walk_kernel(
     const T* __restrict__ r, const T* __restrict__ k, const T* __restrict__ v, int ld, const float* __restrict__ z,
     const float* __restrict__ w0, const float* __restrict__ u, const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int n_seqs,
-    int cht, int H, int d, int dv, float* __restrict__ state, float* __restrict__ cstate, float* __restrict__ cdecay, float* __restrict__ o) {
+    int cht, int H, int d, int dv, float* __restrict__ state, float* __restrict__ cstate, float* __restrict__ cdecay, float* __restrict__ o,
+    Finish fin) {
   constexpr int DP = RS * ROWS;
   extern __shared__ __align__(16) float sm[];
   const int CG = blockDim.x / RS, CW = CG * COLS;
@@ -141,6 +149,7 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
   float* bs_ = vs_ + TT * CW;               // [TT]
   float* us_ = bs_ + TT;                    // [DP]
   float* w0s = us_ + DP;                    // [DP]
+  float* os_ = w0s + DP;                    // MODE 0 and 2: [TT][CW] read-outs of a tile
   float* ds_ = w0s + DP;                    // MODE 1: [token groups][DP] sums of exp(z + w0)
   int b, ci = 0;
   if (MODE == 0) b = blockIdx.x;
@@ -178,6 +187,7 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
   // staging: LG lanes take a token's key channels, four each
   constexpr int LG = DP / 4 < 32 ? DP / 4 : 32, PER = DP / 4 / LG;      // PER: vectors of four a lane takes
   const int groups = blockDim.x / LG, grp = tid / LG, gl = tid % LG;
+  constexpr int LGV = LG, VPER = PER;                                  // the same for a token's value columns (d = dv there)
   float esum[PER][4];
 #pragma unroll
   for (int p = 0; p < PER; ++p)
@@ -293,12 +303,69 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
           const float bonus = bs_[tt];
 #pragma unroll
           for (int j = 0; j < COLS; ++j)
-            if (j < left && c0 + c + j < dv)
-              o[(size_t)(t0 + tt) * H * dv + voff + c0 + c + j] = fmaf(bonus, vs_[tt * CW + cg * COLS + c + j], a[j]);
+            if (j < left) {
+              const int cc = cg * COLS + c + j;
+              const float y = fmaf(bonus, vs_[tt * CW + cc], a[j]);
+              if (fin.out != nullptr) os_[tt * CW + cc] = y;
+              else if (col0 + cc < dv) o[(size_t)(t0 + tt) * H * dv + voff + col0 + cc] = y;
+            }
         }
       }
     }
     __syncthreads();
+    if (MODE != 1 && fin.out != nullptr) {
+      // a tile's read-outs: LGV lanes a token, four value columns each (columns beyond dv hold zeros)
+      const T* gate = static_cast<const T*>(fin.g);
+      T* out = static_cast<T*>(fin.out);
+      const int vgrp = tid / LGV, vl = tid % LGV, vgroups = blockDim.x / LGV;
+      for (int tt = vgrp; tt < cnt; tt += vgroups) {
+        const size_t at = (size_t)(t0 + tt) * H * dv + voff;
+        float y[VPER][4], gg[VPER][4];
+        float ss = 0.f;
+#pragma unroll
+        for (int p = 0; p < VPER; ++p) {
+          const int c = 4 * (vl + LGV * p);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) { y[p][e] = 0.f; gg[p][e] = 0.f; }
+          if (c < CW) {
+            const float4 y4 = *reinterpret_cast<const float4*>(os_ + tt * CW + c);
+            y[p][0] = y4.x; y[p][1] = y4.y; y[p][2] = y4.z; y[p][3] = y4.w;
+          }
+          if (V == 4) {
+            if (c < dv) load_piece<T, 4>(gate + at + c, gg[p]);
+          } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              if (c + e < dv) gg[p][e] = to_f32<T>(gate[at + c + e]);
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) ss = fmaf(y[p][e], y[p][e], ss);
+        }
+        const unsigned mask = LGV == 32 ? 0xffffffffu : ((1u << LGV) - 1u) << ((tid & 31) / LGV * LGV);
+#pragma unroll
+        for (int s = LGV / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(mask, ss, s);
+        const float rinv = 1.f / sqrtf(ss / (float)dv + fin.eps);
+#pragma unroll
+        for (int p = 0; p < VPER; ++p) {
+          const int c = 4 * (vl + LGV * p);
+          float f[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) f[e] = c + e < dv ? y[p][e] * rinv * fin.norm_w[voff + c + e] * silu(gg[p][e]) : 0.f;
+          if (V == 4) {
+            if (c < dv) store_piece<T, 4>(out + at + c, f);
+          } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              if (c + e < dv) out[at + c + e] = from_f32<T>(f[e]);
+          }
+        }
+      }
+    }
+  }
+  if (MODE != 1 && fin.out != nullptr && t_end == cu_q[b + 1]) {      // the sequence's last token of this step: a slice a head
+    const T* h = static_cast<const T*>(fin.h) + (size_t)(t_end - 1) * fin.width;
+    T* last = static_cast<T*>(fin.last) + (size_t)slot * fin.width;
+    for (int c = hd * blockDim.x + tid; c < fin.width; c += H * blockDim.x) last[c] = h[c];
   }
   // MODE 0: the slot's new state; MODE 1: the chunk's own state
 #pragma unroll
@@ -481,6 +548,7 @@ __global__ void __launch_bounds__(DEC_THREADS) wkv_decode_kernel(
 
 struct Walk {
   const void *r, *k, *v; int ld; const float *z, *w0, *u; const int *cu_q, *seq_slot; int n_seqs, cht, H, d, dv; float *state, *cstate, *cdecay, *o;
+  Finish fin;
 };
 
 template <typename T, int RS, int MODE, int V>
@@ -493,7 +561,7 @@ int walk_mode(const Walk& a, int blocks_x, cudaStream_t st) {
   cg = (cg + unit - 1) / unit * unit;
   if (cg > most) cg = most;
   const int slices = (a.dv + cg * COLS - 1) / (cg * COLS), threads = RS * cg;
-  const size_t smem = sizeof(float) * ((size_t)TT * (3 * DP + cg * COLS + 1) + 2 * DP + (MODE == 1 ? (size_t)(threads / LG) * DP : 0));
+  const size_t smem = sizeof(float) * ((size_t)TT * (3 * DP + cg * COLS + 1) + 2 * DP + (MODE == 1 ? (size_t)(threads / LG) * DP : (size_t)TT * cg * COLS));
   if (smem > 200 * 1024) return DRYFT_ERR_UNSUPPORTED;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(wkv_walk_kernel<T, RS, MODE, V, TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -501,7 +569,7 @@ int walk_mode(const Walk& a, int blocks_x, cudaStream_t st) {
   }
   dim3 grid(blocks_x, a.H, slices);
   wkv_walk_kernel<T, RS, MODE, V, TT><<<grid, threads, smem, st>>>((const T*)a.r, (const T*)a.k, (const T*)a.v, a.ld, a.z, a.w0, a.u, a.cu_q, a.seq_slot,
-                                                                 a.n_seqs, a.cht, a.H, a.d, a.dv, a.state, a.cstate, a.cdecay, a.o);
+                                                                 a.n_seqs, a.cht, a.H, a.d, a.dv, a.state, a.cstate, a.cdecay, a.o, a.fin);
   return launch_status();
 }
 
@@ -520,7 +588,8 @@ int walk_all(const Walk& a, int n_chunks, cudaStream_t st) {
 
 template <typename T>
 int walk_sizes(const Walk& a, int n_chunks, cudaStream_t st) {
-  const bool vec = a.d % 4 == 0 && a.dv % 4 == 0 && a.ld % 4 == 0 && (((uintptr_t)a.r | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.z) & 15) == 0;
+  const bool vec = a.d % 4 == 0 && a.dv % 4 == 0 && a.ld % 4 == 0 &&
+                   (((uintptr_t)a.r | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.z | (uintptr_t)a.fin.g | (uintptr_t)a.fin.out) & 15) == 0;
 #define DRYFT_WALK(RS) return vec ? walk_all<T, RS, 4>(a, n_chunks, st) : walk_all<T, RS, 1>(a, n_chunks, st)
   if (a.d <= 16) { DRYFT_WALK(1); }
   if (a.d <= 32) { DRYFT_WALK(2); }
@@ -557,14 +626,21 @@ DRYFT_API int dryft_wkv_tanh(int is_bf16, const float* low, void* out, long long
   return launch_status();
 }
 
+// head sizes up to this run the norm and the gate inside the walk (a block holds all of a head's value columns)
+DRYFT_API int dryft_wkv_fused_dim() { return 128; }
+
+// `out` given (d = dv up to dryft_wkv_fused_dim): norm, gate and the step's last inputs inside; else the read-outs go to o.
 // n_chunks = 0: the tokens of each sequence in order (one launch); else the chunked form (three launches) with scratch
 // cstate [n_chunks, H, d, dv] and cdecay [n_chunks, H, d], n_chunks at least the number of chunks of `cht` tokens in the step.
 DRYFT_API int dryft_wkv_walk(int is_bf16, const void* r, const void* k, const void* v, int ld, const float* z, const float* w0, const float* u,
                              const int* cu_q, const int* seq_slot, int n_seqs, int cht, int n_chunks, int H, int d, int dv, float* state,
-                             float* cstate, float* cdecay, float* o, cudaStream_t st) {
+                             float* cstate, float* cdecay, float* o, const void* g, const float* norm_w, float eps, const void* h, int width,
+                             void* last, void* out, cudaStream_t st) {
   if (n_seqs <= 0) return 0;
+  if (out == nullptr && o == nullptr) return DRYFT_ERR_UNSUPPORTED;
+  if (out != nullptr && (d != dv || d > dryft_wkv_fused_dim() || ld != H * dv || !g || !norm_w || !h || !last || width < 1)) return DRYFT_ERR_UNSUPPORTED;
   if (H < 1 || H > 65535 || d < 1 || d > 256 || dv < 1 || (n_chunks > 0 && (cht <= 0 || !cstate || !cdecay))) return DRYFT_ERR_UNSUPPORTED;
-  Walk a{r, k, v, ld, z, w0, u, cu_q, seq_slot, n_seqs, cht, H, d, dv, state, cstate, cdecay, o};
+  Walk a{r, k, v, ld, z, w0, u, cu_q, seq_slot, n_seqs, cht, H, d, dv, state, cstate, cdecay, o, {g, norm_w, eps, h, width, last, out}};
   return is_bf16 ? walk_sizes<__nv_bfloat16>(a, n_chunks, st) : walk_sizes<float>(a, n_chunks, st);
 }
 

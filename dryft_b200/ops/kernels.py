@@ -2340,7 +2340,8 @@ def wkv_lib() -> ctypes.CDLL:
     return _single_lib("wkv", {
         "dryft_wkv_mix": [_i, _p, _p, _p, _p, _p, _i, _i, _p],
         "dryft_wkv_tanh": [_i, _p, _p, _ll, _p],
-        "dryft_wkv_walk": [_i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _p, _p, _p, _p],
+        "dryft_wkv_fused_dim": [],
+        "dryft_wkv_walk": [_i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p, _f, _p, _i, _p, _p, _p],
         "dryft_wkv_norm": [_i, _p, _p, _i, _p, _f, _p, _i, _p, _p, _i, _i, _i, _p, _p],
         "dryft_wkv_decode": [_i, _p, _p, _p, _p, _i, _p, _i, _i, _p, _p, _p, _p, _f, _p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _p],
     })
@@ -2383,7 +2384,9 @@ def wkv_tokens(r, k, v, g, z, w0, u, norm_w, eps: float, h, last, ctx, state, ou
     _need(last, "last", h.dtype, (None, width))
     _need(out, "out", h.dtype, (n, heads * dv))
     dev = h.device
-    o = torch.empty((n, heads * dv), dtype=torch.float32, device=dev)
+    lib = wkv_lib()
+    fused = d <= lib.dryft_wkv_fused_dim()       # norm and gate inside the walk
+    o = None if fused else torch.empty((n, heads * dv), dtype=torch.float32, device=dev)
     cht = n_chunks = 0
     cstate = cdecay = None
     if chunked:
@@ -2392,10 +2395,13 @@ def wkv_tokens(r, k, v, g, z, w0, u, norm_w, eps: float, h, last, ctx, state, ou
         cstate = torch.empty((n_chunks, heads, d, dv), dtype=torch.float32, device=dev)
         cdecay = torch.empty((n_chunks, heads, d), dtype=torch.float32, device=dev)
     what = f"({heads} heads of {d})"
-    _ok(wkv_lib().dryft_wkv_walk(_act(h, "h"), _ptr(r), _ptr(k), _ptr(v), heads * d, _ptr(z), _ptr(w0), _ptr(u), _ptr(ctx.cu_q), _ptr(ctx.seq_slot),
-                                 int(ctx.n_seqs), cht, n_chunks, heads, d, dv, _ptr(state), _ptr(cstate), _ptr(cdecay), _ptr(o), _stream()),
+    _ok(lib.dryft_wkv_walk(_act(h, "h"), _ptr(r), _ptr(k), _ptr(v), heads * d, _ptr(z), _ptr(w0), _ptr(u), _ptr(ctx.cu_q), _ptr(ctx.seq_slot),
+                                 int(ctx.n_seqs), cht, n_chunks, heads, d, dv, _ptr(state), _ptr(cstate), _ptr(cdecay), _ptr(o), _ptr(g), _ptr(norm_w), float(eps), _ptr(h),
+                                 width, _ptr(last), _ptr(out if fused else None), _stream()),
         "wkv_walk " + what, n_kernels=3 if chunked else 1)
-    _ok(wkv_lib().dryft_wkv_norm(_act(h, "h"), _ptr(o), _ptr(g), heads * dv, _ptr(norm_w), float(eps), _ptr(h), width, _ptr(last), _ptr(ctx.tok_slot),
+    if fused:
+        return
+    _ok(lib.dryft_wkv_norm(_act(h, "h"), _ptr(o), _ptr(g), heads * dv, _ptr(norm_w), float(eps), _ptr(h), width, _ptr(last), _ptr(ctx.tok_slot),
                                  n, heads, dv, _ptr(out), _stream()), "wkv_norm " + what)
 
 

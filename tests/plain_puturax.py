@@ -216,14 +216,16 @@ def moe_ffn(h: torch.Tensor, mlp: Mapping, w: Mapping[str, torch.Tensor], pre: s
 
 # ----------------------------------------------------------------------------- the model
 def forward(config: Mapping, weights: Mapping[str, torch.Tensor], tokens: List[int],
-            tap: Optional[Callable[[int, torch.Tensor], None]] = None, rounding: Optional[torch.dtype] = None) -> torch.Tensor:
-    """Logits ``[L, vocab]`` of one sequence.  ``tap(layer, x)`` sees the stream after every layer."""
-    global _ROUND
-    _ROUND = rounding
+            tap: Optional[Callable[[int, torch.Tensor], None]] = None, rounding: Optional[torch.dtype] = None,
+            number: torch.dtype = torch.float64) -> torch.Tensor:
+    """Logits ``[L, vocab]`` of one sequence.  ``tap(layer, x)`` sees the stream after every layer.  ``number``: the type everything is
+    evaluated in (float32 shows which rows of a model are ill-conditioned in 32-bit whoever evaluates them)."""
+    global _ROUND, F
+    _ROUND, F = rounding, number
     try:
         return _forward(config, weights, tokens, tap)
     finally:
-        _ROUND = None
+        _ROUND, F = None, torch.float64
 
 
 def _forward(config, weights, tokens, tap):
