@@ -90,6 +90,34 @@ __global__ void relu2_kernel(const T* __restrict__ z, int ldz, T* __restrict__ o
   }
 }
 
+// rows of whole 16-byte vectors: a thread a vector of one row
+template <typename T>
+__global__ void relu2_vec_kernel(const T* __restrict__ z, int ldz, T* __restrict__ out, int F) {
+  constexpr int V = 16 / (int)sizeof(T);
+  const size_t r = blockIdx.x;
+  const int c = ((int)blockIdx.y * blockDim.x + (int)threadIdx.x) * V;
+  if (c >= F) return;
+  const uint4 raw = *reinterpret_cast<const uint4*>(z + r * ldz + c);
+  const T* e = reinterpret_cast<const T*>(&raw);
+  __align__(16) T o[V];
+#pragma unroll
+  for (int i = 0; i < V; ++i) { const float v = fmaxf(to_f32<T>(e[i]), 0.f); o[i] = from_f32<T>(v * v); }
+  *reinterpret_cast<uint4*>(out + r * F + c) = *reinterpret_cast<const uint4*>(o);
+}
+
+template <typename T>
+int relu2_launch(const T* z, int ldz, T* out, int n, int F, cudaStream_t st) {
+  constexpr int V = 16 / (int)sizeof(T);
+  if (F % V == 0 && ldz % V == 0 && (((uintptr_t)z | (uintptr_t)out) & 15) == 0 && F / V <= 65535 * 128) {
+    relu2_vec_kernel<T><<<dim3(n, (F / V + 127) / 128), 128, 0, st>>>(z, ldz, out, F);
+    return launch_status();
+  }
+  const long long total = (long long)n * F;
+  const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+  relu2_kernel<T><<<blocks, 256, 0, st>>>(z, ldz, out, n, F);
+  return launch_status();
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS) gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z,
                                                                        int ldz, const float* __restrict__ w, int part, float eps,
@@ -149,13 +177,8 @@ DRYFT_API int dryft_polynorm(int is_bf16, const void* z, int ldz, const float* c
 DRYFT_API int dryft_relu2(int is_bf16, const void* z, int ldz, void* out, int n, int F, cudaStream_t st) {
   if (n <= 0) return 0;
   if (F < 1 || ldz < F) return DRYFT_ERR_UNSUPPORTED;
-  const long long total = (long long)n * F;
-  const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-  if (is_bf16)
-    relu2_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>((const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, n, F);
-  else
-    relu2_kernel<float><<<blocks, 256, 0, st>>>((const float*)z, ldz, (float*)out, n, F);
-  return launch_status();
+  return is_bf16 ? relu2_launch<__nv_bfloat16>((const __nv_bfloat16*)z, ldz, (__nv_bfloat16*)out, n, F, st)
+                 : relu2_launch<float>((const float*)z, ldz, (float*)out, n, F, st);
 }
 
 DRYFT_API int dryft_gated_group_norm(int is_bf16, const float* y, const float* z, int ldz, const float* w, int parts, float eps,

@@ -12,7 +12,8 @@
 //                 reads stream row rows[r] (no terms then: nothing is written to the stream).
 //   stream_norm_join  y = s0 * y0[n] + s1 * y1[n] + s2 * y2[n] + sum_k wts[n, k] * yr[n * top + k] ;  x32[n] += y / sqrt(mean(y^2) + eps) * factor :
 //                 the norm on a sublayer's OUTPUT; and, when a norm weight is given, h[n] = T( norm of the new row ), the norm in
-//                 front of the sublayer that comes next, in the same launch.  The row stays in shared memory (4 * width bytes).
+//                 front of the sublayer that comes next, in the same launch.  The row stays in registers (widths up to 4,096 in steps of four, everything
+//                 a thread needs requested before the first sum) or in shared memory (4 * width bytes).
 //   pack_pair     out[n] = T([a32[n] | b32[n]]): two 32-bit rows side by side as one operand row of a product
 //   softcap       z <- cap * tanh(z / cap) over 32-bit logits, in place
 //
@@ -229,9 +230,72 @@ __global__ void __launch_bounds__(THREADS) stream_norm_join_kernel(
   }
 }
 
+// The same for widths up to 1024 * NV in steps of four: a thread owns NV vectors of four and asks for its part of the results, the
+// stream and both factors at once, so that the launch is one trip to memory and two block-wide sums long.
+template <typename T, int NV>
+__global__ void __launch_bounds__(THREADS) stream_norm_join_regs_kernel(
+    float* __restrict__ x32, const T* __restrict__ y0, float s0, const T* __restrict__ y1, float s1, const T* __restrict__ y2, float s2,
+    const T* __restrict__ yr, const float* __restrict__ wts, int top, const float* __restrict__ factor, float eps,
+    const float* __restrict__ norm_w, float norm_eps, T* __restrict__ h, int width) {
+  __shared__ float scratch[33];
+  const size_t n = blockIdx.x;
+  float* x = x32 + n * width;
+  float4 y[NV], xv[NV], f[NV], w[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * THREADS + (int)threadIdx.x) * 4;
+    y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < width) {
+      xv[i] = *reinterpret_cast<const float4*>(x + c);
+      f[i] = *reinterpret_cast<const float4*>(factor + c);
+      if (norm_w != nullptr) w[i] = *reinterpret_cast<const float4*>(norm_w + c);
+      auto term = [&](const T* p, float s) {
+        const float4 t = load4<T>(p + c);
+        y[i].x = fmaf(s, t.x, y[i].x); y[i].y = fmaf(s, t.y, y[i].y); y[i].z = fmaf(s, t.z, y[i].z); y[i].w = fmaf(s, t.w, y[i].w);
+      };
+      if (y0 != nullptr) term(y0 + n * width, s0);
+      if (y1 != nullptr) term(y1 + n * width, s1);
+      if (y2 != nullptr) term(y2 + n * width, s2);
+      if (yr != nullptr) {
+#pragma unroll 4
+        for (int k = 0; k < top; ++k) term(yr + (n * top + k) * width, wts[n * top + k]);      // in the order of the choices
+      }
+    }
+    ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
+  }
+  float rinv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * THREADS + (int)threadIdx.x) * 4;
+    if (c < width) {
+      float4 v = xv[i];
+      v.x = fmaf(y[i].x * rinv, f[i].x, v.x); v.y = fmaf(y[i].y * rinv, f[i].y, v.y);
+      v.z = fmaf(y[i].z * rinv, f[i].z, v.z); v.w = fmaf(y[i].w * rinv, f[i].w, v.w);
+      *reinterpret_cast<float4*>(x + c) = v;
+      y[i] = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+  }
+  if (norm_w == nullptr) return;
+  rinv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + norm_eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * THREADS + (int)threadIdx.x) * 4;
+    if (c < width) store4<T>(h + n * width + c, make_float4(y[i].x * rinv * w[i].x, y[i].y * rinv * w[i].y, y[i].z * rinv * w[i].z, y[i].w * rinv * w[i].w));
+  }
+}
+
 template <typename T, int VEC>
 int norm_join_launch(float* x32, const void* y0, float s0, const void* y1, float s1, const void* y2, float s2, const void* yr, const float* wts,
                      int top, const float* factor, float eps, const float* norm_w, float norm_eps, void* h, int n, int width, cudaStream_t st) {
+  if (VEC == 4 && width <= 4096) {
+    auto kernel = width <= 1024 ? stream_norm_join_regs_kernel<T, 1> : width <= 2048 ? stream_norm_join_regs_kernel<T, 2> : stream_norm_join_regs_kernel<T, 4>;
+    kernel<<<n, THREADS, 0, st>>>(x32, (const T*)y0, s0, (const T*)y1, s1, (const T*)y2, s2, (const T*)yr, wts, top, factor, eps, norm_w, norm_eps, (T*)h,
+                                  width);
+    return launch_status();
+  }
   const size_t smem = sizeof(float) * (size_t)width;
   if (smem > 200 * 1024) return DRYFT_ERR_UNSUPPORTED;
   if (smem > 48 * 1024) {

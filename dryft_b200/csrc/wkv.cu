@@ -410,12 +410,19 @@ __global__ void __launch_bounds__(256) wkv_prefix_kernel(const int* __restrict__
   const int nc = (cu_q[b + 1] - cu_q[b] + cht - 1) / cht;
   const size_t row = e / dv;               // (head, key channel)
   float S = state[(size_t)slot * per + e];
-#pragma unroll 4
-  for (int k = 0; k < nc; ++k) {
-    const size_t at = (size_t)(first + k) * per + e;
-    const float own = cstate[at];
-    cstate[at] = S;
-    S = fmaf(cdecay[(size_t)(first + k) * H * d + row], S, own);
+  constexpr int AHEAD = 8;                 // chunks whose states and decays are requested before the first is used
+  for (int k0 = 0; k0 < nc; k0 += AHEAD) {
+    float own[AHEAD], dec[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      own[i] = k0 + i < nc ? cstate[(size_t)(first + k0 + i) * per + e] : 0.f;
+      dec[i] = k0 + i < nc ? cdecay[(size_t)(first + k0 + i) * H * d + row] : 1.f;
+    }
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      if (k0 + i < nc) cstate[(size_t)(first + k0 + i) * per + e] = S;
+      S = fmaf(dec[i], S, own[i]);         // behind the last chunk: 1 * S + 0
+    }
   }
   state[(size_t)slot * per + e] = S;
 }

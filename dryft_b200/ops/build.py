@@ -19,6 +19,7 @@ import shutil
 import subprocess
 import sys
 import tempfile
+import threading
 import time
 from typing import Dict, Iterable, Optional, Sequence
 
@@ -47,7 +48,7 @@ def find_nvcc() -> str:
 def _writable_dir(path: str) -> bool:
     try:
         os.makedirs(path, exist_ok=True)
-        probe = os.path.join(path, f".probe_{os.getpid()}")
+        probe = os.path.join(path, f".probe_{os.getpid()}_{threading.get_ident()}")
         with open(probe, "w"):
             pass
         os.remove(probe)

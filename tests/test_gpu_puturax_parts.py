@@ -330,7 +330,7 @@ def test_products_of_several_mixtures_in_one_launch(m, k, rows, rest):
 
 # ----------------------------------------------------------------------------- the norm on a sublayer's output
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("width, n_terms, top", [(48, 2, 0), (37, 1, 3), (1024, 0, 4), (64, 3, 2), (2052, 1, 0)])
+@pytest.mark.parametrize("width, n_terms, top", [(48, 2, 0), (37, 1, 3), (1024, 0, 4), (64, 3, 2), (2044, 2, 5), (2052, 1, 0), (5000, 1, 2)])
 def test_the_norm_behind_a_sublayer_and_the_one_in_front_of_the_next(dtype, width, n_terms, top):
     g = torch.Generator().manual_seed(width)
     n, eps, eps2 = 9, 1e-4, 3e-3
@@ -351,3 +351,12 @@ def test_the_norm_behind_a_sublayer_and_the_one_in_front_of_the_next(dtype, widt
         assert rel(xs, want) <= 1e-6
         if with_norm:
             assert rel(h, want_h) <= (2e-6 if dtype == torch.float32 else 5e-3)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("n, F_, ld", [(3, 64, 64), (5, 37, 40), (9, 2056, 2064)])
+def test_the_square_of_relu(dtype, n, F_, ld):
+    z = torch.randn(n, ld, generator=torch.Generator().manual_seed(F_)).to(dtype).to(DEV)
+    out = torch.empty((n, F_), dtype=dtype, device=DEV)
+    K().relu2(z[:, :F_], out)
+    assert rel(out, torch.clamp(z[:, :F_].double().cpu(), min=0.0) ** 2) <= (1e-6 if dtype == torch.float32 else 5e-3)
