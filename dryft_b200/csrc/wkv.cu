@@ -126,6 +126,13 @@ __device__ __forceinline__ bool chunk_of(const int* __restrict__ cu_q, int n_seq
   return false;
 }
 
+// N bytes (8 or 16) from global to shared memory behind the threads' backs
+template <int N> __device__ __forceinline__ void cp_async(void* smem, const void* gmem) {
+  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  if constexpr (N == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem));
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(s), "l"(gmem));
+}
+
 constexpr int ROWS = 16;     // key channels a thread's piece of the state has (four groups of four, RS * 4 apart)
 constexpr int COLS = 4;      // value columns a thread's piece of the state has
 
@@ -134,12 +141,13 @@ constexpr int COLS = 4;      // value columns a thread's piece of the state has
 struct Finish { const void* g; const float* norm_w; float eps; const void* h; int width; void *last, *out; };   // out null: the read-outs leave as they are
 
 template <typename T, int RS, int MODE, int V, int TT>
-__global__ void __launch_bounds__(256) wkv_walk_kernel(
+__global__ void __launch_bounds__(256, 2) wkv_walk_kernel(
     const T* __restrict__ r, const T* __restrict__ k, const T* __restrict__ v, int ld, const float* __restrict__ z,
     const float* __restrict__ w0, const float* __restrict__ u, const int* __restrict__ cu_q, const int* __restrict__ seq_slot, int n_seqs,
     int cht, int H, int d, int dv, float* __restrict__ state, float* __restrict__ cstate, float* __restrict__ cdecay, float* __restrict__ o,
     Finish fin) {
   constexpr int DP = RS * ROWS;
+  constexpr int LG = DP / 4 < 32 ? DP / 4 : 32, PER = DP / 4 / LG;      // lanes that share a token's key channels, vectors of four a lane takes
   extern __shared__ __align__(16) float sm[];
   const int CG = blockDim.x / RS, CW = CG * COLS;
   float* rs_ = sm;                          // [TT][DP]
@@ -151,6 +159,12 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
   float* w0s = us_ + DP;                    // [DP]
   float* os_ = w0s + DP;                    // MODE 0 and 2: [TT][CW] read-outs of a tile
   float* ds_ = w0s + DP;                    // MODE 1: [token groups][DP] sums of exp(z + w0)
+  // V = 4: the next tile's operands as they lie in memory, on their way while this tile is walked
+  float* zn = w0s + DP + (MODE == 1 ? (int)blockDim.x / LG * DP : TT * CW);      // [TT][DP]
+  T* kn = reinterpret_cast<T*>(zn + TT * DP);                                    // [TT][DP]
+  T* rn = kn + TT * DP;                                                          // [TT][DP]
+  T* vn = rn + TT * DP;                                                          // [TT][CW]
+  T* gn = vn + TT * CW;                                                          // [2][TT][CW] this tile's and the next one's gates
   int b, ci = 0;
   if (MODE == 0) b = blockIdx.x;
   else if (!chunk_of(cu_q, n_seqs, cht, blockIdx.x, &b, &ci)) return;
@@ -184,8 +198,7 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
     w0s[c] = c < d ? w0[hd * d + c] : 0.f;
   }
 
-  // staging: LG lanes take a token's key channels, four each
-  constexpr int LG = DP / 4 < 32 ? DP / 4 : 32, PER = DP / 4 / LG;      // PER: vectors of four a lane takes
+  // staging: LG lanes take a token's key channels
   const int groups = blockDim.x / LG, grp = tid / LG, gl = tid % LG;
   constexpr int LGV = LG, VPER = PER;                                  // the same for a token's value columns (d = dv there)
   float esum[PER][4];
@@ -194,9 +207,29 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
 #pragma unroll
     for (int e = 0; e < 4; ++e) esum[p][e] = 0.f;
   const size_t hoff = (size_t)hd * d, voff = (size_t)hd * dv;
-  __syncthreads();
+  constexpr int CB = 4 * (int)sizeof(T);     // bytes of four operands
+  auto request = [&](int t0) {
+    const int cnt = min(TT, t_end - t0), dq = d / 4;
+    for (int i = tid; i < cnt * dq; i += blockDim.x) {
+      const int tt = i / dq, c = (i - tt * dq) * 4;
+      const size_t at = (size_t)(t0 + tt) * ld + hoff + c;
+      cp_async<16>(zn + tt * DP + c, z + (size_t)(t0 + tt) * (size_t)(H * d) + hoff + c);
+      cp_async<CB>(kn + tt * DP + c, k + at);
+      if (MODE != 1) cp_async<CB>(rn + tt * DP + c, r + at);
+    }
+    const int vq = min(CW, dv - col0) / 4;
+    for (int i = tid; i < cnt * vq; i += blockDim.x) {
+      const int tt = i / vq, c = (i - tt * vq) * 4;
+      cp_async<CB>(vn + tt * CW + c, v + (size_t)(t0 + tt) * ld + voff + col0 + c);
+      if (MODE != 1 && fin.out != nullptr) cp_async<CB>(gn + (((t0 - t_begin) / TT & 1) * TT + tt) * CW + c, static_cast<const T*>(fin.g) + (size_t)(t0 + tt) * H * dv + voff + c);
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+  if (V == 4 && t_begin < t_end) request(t_begin);
   for (int t0 = t_begin; t0 < t_end; t0 += TT) {
     const int cnt = min(TT, t_end - t0);
+    if (V == 4) asm volatile("cp.async.wait_group 0;");
+    __syncthreads();          // this tile's operands are there, and the tile before has been walked and left
     for (int tt = grp; tt < TT; tt += groups) {       // every lane of a group takes the same turns
       if (tt >= cnt) break;
       const size_t at = (size_t)(t0 + tt);
@@ -207,9 +240,9 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
         float rr[4] = {0.f, 0.f, 0.f, 0.f}, kk[4] = {0.f, 0.f, 0.f, 0.f}, zz[4] = {0.f, 0.f, 0.f, 0.f}, ww[4];
         if (V == 4) {
           if (c < d) {
-            if (MODE != 1) load_piece<T, 4>(r + at * ld + hoff + c, rr);
-            load_piece<T, 4>(k + at * ld + hoff + c, kk);
-            load_piece<float, 4>(z + at * (size_t)(H * d) + hoff + c, zz);
+            if (MODE != 1) load_piece<T, 4>(rn + tt * DP + c, rr);
+            load_piece<T, 4>(kn + tt * DP + c, kk);
+            load_piece<float, 4>(zn + tt * DP + c, zz);
           }
         } else {
 #pragma unroll
@@ -242,7 +275,7 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
       for (int i = tid; i < cnt * CG; i += blockDim.x) {
         const int tt = i / CG, c = (i % CG) * 4;
         float f[4] = {0.f, 0.f, 0.f, 0.f};
-        if (col0 + c < dv) load_piece<T, 4>(v + (size_t)(t0 + tt) * ld + voff + col0 + c, f);
+        if (col0 + c < dv) load_piece<T, 4>(vn + tt * CW + c, f);
         *reinterpret_cast<float4*>(vs_ + tt * CW + c) = make_float4(f[0], f[1], f[2], f[3]);
       }
     } else {
@@ -252,6 +285,7 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
       }
     }
     __syncthreads();
+    if (V == 4 && t0 + TT < t_end) request(t0 + TT);
     for (int tt = 0; tt < cnt; ++tt) {
       const float4 v4 = *reinterpret_cast<const float4*>(vs_ + tt * CW + cg * COLS);
       const pair_t vv[COLS] = {pack2(v4.x, v4.x), pack2(v4.y, v4.y), pack2(v4.z, v4.z), pack2(v4.w, v4.w)};
@@ -332,7 +366,7 @@ __global__ void __launch_bounds__(256) wkv_walk_kernel(
             y[p][0] = y4.x; y[p][1] = y4.y; y[p][2] = y4.z; y[p][3] = y4.w;
           }
           if (V == 4) {
-            if (c < dv) load_piece<T, 4>(gate + at + c, gg[p]);
+            if (c < dv) load_piece<T, 4>(gn + (((t0 - t_begin) / TT & 1) * TT + tt) * CW + c, gg[p]);
           } else {
 #pragma unroll
             for (int e = 0; e < 4; ++e)
@@ -560,7 +594,7 @@ struct Walk {
 
 template <typename T, int RS, int MODE, int V>
 int walk_mode(const Walk& a, int blocks_x, cudaStream_t st) {
-  constexpr int TT = RS <= 4 ? 16 : 8, DP = RS * ROWS, LG = DP / 4 < 32 ? DP / 4 : 32;
+  constexpr int TT = 8, DP = RS * ROWS, LG = DP / 4 < 32 ? DP / 4 : 32;
   int cg = (a.dv + COLS - 1) / COLS;
   const int least = (32 + RS - 1) / RS, most = 256 / RS;
   cg = cg > most ? most : cg;
@@ -568,7 +602,8 @@ int walk_mode(const Walk& a, int blocks_x, cudaStream_t st) {
   cg = (cg + unit - 1) / unit * unit;
   if (cg > most) cg = most;
   const int slices = (a.dv + cg * COLS - 1) / (cg * COLS), threads = RS * cg;
-  const size_t smem = sizeof(float) * ((size_t)TT * (3 * DP + cg * COLS + 1) + 2 * DP + (MODE == 1 ? (size_t)(threads / LG) * DP : (size_t)TT * cg * COLS));
+  const size_t smem = sizeof(float) * ((size_t)TT * (3 * DP + cg * COLS + 1) + 2 * DP + (MODE == 1 ? (size_t)(threads / LG) * DP : (size_t)TT * cg * COLS)) +
+                      (V == 4 ? TT * (sizeof(float) * DP + sizeof(T) * (2 * DP + 3 * (size_t)cg * COLS)) : 0);
   if (smem > 200 * 1024) return DRYFT_ERR_UNSUPPORTED;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(wkv_walk_kernel<T, RS, MODE, V, TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
