@@ -90,7 +90,7 @@ class PooledWindowAttention:
         if params.get("value_gate", False):
             t[nm["gate"]] = TensorInfo((nh * dv, w), "matrix")
         if params.get("distance_bias", False):
-            t[nm["r1"]], t[nm["r2"]] = TensorInfo((nh,), "vector", False, 0.5), TensorInfo((nh,), "vector", False, 0.25)
+            t[nm["r1"]], t[nm["r2"]] = TensorInfo((nh,), "vector"), TensorInfo((nh,), "vector")    # both positive
         taps = params.get("conv_taps")
         if taps:
             for role, ch in (("q_conv", nh * d), ("k_conv", nkv * d), ("v_conv", nkv * dv)):
