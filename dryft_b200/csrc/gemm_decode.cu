@@ -89,7 +89,9 @@ constexpr size_t SMEM_MOST = 164 * 1024;   // one block under the 164 KB cut: L1
 enum Mode { STORE_BF16 = 0, STORE_F32 = 1, RESIDUAL = 2, SILU = 3 };
 // what happens to the activations: nothing; RMSNorm in the prologue (rows normalised into shared memory);
 // or they come weighted already (T(x * w)) and the sums are scaled by inv[m] in the epilogue
-enum Pro { PLAIN = 0, NORMED = 1, SCALED = 2 };
+// GROUPED: plain activations that differ by group of outputs (a form of its own: the plain one stays as lean as it is)
+enum Pro { PLAIN = 0, NORMED = 1, SCALED = 2, GROUPED = 3 };
+__host__ __device__ constexpr bool staged_form(int pro) { return pro == NORMED || pro == SCALED; }
 
 __device__ __forceinline__ uint4 ld_stream(const void* p) {
   uint4 v;
@@ -128,7 +130,7 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
   constexpr int MP = 8 * MB;
   constexpr int WARPS = GW, THREADS = GW * 32, SPW = K / 32 / GW;   // of a group; SPW: 32-wide k steps a warp
   constexpr int RED = WARPS * ROWS * (MP + 1);
-  constexpr int CHUNK = pick_chunk(SPW, MB == 2 && PRO == PLAIN ? 8 : 10);
+  constexpr int CHUNK = pick_chunk(SPW, MB == 2 && !staged_form(PRO) ? 8 : 10);
   constexpr int SPWP = (SPW + CHUNK - 1) / CHUNK * CHUNK;
   extern __shared__ __align__(16) unsigned char smem[];
   // [WARPS][ROWS][MP + 1] partial sums (the norm's weight lies in the same bytes until the first tile is
@@ -287,12 +289,12 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
     __syncthreads();
   }
   // this thread's activation fragments: batch row mb*8 + g, k as for the weights
-  constexpr bool STAGED = PRO != PLAIN;   // the block's activations are in shared memory
+  constexpr bool STAGED = staged_form(PRO);   // the block's activations are in shared memory
   const bf16* a_frag = A + (size_t)g * lda + k_warp;
   const size_t a_mb = (size_t)8 * lda;
-  // where the activations of a tile's group of products start (one group: at A)
+  // where the activations of a tile's group of products start
   auto group_of = [&](int tl) {
-    return grp_rows > 0 ? a_frag + (size_t)min(tl * TILE_N / grp_rows, grp_last) * grp_stride : a_frag;
+    return a_frag + (size_t)min(tl * TILE_N / grp_rows, grp_last) * grp_stride;
   };
   const bf16* a_row[MB];   // STAGED: where batch row mb * 8 + g lies (the row of zeros from rs on)
 #pragma unroll
@@ -300,7 +302,7 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
   // plain activations come from L2 AD steps ahead, in a ring of registers of their own
   constexpr int AD = STAGED ? 1 : pick_ahead(CHUNK, MB == 1 ? 5 : 4);
   uint4 ar[MB][AD];
-  const bf16* a_cur = PRO == PLAIN ? group_of(tile) : a_frag;
+  const bf16* a_cur = PRO == GROUPED ? group_of(tile) : a_frag;
   auto plain_a = [&](const bf16* from, int mb, int step) {
     return mb * 8 + g < M ? ld_prev(reinterpret_cast<const uint4*>(from + mb * a_mb + step * 32)) : zero;
   };
@@ -320,7 +322,7 @@ __global__ void __launch_bounds__(GW * 32 * GROUPS, GW * GROUPS == 8 ? 2 : 1) ge
     const bool has_next = next < n_tiles;
     const bf16 *nw0 = nullptr, *nw1 = nullptr;
     if (has_next) rows_of(next, nw0, nw1);
-    const bf16* a_next = PRO == PLAIN && has_next ? group_of(next) : a_cur;
+    const bf16* a_next = PRO == GROUPED && has_next ? group_of(next) : a_cur;
 
 #pragma unroll
     for (int s = 0; s < SPWP; ++s) {
@@ -443,7 +445,7 @@ int launch4(const void* A, int lda, const void* W, void* C, int ldc, int M, int 
             int rs, int staged, int blocks_per_sm, int grp_rows, int grp_last, long long grp_stride, cudaStream_t st) {
   constexpr int MP = 8 * MB;
   const size_t smem = smem_of<MB, PRO, GROUPS, GW>(staged);
-  const size_t smem_max = smem_of<MB, PRO, GROUPS, GW>(PRO == PLAIN ? 0 : MP);
+  const size_t smem_max = smem_of<MB, PRO, GROUPS, GW>(!staged_form(PRO) ? 0 : MP);
   if (smem + 1024 > SMEM_MOST) return DRYFT_ERR_UNSUPPORTED;
   static bool attr_done = false;  // per instantiation; set by an eager launch before any capture
   if (!attr_done) {
@@ -487,14 +489,14 @@ int launch3(const void* A, int lda, const void* W, void* C, int ldc, int M, int 
             int grp_rows, int grp_last, long long grp_stride, cudaStream_t st) {
   constexpr int MP = 8 * MB;
   const int rs = M < MP ? M : MP;                                  // activation rows there are
-  const int staged = PRO == PLAIN ? 0 : (rs < MP ? rs + 1 : MP);   // and the row of zeros behind them
+  const int staged = !staged_form(PRO) ? 0 : (rs < MP ? rs + 1 : MP);   // and the row of zeros behind them
 #define DRYFT_GO(GROUPS, GW, PER_SM) \
   launch4<MB, MODE, PRO, GROUPS, GW>(A, lda, W, C, ldc, M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, xw_out, pdl, rs, staged, PER_SM, grp_rows, grp_last, grp_stride, st)
   constexpr int WIDE = (K % 512 == 0 && K / 512 >= 8 && PRO != SCALED) ? 16 : 8;   // 16 warps on one tile where a warp keeps 8 steps
   const int n_tiles = MODE == SILU ? (N + 7) / 8 : (N + ROWS - 1) / ROWS;
   // (decided by what 8 / 16 rows would need, not by M: the split of K, and with it the order of the sums,
   // is then the same for every M up to 8, and for every M from 9 to 16)
-  if (WIDE == 16 && n_tiles >= 2 * sm_count() && smem_of<MB, PRO, 1, WIDE>(PRO == PLAIN ? 0 : MP) + 1024 <= CARVEOUT_BYTES)
+  if (WIDE == 16 && n_tiles >= 2 * sm_count() && smem_of<MB, PRO, 1, WIDE>(!staged_form(PRO) ? 0 : MP) + 1024 <= CARVEOUT_BYTES)
     return DRYFT_GO(1, WIDE, 1);
   if (PRO != NORMED && 2 * (smem_of<MB, PRO, 1, 8>(staged) + 1024) <= CARVEOUT_BYTES) return DRYFT_GO(1, 8, 2);
   if (PRO == NORMED && smem_of<MB, PRO, 2, 8>(staged) + 1024 <= CARVEOUT_BYTES) return DRYFT_GO((PRO == NORMED ? 2 : 1), 8, 1);
@@ -519,7 +521,7 @@ template <int MB>
 int launch1(int mode, int pro, const Args& a) {
   switch (mode) {
     case STORE_BF16: return launch2<MB, STORE_BF16>(pro, a);
-    case STORE_F32: return launch2<MB, STORE_F32>(pro, a);
+    case STORE_F32: return pro == GROUPED ? launch_a<MB, STORE_F32, GROUPED>(a) : launch2<MB, STORE_F32>(pro, a);
     case RESIDUAL: return launch2<MB, RESIDUAL>(pro, a);
     case SILU: return launch2<MB, SILU>(pro, a);
   }
@@ -534,7 +536,7 @@ DRYFT_API int dryft_gemm_decode_k() { return K; }
 // next_w [N] and xw_out [M, ldc], the weighted activations T(x * next_w) for the product after it.
 // scaled != 0: A holds such weighted activations; the sums are scaled by rsqrt(mean(x^2) + eps) from
 // ss_in (norm_w is not read).
-// grp_rows > 0 (a multiple of 16): products of several activations in one launch, see the top of this file; grp_count groups.
+// grp_rows > 0 (a multiple of 16): products of several activations in one launch, see the top of this file; grp_count groups; 32-bit results.
 DRYFT_API int dryft_gemm_decode(const void* A, int lda, const void* W, void* C, int ldc, int mode, int M, int N,
                                 const float* norm_w, const float* ss_in, int ss_parts, float eps, float* ss_out, int pdl,
                                 int scaled, const float* next_w, void* xw_out, int grp_rows, int grp_count, long long grp_stride,
@@ -542,11 +544,11 @@ DRYFT_API int dryft_gemm_decode(const void* A, int lda, const void* W, void* C, 
   if (M <= 0 || N <= 0) return 0;
   if ((lda & 7) || M > 16) return DRYFT_ERR_UNSUPPORTED;
   if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return DRYFT_ERR_UNSUPPORTED;
-  const int pro = scaled ? SCALED : (norm_w != nullptr ? NORMED : PLAIN);
-  if (pro != PLAIN && (!ss_in || ss_parts <= 0)) return DRYFT_ERR_UNSUPPORTED;
+  const int pro = scaled ? SCALED : (norm_w != nullptr ? NORMED : (grp_rows > 0 ? GROUPED : PLAIN));
+  if (staged_form(pro) && (!ss_in || ss_parts <= 0)) return DRYFT_ERR_UNSUPPORTED;
   if (pro == NORMED && ((uintptr_t)norm_w & 15)) return DRYFT_ERR_UNSUPPORTED;
   if ((xw_out != nullptr) != (next_w != nullptr) || (xw_out && mode != RESIDUAL)) return DRYFT_ERR_UNSUPPORTED;
-  if (grp_rows < 0 || (grp_rows > 0 && (grp_rows % ROWS || grp_count < 1 || (grp_stride & 7) || pro != PLAIN || mode == SILU)))
+  if (grp_rows < 0 || (grp_rows > 0 && (grp_rows % ROWS || grp_count < 1 || (grp_stride & 7) || pro != GROUPED || mode != STORE_F32)))
     return DRYFT_ERR_UNSUPPORTED;
   Args a = {A, lda, W, C, ldc, M, N, norm_w, ss_in, ss_parts, eps, ss_out, next_w, xw_out, pdl, grp_rows, grp_count - 1,
             grp_stride, st};
